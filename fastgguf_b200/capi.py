@@ -273,10 +273,10 @@ def kernel_modules_for(spec_json, dtype_code: int) -> tuple:
                 and p.get("v_head_dim", 0) <= p.get("head_dim", 0) + p.get("rot_dim", 0):
             fast_attention = True
     builtin = {"gqa_attention", "swiglu", "retention", "mlp", "moe", "gated_linear_attention", "sink_attention", "latent_attention", "mixer_pair",
-               "state_space", "gated_delta", None}
+               "state_space", "gated_delta", "rglru", None}
     if dtype_code == FG_BF16 and (fast_attention or kinds - builtin):
         modules.append("attn")
-    if kinds & {"retention", "moe", "gated_linear_attention", "sink_attention", "latent_attention", "state_space", "gated_delta"}:
+    if kinds & {"retention", "moe", "gated_linear_attention", "sink_attention", "latent_attention", "state_space", "gated_delta", "rglru"}:
         modules.append("mix")
     return tuple(modules)
 

@@ -5,5 +5,6 @@ from .zirivik import ZirivikConfig
 from .salulorn import SalulornConfig
 from .pirozen import PirozenConfig
 from .saluzen import SaluzenConfig
+from .zifelorn import ZifelornConfig
 
-__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "ZirivikConfig", "SalulornConfig", "PirozenConfig", "SaluzenConfig", "architecture_name", "read_config_json"]
+__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "ZirivikConfig", "SalulornConfig", "PirozenConfig", "SaluzenConfig", "ZifelornConfig", "architecture_name", "read_config_json"]

@@ -294,6 +294,7 @@ extern "C" int fg_kv_append(const void *qkv, int dtype, int ld, int k_off, const
 // For blocks that normalise a sublayer's output before adding it: x[m] += t[m] / rms(t[m]) * w_post, and,
 // when w_next is given, out[m] = x[m] / rms(x[m]) * w_next for the sublayer that reads x next - one pass over
 // the row instead of three kernels.  Statistics and the sum are 32-bit; one block a row, fixed reduction order.
+// Without w_next, out (when given) receives the updated x[m] itself: the input of a sublayer that reads the stream as it is.
 // VEC: rows are read and written four elements at a time (E % 4 == 0, 16-byte aligned rows)
 template <typename TO, bool VEC>
 __global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *__restrict__ w_post, float *__restrict__ x,
@@ -322,12 +323,14 @@ __global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *_
             v.x += a.x * inv * g.x; v.y += a.y * inv * g.y; v.z += a.z * inv * g.z; v.w += a.w * inv * g.w;
             x4[i] = v;
             if (w_next) { r4[i] = v; ss2 += v.x * v.x; ss2 += v.y * v.y; ss2 += v.z * v.z; ss2 += v.w * v.w; }
+            else if (out) store4<TO>(out + base + 4 * i, v.x, v.y, v.z, v.w);
         }
     } else {
         for (int i = threadIdx.x; i < E; i += blockDim.x) {
             float v = x[base + i] + t[base + i] * inv * w_post[i];
             x[base + i] = v;
             if (w_next) { row[i] = v; ss2 += v * v; }
+            else if (out) out[base + i] = from_f32<TO>(v);
         }
     }
     if (!w_next) return;
@@ -352,7 +355,7 @@ extern "C" int fg_norm_add_norm(const float *t, const float *w_post, float *x, c
     const bool vec = E % 4 == 0 && ((((uintptr_t)t) | ((uintptr_t)w_post) | ((uintptr_t)x) | ((uintptr_t)w_next) | ((uintptr_t)out)) & 15) == 0;
     int per = vec ? E / 4 : E;
     int threads = per >= 1024 ? 256 : (per >= 256 ? 128 : 64);
-    const bool wide = out_dtype == FG_F32 || !w_next;
+    const bool wide = out_dtype == FG_F32 || (!w_next && !out);
     if (!wide && out_dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
 #define NAN_LAUNCH(TO, VEC) fg_launch(norm_add_norm_kernel<TO, VEC>, dim3(M), dim3(threads), smem, stream, t, w_post, x, w_next, (TO *)out, E, \
                                       eps_post, eps_next)
@@ -444,10 +447,14 @@ extern "C" int fg_softcap(float *logits, int R, int V, int ld, float cap, cudaSt
     return fg_launch(softcap_kernel, dim3(blocks), dim3(256), 0, stream, logits, V, ld, total, cap, 1.0f / cap);
 }
 
-// ------------------------------------------------------------------ SiLU(g) * u
-// gu: [M, 2F] rows of (gate | up); out: [M, F].
-template <typename T>
-__global__ void silu_mul_kernel(const T *__restrict__ gu, T *__restrict__ out, size_t total, int F) {
+// ------------------------------------------------------------------ act(g) * u
+// gu: [M, 2F] rows of (gate | up); out: [M, F].  act: SiLU, or the tanh form of gelu.
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+template <typename T, bool GELU>
+__global__ void gated_mul_kernel(const T *__restrict__ gu, T *__restrict__ out, size_t total, int F) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -456,23 +463,26 @@ __global__ void silu_mul_kernel(const T *__restrict__ gu, T *__restrict__ out, s
         size_t m = i / F;
         int f = (int)(i - m * F);
         float g = to_f32<T>(gu[m * 2 * F + f]), u = to_f32<T>(gu[m * 2 * F + F + f]);
-        out[i] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+        out[i] = from_f32<T>(GELU ? gelu_tanh_f32(g) * u : g / (1.0f + expf(-g)) * u);
     }
 }
 
-extern "C" int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) {
+template <bool GELU>
+static int gated_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) {
     size_t total = (size_t)M * F;
     if (total == 0) return 0;
     int threads = 256;
     size_t want = (total + threads - 1) / threads;
     int blocks = (int)(want > 148 * 16 ? 148 * 16 : want);
     if (dtype == FG_F32)
-        return fg_launch(silu_mul_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float *)gu, (float *)out, total, F);
-    else if (dtype == FG_BF16)
-        return fg_launch(silu_mul_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream, (const bf16 *)gu, (bf16 *)out, total, F);
-    else return FG_ERR_BAD_DTYPE;
-    return FG_LAUNCH_CHECK();
+        return fg_launch(gated_mul_kernel<float, GELU>, dim3(blocks), dim3(threads), 0, stream, (const float *)gu, (float *)out, total, F);
+    if (dtype == FG_BF16)
+        return fg_launch(gated_mul_kernel<bf16, GELU>, dim3(blocks), dim3(threads), 0, stream, (const bf16 *)gu, (bf16 *)out, total, F);
+    return FG_ERR_BAD_DTYPE;
 }
+
+extern "C" int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<false>(gu, out, dtype, M, F, stream); }
+extern "C" int fg_gelu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<true>(gu, out, dtype, M, F, stream); }
 
 // ------------------------------------------------------------------ decode feedback
 // After a decode step of a fixed-shape (graph-replayed) batch: the sampled token of every row
@@ -618,9 +628,6 @@ extern "C" int fg_cast_rows(const float *x, int ldx, void *out, int out_dtype, i
 // ------------------------------------------------------------------ gelu(z) * (a slice of a token's row of a table)
 // out[m, j] = gelu_tanh(z[m, j]) * table[tokens[m], col0 + j], j < D, with
 // gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).  z is float32; the product is formed in float32.
-__device__ __forceinline__ float gelu_tanh_f32(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
 
 template <typename TT, typename TO>
 __global__ void gelu_mul_gather_kernel(const float *__restrict__ z, int ldz, const TT *__restrict__ table, int ldt, int col0,

@@ -6,6 +6,9 @@
 //   and since both first contractions are linear in x, s_e is applied to their float32 results instead of to h.
 //   act, kind 0:  g = min(g, limit), u = clamp(u, -limit, limit), y = g * sigmoid(alpha g) * (u + 1).
 //
+// Other routers and experts stand beside this one, see their kernels: softmax scores with a selection bias and groups, softmax
+// over the chosen logits alone, weights on the experts' OUTPUTS, and experts of two matrices, W_down max(W_up x, 0)^2.
+//
 // Layout.  A "pair" p = row * top + k is a row's k-th choice.  route() writes the pair's expert and weight and groups
 // pairs by expert: `order[slot] = pair`, `slot_of[pair] = slot`, expert e owning slots [offsets[e], offsets[e + 1]).
 // The contractions run over slots, so that a tile of rows shares one expert's weights; all sizes that depend on the
@@ -14,12 +17,13 @@
 // tile or slot its row lands in, and a row's experts are added in the order of its choices, so a row's result does not
 // depend on what else is in the step.
 //
-// Weights: w_in [X, 2F, E] (gate rows, then up rows, of each expert), w_out [X, E, F]; activations and weights share
+// Weights: w_in [X, 2F, E] (gate rows, then up rows, of each expert; [X, F, E] where an expert has no gate), w_out [X, E, F];
+// activations and weights share
 // the engine's dtype T, accumulation is float32.
 #include "common.cuh"
 
 #define MOE_MAX_EXPERTS 256
-#define MOE_MAX_TOP 8
+#define MOE_MAX_TOP 16
 
 // ------------------------------------------------------------------ router logits
 // z[m, e] = x[m] . W[e], float32 accumulation of the inputs as they are.  A block per row: every thread takes runs of
@@ -84,9 +88,10 @@ extern "C" int fg_moe_logits(const void *x, int ldx, const void *W, int ldw, int
 }
 
 // ------------------------------------------------------------------ routing
-// One block.  logits: [M, X] float32.
+// One block.  logits: [M, X] float32, to which `bias` (a float per output, or null) is added first.  chosen_softmax: the weights
+// are the softmax over the chosen logits alone; else each choice weighs in with the sigmoid of its logit.
 __global__ void __launch_bounds__(1024)
-moe_route_kernel(const float *__restrict__ logits, int M, int X, int top, int *__restrict__ pair_expert, float *__restrict__ pair_weight,
+moe_route_kernel(const float *__restrict__ logits, const float *__restrict__ bias, int chosen_softmax, int M, int X, int top, int *__restrict__ pair_expert, float *__restrict__ pair_weight,
                  int *__restrict__ offsets, int *__restrict__ order, int *__restrict__ slot_of) {
     __shared__ int counts[MOE_MAX_EXPERTS], cursor[MOE_MAX_EXPERTS];
     pdl_launch_dependents();
@@ -96,6 +101,7 @@ moe_route_kernel(const float *__restrict__ logits, int M, int X, int top, int *_
     for (int r = threadIdx.x; r < M; r += blockDim.x) {
         const float *z = logits + (size_t)r * X;
         int chosen[MOE_MAX_TOP];
+        float z_of[MOE_MAX_TOP];
         for (int k = 0; k < top; k++) {
             int best = -1;
             float bz = 0.f;
@@ -103,13 +109,19 @@ moe_route_kernel(const float *__restrict__ logits, int M, int X, int top, int *_
                 bool taken = false;
                 for (int q = 0; q < k; q++) taken = taken || chosen[q] == e;
                 if (taken) continue;
-                float v = z[e];
+                float v = bias ? z[e] + bias[e] : z[e];
                 if (best < 0 || v > bz) { best = e; bz = v; }       // sigmoid is monotonic: the largest logit; ties to the lower index
             }
             chosen[k] = best;
+            z_of[k] = bz;
             pair_expert[(size_t)r * top + k] = best;
-            pair_weight[(size_t)r * top + k] = 1.0f / (1.0f + expf(-bz));
+            if (!chosen_softmax) pair_weight[(size_t)r * top + k] = 1.0f / (1.0f + expf(-bz));
             atomicAdd(&counts[best], 1);
+        }
+        if (chosen_softmax) {                      // (the first choice has the largest logit)
+            float sum = 0.f;
+            for (int k = 0; k < top; k++) sum += expf(z_of[k] - z_of[0]);
+            for (int k = 0; k < top; k++) pair_weight[(size_t)r * top + k] = expf(z_of[k] - z_of[0]) / sum;
         }
     }
     __syncthreads();
@@ -126,13 +138,18 @@ moe_route_kernel(const float *__restrict__ logits, int M, int X, int top, int *_
     }
 }
 
-extern "C" int fg_moe_route(const float *logits, int M, int X, int top, int *pair_expert, float *pair_weight, int *offsets, int *order,
-                            int *slot_of, cudaStream_t stream) {
+extern "C" int fg_moe_route_ext(const float *logits, const float *bias, int chosen_softmax, int M, int X, int top, int *pair_expert,
+                                float *pair_weight, int *offsets, int *order, int *slot_of, cudaStream_t stream) {
     if (M <= 0) return 0;
     if (X <= 0 || X > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP || top > X) return FG_ERR_BAD_SIZE;
     int threads = M >= 1024 ? 1024 : ((M + 31) / 32) * 32;
-    return fg_launch(moe_route_kernel, dim3(1), dim3(threads), 0, stream, logits, M, X, top, pair_expert, pair_weight, offsets, order,
-                     slot_of);
+    return fg_launch(moe_route_kernel, dim3(1), dim3(threads), 0, stream, logits, bias, chosen_softmax, M, X, top, pair_expert, pair_weight, offsets,
+                     order, slot_of);
+}
+
+extern "C" int fg_moe_route(const float *logits, int M, int X, int top, int *pair_expert, float *pair_weight, int *offsets, int *order,
+                            int *slot_of, cudaStream_t stream) {
+    return fg_moe_route_ext(logits, nullptr, 0, M, X, top, pair_expert, pair_weight, offsets, order, slot_of, stream);
 }
 
 // ------------------------------------------------------------------ routing, kind 1: softmax scores, a selection bias, groups
@@ -253,6 +270,16 @@ __device__ __forceinline__ float expert_act(float g, float u, float limit, float
     return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
 }
 
+// What a contraction of the experts is: the second one (W_down over slots, float32 out), the first one of gated experts (two
+// matrices an expert, over the rows behind the slots), or the first one of experts with one input matrix, max(z, 0)^2 behind it.
+enum { MOE_SECOND = 0, MOE_FIRST_GATED = 1, MOE_FIRST_RELU2 = 2 };
+#define MOE_KIND_FLAGS constexpr bool FIRST = KIND != MOE_SECOND, GATED = KIND == MOE_FIRST_GATED
+template <int KIND>
+__device__ __forceinline__ float first_act(float g, float u, float limit, float alpha) {
+    if (KIND == MOE_FIRST_RELU2) return g > 0.f ? g * g : 0.f;
+    return expert_act(g, u, limit, alpha);
+}
+
 // ------------------------------------------------------------------ tiles of 64 slots x 64 outputs on the FMA units
 // The tile of a block: walk the experts, each padded to whole tiles; blocks beyond the last tile leave.
 #define MT 64
@@ -268,12 +295,13 @@ __device__ __forceinline__ bool moe_find_tile(const int *__restrict__ offsets, i
 }
 
 // FIRST: y[slot, n] = act(w (x . gate_n), w (x . up_n)) with x = xn[pair / top]; else out[slot, n] = y[slot] . down_n
-template <typename T, bool FIRST>
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
 moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void *__restrict__ out, int ldo,
                 const int *__restrict__ offsets, const int *__restrict__ order, const float *__restrict__ pair_weight, int X, int top,
                 int N, int K, float limit, float alpha) {
-    __shared__ float As[MK][MT + 1], Bs[FIRST ? 2 : 1][MK][MT + 1];
+    MOE_KIND_FLAGS;
+    __shared__ float As[MK][MT + 1], Bs[GATED ? 2 : 1][MK][MT + 1];
     __shared__ int arow[MT];
     pdl_launch_dependents();
     pdl_wait();
@@ -282,9 +310,9 @@ moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
     const int n0 = blockIdx.x * MT, tid = threadIdx.x;
     if (tid < MT) arow[tid] = s0 + tid < s1 ? (FIRST ? order[s0 + tid] / top : s0 + tid) : -1;
     __syncthreads();
-    const T *We = W + (size_t)e * (FIRST ? 2 : 1) * N * K;
+    const T *We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
     const int tx = tid & 15, ty = tid >> 4;          // outputs n0 + tx + 16 j, slots s0 + ty + 16 i
-    float acc[FIRST ? 2 : 1][4][4] = {};
+    float acc[GATED ? 2 : 1][4][4] = {};
     for (int k0 = 0; k0 < K; k0 += MK) {
         for (int i = tid; i < MT * MK; i += 256) {
             const int r = i / MK, k = i % MK;
@@ -292,7 +320,7 @@ moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
             As[k][r] = (ar >= 0 && k0 + k < K) ? to_f32<T>(A[(size_t)ar * lda + k0 + k]) : 0.f;
             const bool ok = n0 + r < N && k0 + k < K;
             Bs[0][k][r] = ok ? to_f32<T>(We[(size_t)(n0 + r) * K + k0 + k]) : 0.f;
-            if (FIRST) Bs[FIRST ? 1 : 0][k][r] = ok ? to_f32<T>(We[(size_t)(N + n0 + r) * K + k0 + k]) : 0.f;
+            if (GATED) Bs[GATED ? 1 : 0][k][r] = ok ? to_f32<T>(We[(size_t)(N + n0 + r) * K + k0 + k]) : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -301,13 +329,13 @@ moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
 #pragma unroll
             for (int i = 0; i < 4; i++) a[i] = As[k][ty + 16 * i];
 #pragma unroll
-            for (int j = 0; j < 4; j++) { b[j] = Bs[0][k][tx + 16 * j]; b2[j] = FIRST ? Bs[FIRST ? 1 : 0][k][tx + 16 * j] : 0.f; }
+            for (int j = 0; j < 4; j++) { b[j] = Bs[0][k][tx + 16 * j]; b2[j] = GATED ? Bs[GATED ? 1 : 0][k][tx + 16 * j] : 0.f; }
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     acc[0][i][j] = fmaf(a[i], b[j], acc[0][i][j]);
-                    if (FIRST) acc[FIRST ? 1 : 0][i][j] = fmaf(a[i], b2[j], acc[FIRST ? 1 : 0][i][j]);
+                    if (GATED) acc[GATED ? 1 : 0][i][j] = fmaf(a[i], b2[j], acc[GATED ? 1 : 0][i][j]);
                 }
         }
         __syncthreads();
@@ -321,7 +349,7 @@ moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx + 16 * j;
             if (n >= N) continue;
-            if (FIRST) ((T *)out)[(size_t)slot * ldo + n] = from_f32<T>(expert_act(w * acc[0][i][j], w * acc[FIRST ? 1 : 0][i][j], limit, alpha));
+            if (FIRST) ((T *)out)[(size_t)slot * ldo + n] = from_f32<T>(first_act<KIND>(w * acc[0][i][j], w * acc[GATED ? 1 : 0][i][j], limit, alpha));
             else ((float *)out)[(size_t)slot * ldo + n] = acc[0][i][j];
         }
     }
@@ -331,12 +359,13 @@ moe_tile_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
 // (Pairs of one expert read the same rows at about the same time, so the second reader finds them in L2.  The kernel
 // further down reads an expert's rows once for all its slots; this one takes what that one refuses.)
 // output rows a warp takes together: gate and up double the loads of a row, so two there and four for down
-#define MR_ROWS_OF(FIRST) ((FIRST) ? 2 : 4)
-template <typename T, bool FIRST>
+#define MR_ROWS_OF(KIND) ((KIND) == MOE_FIRST_GATED ? 2 : 4)
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
 moe_rows_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void *__restrict__ out, int ldo,
                 const int *__restrict__ pair_expert, const int *__restrict__ order, const float *__restrict__ pair_weight, int top,
                 int X, int N, int K, float limit, float alpha) {
+    MOE_KIND_FLAGS;
     extern __shared__ __align__(16) float xs[];      // [K] the slot's input row
     pdl_launch_dependents();
     pdl_wait();
@@ -346,11 +375,11 @@ moe_rows_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
     for (int k = threadIdx.x; k < K; k += 256) xs[k] = to_f32<T>(a[k]);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const T *We = W + (size_t)e * (FIRST ? 2 : 1) * N * K;
+    const T *We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
     const float w = (FIRST && pair_weight) ? pair_weight[pair] : 1.0f;
     constexpr int VEC = 16 / (int)sizeof(T);         // elements a 16-byte load brings
     const bool vec = (K % VEC) == 0 && (((uintptr_t)W) & 15) == 0;
-    constexpr int MR_ROWS = MR_ROWS_OF(FIRST);
+    constexpr int MR_ROWS = MR_ROWS_OF(KIND);
     // a warp takes MR_ROWS neighbouring output rows at a time: their weight rows are fetched together, so that many
     // 16-byte loads are in flight in every lane
     for (int n0 = (blockIdx.x * 8 + warp) * MR_ROWS; n0 < N; n0 += gridDim.x * 8 * MR_ROWS) {
@@ -365,7 +394,7 @@ moe_rows_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
                 for (int r = 0; r < MR_ROWS; r++) {
                     const int n = min(n0 + r, N - 1);                  // rows past the end repeat the last one; never stored
                     gv[r] = *(const uint4 *)(We + (size_t)n * K + k);
-                    if (FIRST) uv[r] = *(const uint4 *)(We + (size_t)(N + n) * K + k);
+                    if (GATED) uv[r] = *(const uint4 *)(We + (size_t)(N + n) * K + k);
                 }
                 float x[VEC];
 #pragma unroll
@@ -376,7 +405,7 @@ moe_rows_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
 #pragma unroll
                     for (int i = 0; i < VEC; i++) {
                         sg[r] = fmaf(x[i], to_f32<T>(ge[i]), sg[r]);
-                        if (FIRST) su[r] = fmaf(x[i], to_f32<T>(ue[i]), su[r]);
+                        if (GATED) su[r] = fmaf(x[i], to_f32<T>(ue[i]), su[r]);
                     }
                 }
             }
@@ -386,21 +415,21 @@ moe_rows_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void 
                 for (int r = 0; r < MR_ROWS; r++) {
                     const int n = min(n0 + r, N - 1);
                     sg[r] = fmaf(xs[k], to_f32<T>(We[(size_t)n * K + k]), sg[r]);
-                    if (FIRST) su[r] = fmaf(xs[k], to_f32<T>(We[(size_t)(N + n) * K + k]), su[r]);
+                    if (GATED) su[r] = fmaf(xs[k], to_f32<T>(We[(size_t)(N + n) * K + k]), su[r]);
                 }
             }
         }
 #pragma unroll
         for (int r = 0; r < MR_ROWS; r++) {
             sg[r] = warp_sum(sg[r]);
-            if (FIRST) su[r] = warp_sum(su[r]);
+            if (GATED) su[r] = warp_sum(su[r]);
         }
         if (lane == 0) {
 #pragma unroll
             for (int r = 0; r < MR_ROWS; r++) {
                 const int n = n0 + r;
                 if (n >= N) break;
-                if (FIRST) ((T *)out)[(size_t)slot * ldo + n] = from_f32<T>(expert_act(w * sg[r], w * su[r], limit, alpha));
+                if (FIRST) ((T *)out)[(size_t)slot * ldo + n] = from_f32<T>(first_act<KIND>(w * sg[r], w * su[r], limit, alpha));
                 else ((float *)out)[(size_t)slot * ldo + n] = sg[r];
             }
         }
@@ -419,10 +448,11 @@ static bool moe_grouped_enabled() {
     if (v < 0) { const char *e = getenv("FASTGGUF_MOE_GROUPED"); v = !(e && e[0] == '0'); }
     return v != 0;
 }
-template <typename T, bool FIRST, int CNT>
+template <typename T, int KIND, int CNT>
 __device__ __forceinline__ void moe_group_rows(const T *__restrict__ We, const float *xs, void *__restrict__ out, int ldo, int s0,
                                                const float (&w)[MG_SLOTS], int N, int K, float limit, float alpha, int n0, int lane) {
-    constexpr int R = MR_ROWS_OF(FIRST), VEC = 16 / (int)sizeof(T);
+    MOE_KIND_FLAGS;
+    constexpr int R = MR_ROWS_OF(KIND), VEC = 16 / (int)sizeof(T);
     float sg[CNT][R], su[CNT][R];
 #pragma unroll
     for (int i = 0; i < CNT; i++)
@@ -435,7 +465,7 @@ __device__ __forceinline__ void moe_group_rows(const T *__restrict__ We, const f
         for (int r = 0; r < R; r++) {
             const int n = min(n0 + r, N - 1);
             gv[r] = *(const uint4 *)(We + (size_t)n * K + k);
-            if (FIRST) uv[r] = *(const uint4 *)(We + (size_t)(N + n) * K + k);
+            if (GATED) uv[r] = *(const uint4 *)(We + (size_t)(N + n) * K + k);
         }
 #pragma unroll
         for (int i = 0; i < CNT; i++) {
@@ -448,7 +478,7 @@ __device__ __forceinline__ void moe_group_rows(const T *__restrict__ We, const f
 #pragma unroll
                 for (int j = 0; j < VEC; j++) {
                     sg[i][r] = fmaf(x[j], to_f32<T>(ge[j]), sg[i][r]);
-                    if (FIRST) su[i][r] = fmaf(x[j], to_f32<T>(ue[j]), su[i][r]);
+                    if (GATED) su[i][r] = fmaf(x[j], to_f32<T>(ue[j]), su[i][r]);
                 }
             }
         }
@@ -458,7 +488,7 @@ __device__ __forceinline__ void moe_group_rows(const T *__restrict__ We, const f
 #pragma unroll
         for (int r = 0; r < R; r++) {
             sg[i][r] = warp_sum(sg[i][r]);
-            if (FIRST) su[i][r] = warp_sum(su[i][r]);
+            if (GATED) su[i][r] = warp_sum(su[i][r]);
         }
     if (lane == 0) {
 #pragma unroll
@@ -467,25 +497,26 @@ __device__ __forceinline__ void moe_group_rows(const T *__restrict__ We, const f
             for (int r = 0; r < R; r++) {
                 const int n = n0 + r;
                 if (n >= N) break;
-                if (FIRST) ((T *)out)[(size_t)(s0 + i) * ldo + n] = from_f32<T>(expert_act(w[i] * sg[i][r], w[i] * su[i][r], limit, alpha));
+                if (FIRST) ((T *)out)[(size_t)(s0 + i) * ldo + n] = from_f32<T>(first_act<KIND>(w[i] * sg[i][r], w[i] * su[i][r], limit, alpha));
                 else ((float *)out)[(size_t)(s0 + i) * ldo + n] = sg[i][r];
             }
     }
 }
 
-template <typename T, bool FIRST>
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
 moe_rows_grouped_kernel(const T *__restrict__ A, int lda, const T *__restrict__ W, void *__restrict__ out, int ldo,
                         const int *__restrict__ offsets, const int *__restrict__ order, const float *__restrict__ pair_weight, int top,
                         int N, int K, float limit, float alpha) {
+    MOE_KIND_FLAGS;
     extern __shared__ __align__(16) float xs[];      // [MG_SLOTS][K]
     pdl_launch_dependents();
     pdl_wait();
     const int e = blockIdx.y, s_begin = offsets[e], s_end = offsets[e + 1];
     if (s_end <= s_begin) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const T *We = W + (size_t)e * (FIRST ? 2 : 1) * N * K;
-    const int n0 = (blockIdx.x * 8 + warp) * MR_ROWS_OF(FIRST);
+    const T *We = W + (size_t)e * (GATED ? 2 : 1) * N * K;
+    const int n0 = (blockIdx.x * 8 + warp) * MR_ROWS_OF(KIND);
     for (int s0 = s_begin; s0 < s_end; s0 += MG_SLOTS) {
         const int cnt = min(MG_SLOTS, s_end - s0);
         __syncthreads();                             // the rows of the group before are no longer read
@@ -499,10 +530,10 @@ moe_rows_grouped_kernel(const T *__restrict__ A, int lda, const T *__restrict__ 
         for (int i = 0; i < MG_SLOTS; i++) w[i] = (FIRST && pair_weight && i < cnt) ? pair_weight[order[s0 + i]] : 1.0f;
         if (n0 >= N) continue;
         switch (cnt) {
-        case 1: moe_group_rows<T, FIRST, 1>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
-        case 2: moe_group_rows<T, FIRST, 2>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
-        case 3: moe_group_rows<T, FIRST, 3>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
-        default: moe_group_rows<T, FIRST, 4>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
+        case 1: moe_group_rows<T, KIND, 1>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
+        case 2: moe_group_rows<T, KIND, 2>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
+        case 3: moe_group_rows<T, KIND, 3>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
+        default: moe_group_rows<T, KIND, 4>(We, xs, out, ldo, s0, w, N, K, limit, alpha, n0, lane); break;
         }
     }
 }
@@ -512,17 +543,37 @@ static bool moe_grouped_ok(int dtype, int K, const void *W) {
     const int per = dtype == FG_F32 ? 4 : 8;
     return K % per == 0 && (((uintptr_t)W) & 15) == 0 && (size_t)MG_SLOTS * K * sizeof(float) <= 96 * 1024;
 }
-template <typename T, bool FIRST>
+template <typename T, int KIND>
 static int moe_grouped_launch(const void *A, int lda, const void *W, void *out, int ldo, const int *offsets, const int *order,
                               const float *pair_weight, int X, int top, int N, int K, float limit, float alpha, cudaStream_t stream) {
     static FgPerDevice setup;
     if (fg_needs_setup(setup)) {
-        cudaError_t e = cudaFuncSetAttribute(moe_rows_grouped_kernel<T, FIRST>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+        cudaError_t e = cudaFuncSetAttribute(moe_rows_grouped_kernel<T, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
         if (e != cudaSuccess) return (int)e;
     }
-    const int per_block = 8 * MR_ROWS_OF(FIRST);
-    return fg_launch(moe_rows_grouped_kernel<T, FIRST>, dim3((N + per_block - 1) / per_block, X), dim3(256), (size_t)MG_SLOTS * K * sizeof(float),
+    const int per_block = 8 * MR_ROWS_OF(KIND);
+    return fg_launch(moe_rows_grouped_kernel<T, KIND>, dim3((N + per_block - 1) / per_block, X), dim3(256), (size_t)MG_SLOTS * K * sizeof(float),
                      stream, (const T *)A, lda, (const T *)W, out, ldo, offsets, order, pair_weight, top, N, K, limit, alpha);
+}
+
+// One of the three contractions over the pairs of a step.  A: the rows (first contractions) or the slots; W: the experts' matrices,
+// [X][1 or 2][N][K]; out [M * top, ldo] in T (first) or float32 (second).
+template <typename T, int KIND>
+static int moe_contract(const void *A, int lda, const void *W, void *out, int ldo, int dtype, const int *pair_expert, const int *offsets,
+                        const int *order, const float *pair_weight, int M, int X, int top, int N, int K, float limit, float alpha,
+                        cudaStream_t stream) {
+    const int P = M * top;
+    if (P <= 64 && moe_grouped_ok(dtype, K, W) && moe_grouped_enabled())
+        return moe_grouped_launch<T, KIND>(A, lda, W, out, ldo, offsets, order, pair_weight, X, top, N, K, limit, alpha, stream);
+    if (P <= 64 && (size_t)K * 4 <= 48 * 1024) {
+        dim3 grid((N + 8 * MR_ROWS_OF(KIND) - 1) / (8 * MR_ROWS_OF(KIND)), P);
+        return fg_launch(moe_rows_kernel<T, KIND>, grid, dim3(256), (size_t)K * 4, stream, (const T *)A, lda, (const T *)W, out, ldo, pair_expert,
+                         order, pair_weight, top, X, N, K, limit, alpha);
+    }
+    dim3 grid((N + MT - 1) / MT, (P + MT - 1) / MT + X);
+    if (grid.y > 65535) return FG_ERR_BAD_SIZE;
+    return fg_launch(moe_tile_kernel<T, KIND>, grid, dim3(256), 0, stream, (const T *)A, lda, (const T *)W, out, ldo, offsets, order, pair_weight, X,
+                     top, N, K, limit, alpha);
 }
 
 // y: [M * top, F] in T.  x: [M, E].  w_in: [X, 2F, E].
@@ -530,54 +581,33 @@ extern "C" int fg_moe_first(const void *x, int ldx, const void *w_in, void *y, i
                             const int *offsets, const int *order, const float *pair_weight, int M, int X, int top, int F, int E,
                             float limit, float alpha, cudaStream_t stream) {
     if (M <= 0) return 0;
-    const int P = M * top;
-    if (dtype != FG_F32 && dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
-    if (P <= 64 && moe_grouped_ok(dtype, E, w_in) && moe_grouped_enabled()) {
-        if (dtype == FG_F32) return moe_grouped_launch<float, true>(x, ldx, w_in, y, ldy, offsets, order, pair_weight, X, top, F, E, limit, alpha, stream);
-        return moe_grouped_launch<bf16, true>(x, ldx, w_in, y, ldy, offsets, order, pair_weight, X, top, F, E, limit, alpha, stream);
-    }
-    if (P <= 64 && (size_t)E * 4 <= 48 * 1024) {
-        dim3 grid((F + 8 * MR_ROWS_OF(true) - 1) / (8 * MR_ROWS_OF(true)), P);
-        if (dtype == FG_F32)
-            return fg_launch(moe_rows_kernel<float, true>, grid, dim3(256), (size_t)E * 4, stream, (const float *)x, ldx, (const float *)w_in,
-                             y, ldy, pair_expert, order, pair_weight, top, X, F, E, limit, alpha);
-        return fg_launch(moe_rows_kernel<bf16, true>, grid, dim3(256), (size_t)E * 4, stream, (const bf16 *)x, ldx, (const bf16 *)w_in, y, ldy,
-                         pair_expert, order, pair_weight, top, X, F, E, limit, alpha);
-    }
-    dim3 grid((F + MT - 1) / MT, (P + MT - 1) / MT + X);
-    if (grid.y > 65535) return FG_ERR_BAD_SIZE;
     if (dtype == FG_F32)
-        return fg_launch(moe_tile_kernel<float, true>, grid, dim3(256), 0, stream, (const float *)x, ldx, (const float *)w_in, y, ldy, offsets,
-                         order, pair_weight, X, top, F, E, limit, alpha);
-    return fg_launch(moe_tile_kernel<bf16, true>, grid, dim3(256), 0, stream, (const bf16 *)x, ldx, (const bf16 *)w_in, y, ldy, offsets, order,
-                     pair_weight, X, top, F, E, limit, alpha);
+        return moe_contract<float, MOE_FIRST_GATED>(x, ldx, w_in, y, ldy, dtype, pair_expert, offsets, order, pair_weight, M, X, top, F, E, limit, alpha, stream);
+    if (dtype == FG_BF16)
+        return moe_contract<bf16, MOE_FIRST_GATED>(x, ldx, w_in, y, ldy, dtype, pair_expert, offsets, order, pair_weight, M, X, top, F, E, limit, alpha, stream);
+    return FG_ERR_BAD_DTYPE;
+}
+
+// The same for experts with one input matrix: y = max(w_in[e] x, 0)^2.  w_in: [X, F, E].
+extern "C" int fg_moe_first_relu2(const void *x, int ldx, const void *w_in, void *y, int ldy, int dtype, const int *pair_expert,
+                                  const int *offsets, const int *order, int M, int X, int top, int F, int E, cudaStream_t stream) {
+    if (M <= 0) return 0;
+    if (dtype == FG_F32)
+        return moe_contract<float, MOE_FIRST_RELU2>(x, ldx, w_in, y, ldy, dtype, pair_expert, offsets, order, nullptr, M, X, top, F, E, 0.f, 0.f, stream);
+    if (dtype == FG_BF16)
+        return moe_contract<bf16, MOE_FIRST_RELU2>(x, ldx, w_in, y, ldy, dtype, pair_expert, offsets, order, nullptr, M, X, top, F, E, 0.f, 0.f, stream);
+    return FG_ERR_BAD_DTYPE;
 }
 
 // out: [M * top, E] float32.  y: [M * top, F].  w_out: [X, E, F].
 extern "C" int fg_moe_second(const void *y, int ldy, const void *w_out, float *out, int ldo, int dtype, const int *pair_expert,
                              const int *offsets, const int *order, int M, int X, int top, int F, int E, cudaStream_t stream) {
     if (M <= 0) return 0;
-    const int P = M * top;
-    if (dtype != FG_F32 && dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
-    if (P <= 64 && moe_grouped_ok(dtype, F, w_out) && moe_grouped_enabled()) {
-        if (dtype == FG_F32) return moe_grouped_launch<float, false>(y, ldy, w_out, out, ldo, offsets, order, nullptr, X, top, E, F, 0.f, 0.f, stream);
-        return moe_grouped_launch<bf16, false>(y, ldy, w_out, out, ldo, offsets, order, nullptr, X, top, E, F, 0.f, 0.f, stream);
-    }
-    if (P <= 64 && (size_t)F * 4 <= 48 * 1024) {
-        dim3 grid((E + 8 * MR_ROWS_OF(false) - 1) / (8 * MR_ROWS_OF(false)), P);
-        if (dtype == FG_F32)
-            return fg_launch(moe_rows_kernel<float, false>, grid, dim3(256), (size_t)F * 4, stream, (const float *)y, ldy, (const float *)w_out,
-                             (void *)out, ldo, pair_expert, order, (const float *)nullptr, top, X, E, F, 0.f, 0.f);
-        return fg_launch(moe_rows_kernel<bf16, false>, grid, dim3(256), (size_t)F * 4, stream, (const bf16 *)y, ldy, (const bf16 *)w_out,
-                         (void *)out, ldo, pair_expert, order, (const float *)nullptr, top, X, E, F, 0.f, 0.f);
-    }
-    dim3 grid((E + MT - 1) / MT, (P + MT - 1) / MT + X);
-    if (grid.y > 65535) return FG_ERR_BAD_SIZE;
     if (dtype == FG_F32)
-        return fg_launch(moe_tile_kernel<float, false>, grid, dim3(256), 0, stream, (const float *)y, ldy, (const float *)w_out, (void *)out,
-                         ldo, offsets, order, (const float *)nullptr, X, top, E, F, 0.f, 0.f);
-    return fg_launch(moe_tile_kernel<bf16, false>, grid, dim3(256), 0, stream, (const bf16 *)y, ldy, (const bf16 *)w_out, (void *)out, ldo,
-                     offsets, order, (const float *)nullptr, X, top, E, F, 0.f, 0.f);
+        return moe_contract<float, MOE_SECOND>(y, ldy, w_out, out, ldo, dtype, pair_expert, offsets, order, nullptr, M, X, top, E, F, 0.f, 0.f, stream);
+    if (dtype == FG_BF16)
+        return moe_contract<bf16, MOE_SECOND>(y, ldy, w_out, out, ldo, dtype, pair_expert, offsets, order, nullptr, M, X, top, E, F, 0.f, 0.f, stream);
+    return FG_ERR_BAD_DTYPE;
 }
 
 // ------------------------------------------------------------------ long portions: the experts' contractions as plain ones

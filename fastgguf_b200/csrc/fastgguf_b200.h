@@ -43,6 +43,7 @@ int fg_softcap(float *logits, int R, int V, int ld, float cap, cudaStream_t stre
 int fg_concat2(const float *a, int lda, const float *b, int ldb, void *out, int out_dtype, int ldo, int M, int E,
                cudaStream_t stream);
 int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream);
+int fg_gelu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream);      /* the tanh form of gelu instead */
 /* out (+)= scale_a * f_a(a) + scale_b * f_b(b) over float32 rows [M, E]; f(t) = t / rms(t) * w with a weight, t itself without */
 int fg_pair_combine(const float *a, const float *b, const float *w_a, const float *w_b, float scale_a, float scale_b, float eps,
                     float *out, int M, int E, int accumulate, cudaStream_t stream);
@@ -100,6 +101,20 @@ int fg_gla_chunked_ok(int dk, int dv);
 int fg_gla_chunked(const float *proj, int ld, const float *z, int ldz, const float *z_bias, const float *norm_w, void *out,
                    int out_dtype, int ldo, const int *cu_rows, const int *slots, float *state, int *plan, float *U, float *D,
                    int n_seq, int n_chunks, int H, int dk, int dv, float tau, float q_scale, float eps, cudaStream_t stream);
+/* the real-gated linear recurrent unit (rglru.cu): a step of single tokens in one launch; portions as convolution, gates (a
+   contraction between the two), recurrence.  A state row holds fg_rglru_state_floats(C, taps) floats */
+long long fg_rglru_state_floats(int C, int taps);
+int fg_rglru_tiles(int M, int C, int part, int bn);
+int fg_rglru_conv(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps, const float *state,
+                  long long state_stride, const int *positions, const int *row_seq, const int *cu_rows, const int *slots, float *u, int ldu,
+                  void *pieces, void *tiles, int bn, int M, int C, int part, cudaStream_t stream);
+int fg_rglru_scan(const float *z, long long z_row, long long z_part, const float *gate_bias, const float *u, int ldu, const float *lam, float gain,
+                  const float *proj, int ldp, const float *proj_bias, void *out, int out_dtype, int ldo, const int *cu_rows, const int *slots,
+                  const int *positions, float *state, long long state_stride, int n_seq, int max_new, int C, int part, int taps, cudaStream_t stream);
+int fg_rglru_step_ok(int part);
+int fg_rglru_step(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps, const void *W, int w_dtype,
+                  const float *gate_bias, const float *lam, float gain, const int *positions, const int *row_seq, const int *slots, float *state,
+                  long long state_stride, void *out, int out_dtype, int ldo, int M, int C, int part, cudaStream_t stream);
 /* recurrences with one decay a head and token (recurrence.cu): S <- a S; u = b (v - [delta] S^T k); S <- S + k u^T;
    o = S^T q + skip v.  q, k [M, Hq, d], v [M, H, dv], decay and step [M, H], out [M, H * dv], all float32; a sequence's state
    row (state_stride floats apart) holds fg_decay_recurrence_state_floats(H, d, dv) floats in the kernel's own layout */
@@ -180,6 +195,12 @@ int fg_moe_act(const float *gu, const int *order, const float *pair_weight, void
                float alpha, cudaStream_t stream);
 int fg_moe_route(const float *logits, int M, int X, int top, int *pair_expert, float *pair_weight, int *offsets, int *order,
                  int *slot_of, cudaStream_t stream);
+/* bias (or null) is added to the logits; chosen_softmax: weights are the softmax over the chosen logits alone */
+int fg_moe_route_ext(const float *logits, const float *bias, int chosen_softmax, int M, int X, int top, int *pair_expert, float *pair_weight,
+                     int *offsets, int *order, int *slot_of, cudaStream_t stream);
+/* experts with one input matrix, w_in [X, F, E]: y = max(w_in[e] x, 0)^2 */
+int fg_moe_first_relu2(const void *x, int ldx, const void *w_in, void *y, int ldy, int dtype, const int *pair_expert, const int *offsets,
+                       const int *order, int M, int X, int top, int F, int E, cudaStream_t stream);
 /* softmax scores, choice on score + bias among the `keep` best of n_groups groups, weights = chosen scores / their sum * scale */
 int fg_moe_route_grouped(const float *logits, const float *bias, int M, int X, int top, int n_groups, int keep, float scale,
                          int *pair_expert, float *pair_weight, int *offsets, int *order, int *slot_of, cudaStream_t stream);
@@ -197,7 +218,8 @@ int fg_moe_combine_weighted(const float *slot_out, int ld, const int *slot_of, c
                             cudaStream_t stream);
 
 /* ---- libfg_tc: bf16 contraction on tcgen05 / TMA / tensor memory
- * epi: 0 bf16 out, 1 f32 out, 2 f32 out += (residual add), 3 silu(gate) * up on interleaved rows, 4 bf16 out of max(x, 0)^2 */
+ * epi: 0 bf16 out, 1 f32 out, 2 f32 out += (residual add), 3 silu(gate) * up on interleaved rows, 4 bf16 out of max(x, 0)^2,
+ * 5 gelu_tanh(gate) * up on interleaved rows */
 int fg_gemm_tc(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int epi, int M, int N, int K,
                int force_splits, const float *ss_in, int ss_tiles, int ss_size, float ss_eps, const float *norm_w,
                void *xw_out, float *ss_out, int *ss_tiles_out /* host */, cudaStream_t stream);
@@ -213,6 +235,8 @@ int fg_gemm_tc_max_ss_tiles(int N);
 int fg_gemm_tc_grouped_bn(int N);
 int fg_gemm_tc_grouped(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, float *out, int ldc, int N, int K,
                        const void *tiles, int n_tiles, cudaStream_t stream);
+int fg_gemm_tc_grouped_ext(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, void *out, int ldc, int epi /* 1 or 4 */, int N,
+                           int K, const void *tiles, int n_tiles, cudaStream_t stream);
 int fg_gemm_tc_error(void);
 /* tests only: shorten the bounded waits and make the decode kernel's pipeline stall, see gemm_tc.cu */
 int fg_gemm_tc_test_hook(long long wait_limit_cycles, int skip_copy);

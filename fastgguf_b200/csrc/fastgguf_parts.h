@@ -15,6 +15,7 @@
  *                                                               "mixer_post_norm", "feed_forward_post_norm": PART;
  *                                                               block "parallel" has no feed_forward_norm, or one
  *                                                               (then each sublayer reads a norm of its own);
+ *                                                               block "postnorm" has neither, only post norms;
  *                                                               optional "token_input": PART, role token_input:
  *                                                               x <- x + f(x, the rows' tokens) behind the sublayers
  *    "schedule": [{"layer": 0, "cache_from": null}, ...],      the order in which layers run: an entry may
@@ -29,7 +30,7 @@
  *   of an attention mixer); nested parts with equal kind and parameters are built once and shared.
  *
  * Built-in kinds
- *   norm          "rmsnorm"        {size, eps, offset: 0.0}     y = x / rms(x) * (offset + w)
+ *   norm          "rmsnorm"        {size, eps, offset: 0.0, gain: 1.0}     y = x / rms(x) * gain * (offset + w)
  *   position      "rope"           {head_dim, theta, scaling: null | {rope_type: "llama3", ...} | {rope_type: "yarn", factor,
  *                                   original_max_position_embeddings, beta_fast, beta_slow},
  *                                   rotary_dim: head_dim, layout: "halves" | "adjacent"}
@@ -69,11 +70,17 @@
  *                                   q_scale: null = 1/sqrt(head_dim)}   convolved q, k, v, unit q and k, S <- g S; u = beta (v -
  *                                   S^T k); S <- S + k u^T; o = S^T q, a norm per head and a SiLU gate; tensors q/k/v/b/a/g/
  *                                   o_proj.weight, q/k/v_conv.weight, A_log, dt_bias, norm.weight
+ *                 "rglru"          {hidden_size, width, n_blocks: 1, conv_taps: 1, gain: 8.0}   a recurrent block around the real-gated
+ *                                   linear recurrent unit: y = gelu_tanh(W_y h + b), u = convolution(W_x h + b) + b, r and i sigmoids
+ *                                   of block-diagonal maps of u, log a = -gain r softplus(lam), S = a S + sqrt(1 - a^2) i u, output
+ *                                   W_o (S y); state (a ring of convolution inputs, and S) float32 per sequence; tensors y/x/
+ *                                   o_proj.weight, y/x_proj.bias, conv.weight, conv.bias, r/i_gate.weight [n_blocks, s, s],
+ *                                   r/i_gate.bias [n_blocks, s], lam
  *                 "mixer_pair"     {hidden_size, left: {kind, params}, right: {kind, params}, left_scale: 1, right_scale: 1,
  *                                   normalize: false, eps}   two mixers on the same rows, y = left_scale f(left) + right_scale
  *                                   f(right), f an RMS norm over the width with a weight where normalize is true; tensors
  *                                   left.<the left mixer's>, right.<the right mixer's>, left_norm.weight, right_norm.weight
- *   feed_forward  "swiglu"         {hidden_size, d_ff}
+ *   feed_forward  "swiglu"         {hidden_size, d_ff, activation: "silu" | "gelu_tanh"}   down(act(gate x) * (up x))
  *                 "mlp"            {hidden_size, d_ff, activation: "relu2"}   down(act(up x))
  *                 "moe"            {hidden_size, d_ff, n_experts, top_k, limit, alpha: 1.702, router: "sigmoid_input"}
  *                                   tensors router.weight, experts.<e>.gate/up/down_proj.weight
@@ -84,8 +91,12 @@
  *                                   outputs; the last n_identity outputs return the input; experts silu(gate) * up; a shared
  *                                   expert on every row; tensors router.weight, router.bias, experts.<e>.*, shared.gate/up/
  *                                   down_proj.weight
+ *                                  {hidden_size, d_ff, n_experts, top_k, router: "softmax_chosen", activation: "gated" | "relu2"}   the
+ *                                   largest logits + router.bias; weights = softmax over the chosen ones, on the experts' outputs;
+ *                                   relu2: experts down(max(up x, 0)^2) without gate_proj; tensors router.weight, router.bias, experts.<e>.*
  *   block         "prenorm"        x += mixer(norm1(x)); x += feed_forward(norm2(x))
  *                 "sandwich"       x += post1(mixer(norm1(x))); x += post2(feed_forward(norm2(x)))
+ *                 "postnorm"       x += post1(mixer(x)); x += post2(feed_forward(x)): the sublayers read the stream itself
  *                 "parallel"       x += mixer(norm1(x)) + feed_forward(norm1(x)), or, with a feed_forward_norm,
  *                                  x += mixer(norm1(x)) + feed_forward(norm2(x)), both norms of the same x
  *   token_input   "gated_token_embedding"  {hidden_size, vocab_size, dim, table_dim, column, eps}   e = table[token, column ..

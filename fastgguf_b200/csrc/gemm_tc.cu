@@ -22,7 +22,7 @@
 //               kernel (weights are never written), so weight traffic overlaps that kernel's tail.
 //   warp 1      MMA issuer (the same way): tcgen05.mma 128 x BN x 16; its commit frees the stage.
 //   warps 2-5   epilogue: tcgen05.ld of the f32 tile, then one of
-//               store bf16 | store f32 | add into f32 (residual) | silu(gate) * up -> bf16
+//               store bf16 | store f32 | add into f32 (residual) | silu(gate) * up -> bf16 (or gelu(gate) * up)
 //               (the decode kernel has eight epilogue warps, 2-9: two per lane group of tensor memory)
 //
 // The silu epilogue expects the gate and up matrices interleaved in blocks of 64 rows
@@ -47,7 +47,8 @@
 #define WAIT_LIMIT_CYCLES 2000000000ll
 #define WAIT_SHORT_CYCLES 1000000ll
 
-enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_RELU2_BF16 = 4 /* launcher only: EPI_BF16 + act */ };
+enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_RELU2_BF16 = 4 /* launcher only: EPI_BF16 + act */,
+       EPI_GELU_MUL = 5 /* launcher only: EPI_SILU_MUL + act */ };
 
 __device__ int g_gemm_error = 0;      // 0, or (code << 8 | role) of the first wait that ran out
 // How long a wait may last, in SM cycles (about a second).  A variable, so that a test can make a wait run out within a
@@ -180,7 +181,11 @@ __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.w
 
 // silu(g) * u in f32 with the fast exponential and division (2 ulp each): the result is rounded to bfloat16
 // (8 bits of mantissa) right after, and the precise forms made the epilogue of a 64-token tile several us long
-__device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
+// gelu: g * u with the tanh form of gelu instead; 0.5 (1 + tanh(y)) = sigmoid(2 y), so it is the same form on another argument
+__device__ __forceinline__ float gated_mul(float g, float u, int gelu) {
+    const float z = gelu ? g * fmaf(0.07135481627f, g * g, 1.5957691216f) : g;       // 2 sqrt(2 / pi) (g + 0.044715 g^3)
+    return __fdividef(g, 1.0f + __expf(-z)) * u;
+}
 
 static int g_test_skip_copy = 0;      // host side of fg_gemm_tc_test_hook
 
@@ -203,7 +208,7 @@ struct GemmArgs {
     int epi, stages;      // decode kernel: epilogue and ring depth are run-time values
     int test_skip_copy;   // tests only: the decode kernel's producer omits the activation copy of its first stage
     int splits;           // prefill kernel: > 1 = partial products of `kb_per_split` K-blocks each into out[split][M][ldc]
-    int act;              // bf16 epilogue only: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward)
+    int act;              // bf16 epilogue: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward); gated epilogue: 1 = gelu, not SiLU
     // prefill kernel, grouped contraction (rows in runs, each run with a weight matrix of its own out of a stack): tile t
     // is tiles[t] = {first row, end of its run, first row of the run's matrix in W, tile index along N}; null: one matrix
     const int4 *tiles;
@@ -240,8 +245,8 @@ __device__ __forceinline__ void epilogue_token_major(const GemmArgs &a, uint32_t
                     uint32_t w[8];
 #pragma unroll
                     for (int j = 0; j < 8; j++) {
-                        __nv_bfloat162 t = __floats2bfloat162_rn(silu_mul(g[2 * j] * iv, u[2 * j] * iv),
-                                                                 silu_mul(g[2 * j + 1] * iv, u[2 * j + 1] * iv));
+                        __nv_bfloat162 t = __floats2bfloat162_rn(gated_mul(g[2 * j] * iv, u[2 * j] * iv, a.act),
+                                                                 gated_mul(g[2 * j + 1] * iv, u[2 * j + 1] * iv, a.act));
                         w[j] = *(uint32_t *)&t;
                     }
                     ((uint4 *)dst)[0] = make_uint4(w[0], w[1], w[2], w[3]);
@@ -249,7 +254,7 @@ __device__ __forceinline__ void epilogue_token_major(const GemmArgs &a, uint32_t
                 } else {
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (f0 + j < F) dst[j] = __float2bfloat16_rn(silu_mul(g[j] * iv, u[j] * iv));
+                        if (f0 + j < F) dst[j] = __float2bfloat16_rn(gated_mul(g[j] * iv, u[j] * iv, a.act));
                 }
             }
         }
@@ -648,7 +653,7 @@ gemm_tc_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
                 for (int c = et >> 6; c < ncol; c += EW / 2) {      // 64 threads a token
                     const float iv = inv_s[c];
                     ((bf16 *)a.out)[(size_t)(q0 + c) * a.ldc + f] =
-                        __float2bfloat16_rn(silu_mul(exg[c * 64 + fl] * iv, exu[c * 64 + fl] * iv));
+                        __float2bfloat16_rn(gated_mul(exg[c * 64 + fl] * iv, exu[c * 64 + fl] * iv, a.act));
                 }
             }
         } else {
@@ -726,7 +731,7 @@ gemm_tc_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
                     for (int i = 0; i < 2; i++) {
                         const int f = (p0 >> 1) + lane + 32 * i;
                         if (f < (a.N >> 1))
-                            ((bf16 *)a.out)[(size_t)m * a.ldc + f] = __float2bfloat16_rn(silu_mul(v[i] * iv, v[i + 2] * iv));
+                            ((bf16 *)a.out)[(size_t)m * a.ldc + f] = __float2bfloat16_rn(gated_mul(v[i] * iv, v[i + 2] * iv, a.act));
                     }
                     continue;
                 }
@@ -1286,7 +1291,7 @@ extern "C" int fg_gemm_tc_max_ss_tiles(int N) {
 // sums of squares of row m over ss_size elements, and 1/sqrt(sum / ss_size + ss_eps) scales row m's results.
 // norm_w (optional, residual-add epilogue): also write xw_out[M, N] = bf16(out * norm_w) and the partial
 // sums of squares ss_out[tile, M]; *ss_tiles_out receives the number of tiles.
-// EPI_SILU_MUL: W is [N = 2F, K] with gate and up interleaved in blocks of 64 rows; out is [M, F] bf16.
+// EPI_SILU_MUL, EPI_GELU_MUL: W is [N = 2F, K] with gate and up interleaved in blocks of 64 rows; out is [M, F] bf16.
 // Returns FG_ERR_BAD_SIZE for shapes TMA cannot describe (K % 8, unaligned bases): the caller
 // then uses the plain kernel.
 // streaming multiprocessors of the current device (148 on a B200)
@@ -1305,7 +1310,7 @@ static int sm_count() {
 static int prefill_splits(int M, int N, int K, int epi, int *kb_per_split) {
     static int off = -1;                           // FASTGGUF_SPLITK=0: never (the prefill kernels as they were without it)
     if (off < 0) { const char *e = getenv("FASTGGUF_SPLITK"); off = (e && e[0] == '0') ? 1 : 0; }
-    if (off || M <= 128 || epi == EPI_SILU_MUL) return 0;
+    if (off || M <= 128 || epi == EPI_SILU_MUL || epi == EPI_GELU_MUL) return 0;
     const int total_kb = (K + BK - 1) / BK, sms = sm_count();
     const long long tiles = (long long)((M + BM - 1) / BM) * ((N + 127) / 128);
     if (tiles * 2 > sms || total_kb < 16) return 0;
@@ -1350,8 +1355,9 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return FG_ERR_BAD_SIZE;
     // epilogue code 4: bfloat16 output of max(x, 0)^2 - the bf16 epilogue with its activation flag set
-    const int act = epi == EPI_RELU2_BF16 ? 1 : 0;
-    if (act) epi = EPI_BF16;
+    // epilogue code 5: the gated epilogue with the tanh form of gelu on the gate
+    const int act = (epi == EPI_RELU2_BF16 || epi == EPI_GELU_MUL) ? 1 : 0;
+    if (act) epi = epi == EPI_GELU_MUL ? EPI_SILU_MUL : EPI_BF16;
     if (epi == EPI_SILU_MUL && N % 128) return FG_ERR_BAD_SIZE;
     // Up to 128 rows the weights stream through the decode kernel, in blocks of 64 tokens whose CTAs run side by side
     // and share each weight tile through L2; beyond that the prefill kernel is faster (measured: 56.6 against 45.5 k tok/s
@@ -1449,11 +1455,13 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
 // of the run's output, float32 out[rows, ldc].  One launch over all runs on the persistent prefill kernel: a tile of the
 // table is a tile of the kernel, the rest (ring, accumulators in tensor memory, epilogue under the next tile's MMAs) is
 // the plain contraction's.  fg_gemm_tc_grouped_bn(N) is the tile width the table must be built for; a tile's rows past
-// its run's end are computed and not stored.
+// its run's end are computed and not stored.  fg_gemm_tc_grouped_ext: the epilogue is a parameter, EPI_F32 or EPI_RELU2_BF16
+// (bfloat16 output of max(x, 0)^2).
 extern "C" int fg_gemm_tc_grouped_bn(int N) { return N % 256 == 0 ? 256 : 128; }
 
-extern "C" int fg_gemm_tc_grouped(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, float *out, int ldc,
-                                  int N, int K, const void *tiles, int n_tiles, cudaStream_t stream) {
+extern "C" int fg_gemm_tc_grouped_ext(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, void *out, int ldc, int epi,
+                                      int N, int K, const void *tiles, int n_tiles, cudaStream_t stream) {
+    if (epi != EPI_F32 && epi != EPI_RELU2_BF16) return FG_ERR_BAD_DTYPE;
     if (rows <= 0 || n_tiles <= 0) return 0;
     if (N <= 0 || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || ((uintptr_t)tiles & 15))
         return FG_ERR_BAD_SIZE;
@@ -1463,11 +1471,18 @@ extern "C" int fg_gemm_tc_grouped(const void *X, int ldx, int rows, const void *
     if (e) return e;
     e = make_map(&tmQ, W, stack_rows, K, ldw, bn);
     if (e) return e;
-    const int vec_ok = ((uintptr_t)out % 16 == 0) && ((size_t)ldc * 4 % 16 == 0);
-    GemmArgs a{out, rows, N, K, ldc, 0, vec_ok, nullptr, 0, 1, 0.f, nullptr, nullptr, nullptr, EPI_F32, 0, g_test_skip_copy, 0, 0,
+    const int vec_ok = ((uintptr_t)out % 16 == 0) && ((size_t)ldc * (epi == EPI_F32 ? 4 : 2) % 16 == 0);
+    GemmArgs a{out, rows, N, K, ldc, 0, vec_ok, nullptr, 0, 1, 0.f, nullptr, nullptr, nullptr, EPI_F32, 0, g_test_skip_copy, 0, epi == EPI_RELU2_BF16 ? 1 : 0,
                (const int4 *)tiles};
+    if (epi == EPI_RELU2_BF16)
+        return bn == 256 ? launch_prefill<256, 4, EPI_BF16>(tmP, tmQ, a, stream, n_tiles) : launch_prefill<128, 6, EPI_BF16>(tmP, tmQ, a, stream, n_tiles);
     if (bn == 256) return launch_prefill<256, 4, EPI_F32>(tmP, tmQ, a, stream, n_tiles);
     return launch_prefill<128, 6, EPI_F32>(tmP, tmQ, a, stream, n_tiles);
+}
+
+extern "C" int fg_gemm_tc_grouped(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, float *out, int ldc,
+                                  int N, int K, const void *tiles, int n_tiles, cudaStream_t stream) {
+    return fg_gemm_tc_grouped_ext(X, ldx, rows, W, ldw, stack_rows, out, ldc, EPI_F32, N, K, tiles, n_tiles, stream);
 }
 
 // For the test of the bounded waits: wait_limit_cycles > 0 sets how long a wait may last (0 restores the default of

@@ -922,7 +922,7 @@ static std::map<std::string, ExpectedTensor> declared_tensors(const ModelSpec &s
     build(FG_ROLE_EMBEDDING, spec.embedding);
     for (auto &l : spec.layers) {
         build(FG_ROLE_MIXER, l.mixer);
-        build(FG_ROLE_NORM, l.mixer_norm);
+        if (!l.mixer_norm.kind.empty()) build(FG_ROLE_NORM, l.mixer_norm);
         if (l.has_feed_forward()) {
             build(FG_ROLE_FEED_FORWARD, l.feed_forward);
             if (!l.feed_forward_norm.kind.empty()) build(FG_ROLE_NORM, l.feed_forward_norm);

@@ -41,7 +41,8 @@ ModelSpec ModelSpec::from_json(const Json &j) {
         if (!l.is_object() || !l.get("block").is_string()) fail(FG_E_CONFIG, "model spec: a layer needs a 'block' kind");
         ls.block = l.get("block").as_string();
         ls.mixer = part_spec_from_json(l.get("mixer"), "mixer");
-        ls.mixer_norm = part_spec_from_json(l.get("mixer_norm"), "mixer_norm");
+        // a block whose sublayers read the stream itself (block "postnorm") has no norms in front of them
+        if (!l.get("mixer_norm").is_null()) ls.mixer_norm = part_spec_from_json(l.get("mixer_norm"), "mixer_norm");
         if (!l.get("feed_forward").is_null()) {                       // null or absent: a layer of a mixer alone
             ls.feed_forward = part_spec_from_json(l.get("feed_forward"), "feed_forward");
             // a block whose sublayers share one norm (block "parallel") gives none for the feed-forward
@@ -102,7 +103,11 @@ DecoderModel::DecoderModel(const ModelSpec &spec_, int dtype, int device, cudaSt
     embedding_ = dynamic_cast<Embedding *>(build(FG_ROLE_EMBEDDING, spec.embedding));
     for (auto &layer : spec.layers) {
         Mixer *mixer = dynamic_cast<Mixer *>(build(FG_ROLE_MIXER, layer.mixer));
-        Norm *n1 = dynamic_cast<Norm *>(build(FG_ROLE_NORM, layer.mixer_norm));
+        Norm *n1 = nullptr;
+        if (!layer.mixer_norm.kind.empty()) {
+            n1 = dynamic_cast<Norm *>(build(FG_ROLE_NORM, layer.mixer_norm));
+            if (!n1) fail(FG_E_INTERNAL, "a part was registered under the wrong role");
+        }
         FeedForward *ffn = nullptr;
         Norm *n2 = nullptr, *p1 = nullptr, *p2 = nullptr;
         if (layer.has_feed_forward()) {
@@ -115,7 +120,7 @@ DecoderModel::DecoderModel(const ModelSpec &spec_, int dtype, int device, cudaSt
         }
         if (!layer.mixer_post_norm.kind.empty()) p1 = dynamic_cast<Norm *>(build(FG_ROLE_NORM, layer.mixer_post_norm));
         if (!layer.feed_forward_post_norm.kind.empty()) p2 = dynamic_cast<Norm *>(build(FG_ROLE_NORM, layer.feed_forward_post_norm));
-        if (!mixer || !n1) fail(FG_E_INTERNAL, "a part was registered under the wrong role");
+        if (!mixer) fail(FG_E_INTERNAL, "a part was registered under the wrong role");
         std::unique_ptr<Block> b = build_block(layer.block, runtime);
         b->mixer = mixer; b->feed_forward = ffn; b->mixer_norm = n1; b->feed_forward_norm = n2;
         b->mixer_post_norm = p1; b->feed_forward_post_norm = p2;
@@ -471,7 +476,7 @@ Tensor DecoderModel::forward(Runtime &rt, const Batch &batch) {
     auto block_at = [&](size_t i) { return blocks_[(size_t)spec.schedule[i].layer].get(); };
     // the norm a block starts with, if whoever writes the residual stream may start it
     auto entry_norm = [&](Block *b) -> Norm * {
-        return (bf16 && b->mixer->supports_deferred_norm() && b->mixer_norm->deferrable()) ? b->mixer_norm : nullptr;
+        return (bf16 && b->mixer_norm && b->mixer->supports_deferred_norm() && b->mixer_norm->deferrable()) ? b->mixer_norm : nullptr;
     };
     // the final norm can be started by the last block when the head takes every row as it is
     Norm *head_norm = (batch.want_all && bf16 && final_norm_->deferrable() && head_->supports_deferred_norm()) ? final_norm_ : nullptr;
@@ -496,7 +501,8 @@ Tensor DecoderModel::forward(Runtime &rt, const Batch &batch) {
         }
         Norm *next = i + 1 < n ? (reenters(i + 1) ? nullptr : entry_norm(block_at(i + 1))) : head_norm;
         // blocks that finish the next norm themselves hand it to a block of the same habit only (any dtype)
-        if (block_at(i)->finished_norms()) next = (i + 1 < n && block_at(i + 1)->finished_norms()) ? block_at(i + 1)->mixer_norm : nullptr;
+        // (the last such block finishes the final norm where the head takes every row)
+        if (block_at(i)->finished_norms()) next = i + 1 == n ? head_norm : block_at(i + 1)->finished_norms() ? block_at(i + 1)->mixer_norm : nullptr;
         else if (i + 1 < n && block_at(i + 1)->finished_norms()) next = nullptr;
         // a layer that adds a token input behind its sublayers changes the stream after its last projection
         if (reenters(i + 1) || block_at(i)->token_input) next = nullptr;
@@ -506,6 +512,8 @@ Tensor DecoderModel::forward(Runtime &rt, const Batch &batch) {
             block_at(i)->token_input->forward(rt, batch, x);
             pending = DeferredNorm();
         }
+        // the rounded stream itself is for a block that reads it so
+        if (pending.defined() && !pending.weight && !(i + 1 < n && block_at(i + 1)->reads_stream())) pending = DeferredNorm();
         rt.arena->end_layers();                        // what follows the block belongs to the step, not to the layer
     }
     rt.arena->end_layers();

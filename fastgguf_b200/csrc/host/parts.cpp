@@ -1,4 +1,4 @@
-// See parts.hpp.  Built-in kinds: rmsnorm, rope, gqa_attention, swiglu, prenorm, sandwich, embedding, lm_head (the
+// See parts.hpp.  Built-in kinds: rmsnorm, rope, gqa_attention, swiglu, prenorm, sandwich, postnorm, embedding, lm_head (the
 // retention mixer lives in parts_recurrent.cpp, the plain and the expert feed-forwards in parts_experts.cpp); and
 // the adapter that runs a part registered from outside through fastgguf_parts.h.
 #include "parts.hpp"
@@ -9,7 +9,7 @@
 
 namespace fg {
 
-static const int EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3;
+static const int EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_GELU_MUL = 5;
 static const int KERNEL_BAD_SIZE = 10002;
 
 const char *role_name(int role) {
@@ -206,7 +206,7 @@ Tensor Linear::forward_relu2(Runtime &rt, const Tensor &a) const {
     return t;
 }
 
-bool Linear::forward_silu(Runtime &rt, const Tensor &a_in, const DeferredNorm *deferred, Tensor *out) const {
+bool Linear::forward_gated(Runtime &rt, const Tensor &a_in, const DeferredNorm *deferred, bool gelu, Tensor *out) const {
     const Tensor &W = w_.t;
     Tensor a = deferred ? deferred->xw : a_in;
     if (!fast_ || rt.plain_kernels || a.dtype != FG_BF16 || W.rows % 128) return false;
@@ -218,12 +218,12 @@ bool Linear::forward_silu(Runtime &rt, const Tensor &a_in, const DeferredNorm *d
     float ss_eps = 0.f;
     if (deferred) { ss_in = deferred->ss; ss_tiles = deferred->tiles; ss_size = deferred->size; ss_eps = deferred->eps; }
     count_launch();
-    ProfileScope scope("fg_gemm_tc", profile_on() ? format("%lld x %lld, %lld rows, silu", (long long)W.rows, (long long)a.cols, (long long)M).c_str() : nullptr);
-    int code = FG_KERNEL("tc", fg_gemm_tc)(a.data, (int)a.ld, W.data, (int)W.ld, t.data, (int)t.ld, EPI_SILU_MUL, (int)M,
+    ProfileScope scope("fg_gemm_tc", profile_on() ? format("%lld x %lld, %lld rows, %s", (long long)W.rows, (long long)a.cols, (long long)M, gelu ? "gelu" : "silu").c_str() : nullptr);
+    int code = FG_KERNEL("tc", fg_gemm_tc)(a.data, (int)a.ld, W.data, (int)W.ld, t.data, (int)t.ld, gelu ? EPI_GELU_MUL : EPI_SILU_MUL, (int)M,
                                            (int)W.rows, (int)a.cols, 0, ss_in, ss_tiles, ss_size, ss_eps, nullptr, nullptr,
                                            nullptr, &tiles_out, rt.stream);
     if (code == KERNEL_BAD_SIZE) return false;
-    check_kernel(code, "fg_gemm_tc (silu)");
+    check_kernel(code, "fg_gemm_tc (gated)");
     *out = t;
     return true;
 }
@@ -328,22 +328,24 @@ Tensor rope_attention(Runtime &rt, const Tensor &qkv, const Batch &b, const Laye
 // ------------------------------------------------------------------------------------ RMSNorm
 // y = x * (1 / sqrt(mean(x^2) + eps)) * w; the weight multiplies directly (no +1), in the order x * inv * w
 // (rmsnorm_w, fastgguf.c:3100-3105).  Statistics are 32-bit here (the reference sums in double).
-// offset: checkpoints that store the weight around zero apply (offset + w); the sum is formed once, in float32, when
-// the weights are loaded, so every kernel (and a norm started inside a contraction) reads a plain weight.
+// offset: checkpoints that store the weight around zero apply (offset + w); gain: the output times a constant (a final norm in
+// front of a head whose logits are scaled).  gain * (offset + w) is formed once, in float32, when the weights are loaded, so
+// every kernel (and a norm started inside a contraction) reads a plain weight.
 class RMSNorm : public Norm {
 public:
     RMSNorm(const Json &p)
         : size_((int)param_int(p, "size", "rmsnorm")), eps_((float)param_float(p, "eps", "rmsnorm")),
-          offset_((float)param_float(p, "offset", 0.0, "rmsnorm")) {
+          offset_((float)param_float(p, "offset", 0.0, "rmsnorm")), gain_((float)param_float(p, "gain", 1.0, "rmsnorm")) {
         if (size_ <= 0 || !(eps_ > 0.f)) fail(FG_E_CONFIG, "rmsnorm: size and eps must be positive");
     }
     std::vector<TensorDecl> tensor_decls() const override { return {{"weight", {size_}, false, offset_ != 0.f ? 0 : 1, offset_ != 0.f ? 0.1f : 0.01f}}; }
     void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
         const Weight &w = tensor_of(tensors, "weight");
         // widening bf16 -> f32 is exact; the kernels read the weight as f32
-        if (w.t.dtype == FG_F32 && offset_ == 0.f) w_ = w;
+        if (w.t.dtype == FG_F32 && offset_ == 0.f && gain_ == 1.f) w_ = w;
         else w_ = concat_rows({w}, FG_F32, rt.stream);
         if (offset_ != 0.f) dev_shift_f32(w_.t.ptr<float>(), w_.t.numel(), offset_, rt.stream);
+        if (gain_ != 1.f) dev_scale_f32(w_.t.ptr<float>(), w_.t.numel(), gain_, rt.stream);
     }
     Tensor forward(Runtime &rt, const Tensor &x, const int *rows, int n_rows) override {
         int R = rows ? n_rows : (int)x.rows;
@@ -359,7 +361,7 @@ public:
 
 private:
     int size_;
-    float eps_, offset_;
+    float eps_, offset_, gain_;
     Weight w_;
 };
 
@@ -636,10 +638,15 @@ private:
 // ------------------------------------------------------------------------------------ SwiGLU
 // down( silu(gate x) * (up x) ): gate and up in one fused pass (fastgguf.c:4870-4872), silu(z) = z / (1 + exp(-z))
 // (:3118) times up (:4876), down projection added onto the layer's input (:4877-4880).
+// activation "gelu_tanh": down(gelu_tanh(gate x) * (up x)) instead.
 class SwiGLU : public FeedForward {
 public:
     SwiGLU(const Json &p) : E_((int)param_int(p, "hidden_size", "swiglu")), F_((int)param_int(p, "d_ff", "swiglu")) {
         if (E_ <= 0 || F_ <= 0) fail(FG_E_CONFIG, "swiglu: sizes must be positive");
+        const Json &a = p.get("activation");
+        const std::string act = a.is_string() ? a.as_string() : "silu";
+        if (act != "silu" && act != "gelu_tanh") fail(FG_E_CONFIG, "swiglu: activation '" + act + "' is not known (known: silu, gelu_tanh)");
+        gelu_ = act == "gelu_tanh";
     }
     std::vector<TensorDecl> tensor_decls() const override {
         return {{"gate_proj.weight", {F_, E_}}, {"up_proj.weight", {F_, E_}}, {"down_proj.weight", {E_, F_}}};
@@ -651,7 +658,7 @@ public:
         int dt = g.t.dtype == u.t.dtype ? g.t.dtype : FG_F32;
         Weight both = concat_rows({g, u}, dt, rt.stream);
         if (dt == FG_BF16 && F_ % 64 == 0 && E_ % 8 == 0 && !rt.plain_kernels) {
-            // gate, up and SiLU-mul in one tensor-core kernel: rows interleaved in blocks of 64
+            // gate, up and their product in one tensor-core kernel: rows interleaved in blocks of 64
             std::vector<int64_t> rows;
             for (int64_t blk = 0; blk < F_ / 64; blk++) {
                 for (int64_t i = 0; i < 64; i++) rows.push_back(blk * 64 + i);
@@ -666,12 +673,13 @@ public:
     DeferredNorm forward(Runtime &rt, const Tensor &xn, const DeferredNorm *deferred, const Batch &, Tensor &residual,
                          Norm *emit_norm) override {
         Tensor t;
-        bool done = fused_.defined() && fused_.forward_silu(rt, xn, deferred, &t);
+        bool done = fused_.defined() && fused_.forward_gated(rt, xn, deferred, gelu_, &t);
         if (!done) {
             if (fused_.defined()) fail(FG_E_KERNEL, "the fused gate/up kernel refused a shape it was planned for");
             Tensor gu = gate_up_.forward(rt, xn, deferred, Tensor(), rt.dtype, false, nullptr, nullptr);
             t = rt.arena->matrix(gu.rows, F_, gu.dtype);
-            if (gu.rows > 0) FG_LAUNCH("core", fg_silu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
+            if (gu.rows > 0 && gelu_) FG_LAUNCH("core", fg_gelu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
+            else if (gu.rows > 0) FG_LAUNCH("core", fg_silu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
         }
         DeferredNorm started;
         down_.forward(rt, t, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
@@ -680,6 +688,7 @@ public:
 
 private:
     int E_, F_;
+    bool gelu_ = false;
     Linear fused_, gate_up_, down_;
 };
 
@@ -785,6 +794,63 @@ public:
         feed_forward->forward(rt, hn, nullptr, batch, t, nullptr);
         rt.overwrite = false;
         return finished(join(feed_forward_post_norm, hand_over), hand_over);
+    }
+};
+
+// ------------------------------------------------------------------------------------ post-norm block
+// x += post1(mixer(x)); x += post2(feed_forward(x)): no norm in front, the sublayers read the stream itself - in bfloat16 its
+// rounding, as every contraction's input is, in float32 the stream.  The norm stands on a sublayer's output only.  ONE kernel
+// normalises that output, adds it to the float32 stream and writes the rounded stream for the next reader (or, where the next
+// reader of the stream is a norm, that norm's output).
+class PostNormBlock : public Block {
+public:
+    void check_layer() const override {
+        if (!mixer || !mixer_post_norm) fail(FG_E_CONFIG, "block 'postnorm' needs a mixer and mixer_post_norm");
+        if (mixer_norm || feed_forward_norm) fail(FG_E_CONFIG, "block 'postnorm' has no norms in front of its sublayers");
+        if ((feed_forward == nullptr) != (feed_forward_post_norm == nullptr)) fail(FG_E_CONFIG, "a layer has a feed-forward and its norm, or neither");
+        for (Norm *n : {mixer_post_norm, feed_forward_post_norm})
+            if (n && !n->deferrable()) fail(FG_E_CONFIG, "block 'postnorm' takes norms of the form x / rms(x) * w");
+    }
+    bool finished_norms() const override { return true; }
+    bool reads_stream() const override { return true; }
+    DeferredNorm forward(Runtime &rt, Tensor &x, const Batch &batch, const LayerIO &io, const DeferredNorm &pending,
+                         Norm *next_norm) override {
+        const int M = (int)x.rows, E = (int)x.cols;
+        const bool rounds = rt.dtype != FG_F32;
+        Tensor xin = x;
+        if (rounds && pending.defined() && pending.tiles == 0 && !pending.weight) xin = pending.xw;
+        else if (rounds) {
+            xin = rt.arena->matrix(M, E, rt.dtype);
+            if (M > 0) FG_LAUNCH("core", fg_cast_rows, x.ptr<float>(), (int)x.ld, xin.data, xin.dtype, (int)xin.ld, M, E, rt.stream);
+        }
+        Tensor t = rt.arena->matrix(M, E, FG_F32);
+        auto run = [&](bool can_overwrite, auto &&sublayer) {
+            rt.overwrite = can_overwrite;
+            if (!can_overwrite && M > 0) FG_CUDA(cudaMemsetAsync(t.data, 0, (size_t)M * E * sizeof(float), rt.stream));
+            sublayer();
+            rt.overwrite = false;
+        };
+        auto join = [&](Norm *post, Norm *reader) -> Tensor {
+            Tensor out;
+            if (reader || rounds) out = rt.arena->matrix(M, E, rt.dtype);
+            if (M > 0)
+                FG_LAUNCH("core", fg_norm_add_norm, t.ptr<float>(), post->weight(), x.ptr<float>(), reader ? reader->weight() : nullptr,
+                          out.data, rt.dtype, M, E, post->eps(), reader ? reader->eps() : 0.f, rt.stream);
+            return out;
+        };
+        Norm *reader = (next_norm && next_norm->deferrable() && next_norm->weight() && E * sizeof(float) <= 48 * 1024) ? next_norm : nullptr;
+        auto hand_over = [&](const Tensor &out) {
+            DeferredNorm d;
+            if (next_norm && !reader) return d;              // (the reader makes its norm itself)
+            if (out.defined()) { d.xw = out; d.tiles = 0; d.size = E; d.eps = reader ? reader->eps() : 0.f; d.x = x; d.weight = reader ? reader->weight() : nullptr; }
+            return d;
+        };
+        run(mixer->can_overwrite(), [&] { mixer->forward(rt, xin, nullptr, batch, io, t, nullptr); });
+        if (!feed_forward) return hand_over(join(mixer_post_norm, reader));
+        Tensor hin = join(mixer_post_norm, nullptr);
+        if (!rounds) hin = x;
+        run(feed_forward->can_overwrite(), [&] { feed_forward->forward(rt, hin, nullptr, batch, t, nullptr); });
+        return hand_over(join(feed_forward_post_norm, reader));
     }
 };
 
@@ -1287,6 +1353,7 @@ static std::map<std::string, PartFactory> &factories(int role) {
 static std::map<std::string, BlockFactory> &block_factories() {
     static std::map<std::string, BlockFactory> r = {{"prenorm", [](Runtime &) { return std::make_unique<PreNormBlock>(); }},
                                                      {"sandwich", [](Runtime &) { return std::make_unique<SandwichBlock>(); }},
+                                                     {"postnorm", [](Runtime &) { return std::make_unique<PostNormBlock>(); }},
                                                      {"parallel", [](Runtime &) { return std::make_unique<ParallelBlock>(); }}};
     return r;
 }

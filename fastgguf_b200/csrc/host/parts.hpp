@@ -171,6 +171,9 @@ public:
     // true: the block hands the NEXT block's first norm over finished (xw = the normalised rows, tiles == 0) instead of
     // started, and takes its own that way; between blocks of different habits nothing is handed over
     virtual bool finished_norms() const { return false; }
+    // true: the sublayers read the stream itself (there is no mixer_norm); such a block hands the rounded stream over (xw, tiles
+    // == 0, no weight) where the next block reads the stream too
+    virtual bool reads_stream() const { return false; }
     // Runs the block on x in place.  pending: the mixer's norm already started by whoever produced x;
     // next_norm: the norm that will read x after this block, to be started by the block's last projection.
     // Returns the started next_norm (or an undefined DeferredNorm).
@@ -256,8 +259,9 @@ public:
     // max(a W^T, 0)^2 in the activation dtype: in the tensor-core kernel's epilogue where that kernel runs, else the
     // contraction and an elementwise pass
     Tensor forward_relu2(Runtime &rt, const Tensor &a) const;
-    // silu(a gate^T) * (a up^T) as bf16 [M, F] from rows interleaved in blocks of 64; false if refused
-    bool forward_silu(Runtime &rt, const Tensor &a, const DeferredNorm *deferred, Tensor *out) const;
+    // act(a gate^T) * (a up^T) as bf16 [M, F] from rows interleaved in blocks of 64, act SiLU or the tanh form of gelu; false if
+    // refused
+    bool forward_gated(Runtime &rt, const Tensor &a, const DeferredNorm *deferred, bool gelu, Tensor *out) const;
 
 private:
     Weight w_;

@@ -20,6 +20,8 @@
 //         n_identity outputs have no expert: their "output" is the feed-forward's input itself.  Expert:
 //         W_down (silu(W_gate x) * (W_up x)).  shared_d_ff > 0: one more gated feed-forward of that size ("shared.*" tensors)
 //         runs on every row and is added.
+//         router "softmax_chosen": the top_k largest logits z + b (router.bias) are chosen; their weights are the softmax over the
+//         chosen logits alone and multiply the experts' OUTPUTS.  Expert with activation "relu2": W_down max(W_up x, 0)^2, no gate.
 #include <algorithm>
 #include <cmath>
 
@@ -63,8 +65,15 @@ public:
         top_ = (int)param_int(p, "top_k", me);
         const Json &r = p.get("router");
         std::string kind = r.is_string() ? r.as_string() : "sigmoid_input";
-        if (kind != "sigmoid_input" && kind != "softmax_grouped") fail(FG_E_CONFIG, "moe: router '" + kind + "' is not known (known: sigmoid_input, softmax_grouped)");
+        if (kind != "sigmoid_input" && kind != "softmax_grouped" && kind != "softmax_chosen")
+            fail(FG_E_CONFIG, "moe: router '" + kind + "' is not known (known: sigmoid_input, softmax_grouped, softmax_chosen)");
         grouped_ = kind == "softmax_grouped";
+        chosen_ = kind == "softmax_chosen";
+        const Json &a = p.get("activation");
+        const std::string act = a.is_string() ? a.as_string() : "gated";
+        if (act != "gated" && act != "relu2") fail(FG_E_CONFIG, "moe: activation '" + act + "' is not known (known: gated, relu2)");
+        relu2_ = act == "relu2";
+        if (relu2_ && !grouped_ && !chosen_) fail(FG_E_CONFIG, "moe: router 'sigmoid_input' weighs the inputs of gated experts");
         if (E_ <= 0 || F_ <= 0 || X_ <= 0 || top_ <= 0) fail(FG_E_CONFIG, "moe: sizes must be positive");
         if (grouped_) {
             identity_ = (int)param_int(p, "n_identity", 0, me);
@@ -84,22 +93,24 @@ public:
                 sp.set("d_ff", (long long)shared_ff_);
                 shared_ = make_swiglu(sp);
             }
+        } else if (chosen_) {
+            limit_ = 0.f;
         } else {
             limit_ = (float)param_float(p, "limit", me);
             alpha_ = (float)param_float(p, "alpha", 1.702, me);
             if (!(limit_ > 0.f)) fail(FG_E_CONFIG, "moe: limit must be positive");
         }
         if (top_ > X_ + identity_) fail(FG_E_CONFIG, format("moe: top_k %d exceeds the %d experts", top_, X_ + identity_));
-        if (X_ + identity_ > 256 || top_ > 8) fail(FG_E_CONFIG, "moe: the routing kernel takes up to 256 experts and top_k up to 8");
+        if (X_ + identity_ > 256 || top_ > 16) fail(FG_E_CONFIG, "moe: the routing kernel takes up to 256 experts and top_k up to 16");
     }
     std::vector<TensorDecl> tensor_decls() const override {
         std::vector<TensorDecl> d = {{"router.weight", {X_ + identity_, E_}}};
-        if (grouped_) d.push_back({"router.bias", {X_ + identity_}, false, 0, 0.05f});
+        if (grouped_ || chosen_) d.push_back({"router.bias", {X_ + identity_}, false, 0, 0.05f});
         if (shared_)
             for (auto &t : shared_->tensor_decls()) { TensorDecl c = t; c.name = "shared." + t.name; d.push_back(c); }
         for (int e = 0; e < X_; e++) {
             std::string pre = "experts." + std::to_string(e) + ".";
-            d.push_back({pre + "gate_proj.weight", {F_, E_}});
+            if (!relu2_) d.push_back({pre + "gate_proj.weight", {F_, E_}});
             d.push_back({pre + "up_proj.weight", {F_, E_}});
             d.push_back({pre + "down_proj.weight", {E_, F_}});
         }
@@ -108,18 +119,18 @@ public:
     bool can_overwrite() const override { return true; }
     void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
         router_ = Linear(tensor_of(tensors, "router.weight"));
-        // experts one after another: [X, 2F, E] (gate rows, then up rows) and [X, E, F], in the engine's dtype
+        // experts one after another: [X, 2F, E] (gate rows, then up rows; [X, F, E] without gates) and [X, E, F], in the engine's dtype
         std::vector<Weight> in, out;
         for (int e = 0; e < X_; e++) {
             std::string pre = "experts." + std::to_string(e) + ".";
-            in.push_back(tensor_of(tensors, (pre + "gate_proj.weight").c_str()));
+            if (!relu2_) in.push_back(tensor_of(tensors, (pre + "gate_proj.weight").c_str()));
             in.push_back(tensor_of(tensors, (pre + "up_proj.weight").c_str()));
             out.push_back(tensor_of(tensors, (pre + "down_proj.weight").c_str()));
         }
         w_in_ = concat_rows(in, rt.dtype, rt.stream);
         w_out_ = concat_rows(out, rt.dtype, rt.stream);
         if (!counts_host_) FG_CUDA(cudaMallocHost((void **)&counts_host_, ((size_t)X_ + identity_ + 1) * sizeof(int)));
-        if (grouped_) {
+        if (grouped_ || chosen_) {
             const Weight &b = tensor_of(tensors, "router.bias");
             route_bias_ = b.t.dtype == FG_F32 ? b : concat_rows({b}, FG_F32, rt.stream);
         }
@@ -166,13 +177,14 @@ private:
             FG_LAUNCH("mix", fg_moe_route_grouped, z.ptr<float>(), route_bias_.t.ptr<float>(), M, XR, top_, groups_, keep_, route_scale_, pair_expert,
                       pair_weight, offsets, order, slot_of, rt.stream);
         else
-            FG_LAUNCH("mix", fg_moe_route, z.ptr<float>(), M, X_, top_, pair_expert, pair_weight, offsets, order, slot_of, rt.stream);
+            FG_LAUNCH("mix", fg_moe_route_ext, z.ptr<float>(), chosen_ ? route_bias_.t.ptr<float>() : nullptr, chosen_ ? 1 : 0, M, X_, top_, pair_expert,
+                      pair_weight, offsets, order, slot_of, rt.stream);
         Tensor y = rt.arena->matrix(P, F_, rt.dtype);
         Tensor o = rt.arena->matrix(P, E_, FG_F32);
         // where the routing weight enters: the experts' inputs (through the float32 gate/up results), or their outputs (the sum)
-        const float *in_weight = grouped_ ? nullptr : pair_weight;
+        const float *in_weight = (grouped_ || chosen_) ? nullptr : pair_weight;
         auto combine = [&]() {
-            if (grouped_)
+            if (grouped_ || chosen_)
                 FG_LAUNCH("mix", fg_moe_combine_weighted, o.ptr<float>(), (int)o.ld, slot_of, pair_expert, pair_weight, xn.data, (int)xn.ld, xn.dtype, X_,
                           residual.ptr<float>(), M, top_, E_, rt.overwrite ? 0 : 1, rt.stream);
             else
@@ -181,22 +193,24 @@ private:
         if (!rt.recording && !rt.plain_kernels && rt.dtype == FG_BF16 && P >= grouped_from_ && E_ % 8 == 0 && F_ % 8 == 0) {
             // a long portion: the experts' row counts come to the host, and the experts' runs of rows go through the
             // tensor-core contraction; gate and up leave it as float32, so the routing weight and the clamps see what
-            // the accumulators held
+            // the accumulators held (experts without gates have their activation in the contraction's epilogue)
             FG_CUDA(cudaMemcpyAsync(counts_host_, offsets, ((size_t)XR + 1) * sizeof(int), cudaMemcpyDeviceToHost, rt.stream));
             FG_CUDA(cudaStreamSynchronize(rt.stream));
             Tensor xs = rt.arena->matrix(P, E_, rt.dtype);
             FG_LAUNCH("mix", fg_moe_gather, xn.data, (int)xn.ld, xn.dtype, order, top_, xs.data, P, E_, rt.stream);
-            Tensor gu = rt.arena->matrix(P, (int64_t)2 * F_, FG_F32);
+            const int in_rows = relu2_ ? F_ : 2 * F_;         // rows of an expert's first matrix
+            Tensor gu;
+            if (!relu2_) gu = rt.arena->matrix(P, (int64_t)2 * F_, FG_F32);
             // both contractions as ONE launch each over all experts: a table of tiles {first row, end of the expert's run,
             // the expert's first row in the stack, tile along the outputs}, an expert's tiles side by side so that its
             // weights stay in L2 while its row tiles pass
-            const int bn1 = FG_KERNEL("tc", fg_gemm_tc_grouped_bn)(2 * F_), bn2 = FG_KERNEL("tc", fg_gemm_tc_grouped_bn)(E_);
+            const int bn1 = FG_KERNEL("tc", fg_gemm_tc_grouped_bn)(in_rows), bn2 = FG_KERNEL("tc", fg_gemm_tc_grouped_bn)(E_);
             auto count_tiles = [&](int N, int bn) {
                 size_t n = 0;
                 for (int e = 0; e < X_; e++) n += (size_t)((counts_host_[e + 1] - counts_host_[e] + 127) / 128) * (size_t)((N + bn - 1) / bn);
                 return n;
             };
-            const size_t n1 = count_tiles(2 * F_, bn1), n2 = count_tiles(E_, bn2);
+            const size_t n1 = count_tiles(in_rows, bn1), n2 = count_tiles(E_, bn2);
             if (tiles_cap_ < n1 + n2) {
                 if (tiles_host_) FG_CUDA(cudaFreeHost(tiles_host_));
                 tiles_host_ = nullptr;
@@ -210,21 +224,31 @@ private:
                         for (int r = a; r < b; r += 128) { *t++ = r; *t++ = b; *t++ = e * N; *t++ = qt; }
                 }
             };
-            fill(tiles_host_, 2 * F_, bn1);
+            fill(tiles_host_, in_rows, bn1);
             fill(tiles_host_ + 4 * n1, E_, bn2);
             int *tiles_dev = (int *)rt.arena->alloc((n1 + n2) * 4 * sizeof(int));
             // (the stream was waited for above, after this buffer's last copy was queued: it is free to be rewritten)
             FG_CUDA(cudaMemcpyAsync(tiles_dev, tiles_host_, (n1 + n2) * 4 * sizeof(int), cudaMemcpyHostToDevice, rt.stream));
-            FG_LAUNCH("tc", fg_gemm_tc_grouped, xs.data, (int)xs.ld, P, w_in_.t.data, (int)w_in_.t.ld, (int)w_in_.t.rows, gu.ptr<float>(),
-                      (int)gu.ld, 2 * F_, E_, tiles_dev, (int)n1, rt.stream);
-            FG_LAUNCH("mix", fg_moe_act, gu.ptr<float>(), order, in_weight, y.data, y.dtype, P, F_, limit_, alpha_, rt.stream);
+            if (relu2_) {
+                const int EPI_RELU2_BF16 = 4;
+                FG_LAUNCH("tc", fg_gemm_tc_grouped_ext, xs.data, (int)xs.ld, P, w_in_.t.data, (int)w_in_.t.ld, (int)w_in_.t.rows, y.data, (int)y.ld,
+                          EPI_RELU2_BF16, F_, E_, tiles_dev, (int)n1, rt.stream);
+            } else {
+                FG_LAUNCH("tc", fg_gemm_tc_grouped, xs.data, (int)xs.ld, P, w_in_.t.data, (int)w_in_.t.ld, (int)w_in_.t.rows, gu.ptr<float>(),
+                          (int)gu.ld, 2 * F_, E_, tiles_dev, (int)n1, rt.stream);
+                FG_LAUNCH("mix", fg_moe_act, gu.ptr<float>(), order, in_weight, y.data, y.dtype, P, F_, limit_, alpha_, rt.stream);
+            }
             FG_LAUNCH("tc", fg_gemm_tc_grouped, y.data, (int)y.ld, P, w_out_.t.data, (int)w_out_.t.ld, (int)w_out_.t.rows, o.ptr<float>(),
                       (int)o.ld, E_, F_, tiles_dev + 4 * n1, (int)n2, rt.stream);
             combine();
             return DeferredNorm();
         }
-        FG_LAUNCH("mix", fg_moe_first, xn.data, (int)xn.ld, w_in_.t.data, y.data, (int)y.ld, rt.dtype, pair_expert, offsets, order, in_weight,
-                  M, X_, top_, F_, E_, limit_, alpha_, rt.stream);
+        if (relu2_)
+            FG_LAUNCH("mix", fg_moe_first_relu2, xn.data, (int)xn.ld, w_in_.t.data, y.data, (int)y.ld, rt.dtype, pair_expert, offsets, order, M, X_, top_, F_,
+                      E_, rt.stream);
+        else
+            FG_LAUNCH("mix", fg_moe_first, xn.data, (int)xn.ld, w_in_.t.data, y.data, (int)y.ld, rt.dtype, pair_expert, offsets, order, in_weight,
+                      M, X_, top_, F_, E_, limit_, alpha_, rt.stream);
         FG_LAUNCH("mix", fg_moe_second, y.data, (int)y.ld, w_out_.t.data, o.ptr<float>(), (int)o.ld, rt.dtype, pair_expert, offsets, order, M,
                   X_, top_, F_, E_, rt.stream);
         combine();
@@ -233,7 +257,8 @@ private:
 
     int E_ = 0, F_ = 0, X_ = 0, top_ = 0;
     int identity_ = 0, groups_ = 1, keep_ = 1, shared_ff_ = 0;      // router "softmax_grouped"
-    bool grouped_ = false;
+    bool grouped_ = false, chosen_ = false;  // the router's kind
+    bool relu2_ = false;                     // experts of two matrices, the squared ReLU between them
     float route_scale_ = 1.f;
     Weight route_bias_;
     std::unique_ptr<FeedForward> shared_;

@@ -423,8 +423,132 @@ private:
     Weight conv_w_, a_log_, dt_bias_, norm_;
 };
 
+// "rglru": a recurrent block around the real-gated linear recurrent unit.  With the mixer's input h, C = width channels and
+// n_blocks equal parts of them:
+//     y = gelu_tanh(W_y h + b_y),  u = causal convolution over time per channel of (W_x h + b_x), plus a bias   weights [C, taps]
+//     r = sigmoid(R u + b_r), i = sigmoid(I u + b_i)                     R, I: one square matrix a part
+//     log a = -gain r softplus(lam);  S_t = a S_(t-1) + sqrt(1 - a^2) i u;  output W_o (S y)
+// W_y and W_x are ONE contraction with float32 output; convolution, gates (their matrix products included), decays and state are
+// 32-bit in every engine dtype (rglru.cu); only S y takes the engine's dtype, as the output projection's input.
+class RecurrentUnitMixer : public Mixer {
+public:
+    RecurrentUnitMixer(const Json &p, BuildContext &) {
+        const char *me = "rglru";
+        E_ = (int)param_int(p, "hidden_size", me);
+        C_ = (int)param_int(p, "width", me);
+        B_ = (int)param_int(p, "n_blocks", 1, me);
+        taps_ = (int)param_int(p, "conv_taps", 1, me);
+        gain_ = (float)param_float(p, "gain", 8.0, me);
+        if (E_ <= 0 || C_ <= 0 || B_ <= 0 || taps_ <= 0) fail(FG_E_CONFIG, "rglru: sizes must be positive");
+        if (C_ % B_) fail(FG_E_CONFIG, format("rglru: %d channels do not split into %d equal blocks", C_, B_));
+        if (!(gain_ > 0.f)) fail(FG_E_CONFIG, "rglru: gain must be positive");
+    }
+    std::vector<TensorDecl> tensor_decls() const override {
+        const int64_t C = C_, B = B_, s = C_ / B_;
+        return {{"y_proj.weight", {C, E_}}, {"y_proj.bias", {C}, false, 0, 0.1f}, {"x_proj.weight", {C, E_}}, {"x_proj.bias", {C}, false, 0, 0.1f},
+                {"conv.weight", {C, (int64_t)taps_}, false, 0, 0.5f}, {"conv.bias", {C}, false, 0, 0.1f},
+                {"r_gate.weight", {B, s, s}, false, 0, 0.1f}, {"r_gate.bias", {B, s}, false, 0, 0.5f}, {"i_gate.weight", {B, s, s}, false, 0, 0.1f},
+                {"i_gate.bias", {B, s}, false, 0, 0.5f}, {"lam", {C}, false, 0, 1.0f}, {"o_proj.weight", {E_, C}}};
+    }
+    bool can_overwrite() const override { return true; }
+    bool supports_deferred_norm() const override { return true; }
+    bool strided_state() const override { return true; }
+    int64_t state_bytes() const override { return (int64_t)(taps_ > 1 ? taps_ + 1 : 1) * C_ * (int64_t)sizeof(float); }
+    void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
+        if (FG_KERNEL("mix", fg_rglru_state_floats)(C_, taps_) * (int64_t)sizeof(float) != state_bytes())
+            fail(FG_E_INTERNAL, "rglru: host and kernel library disagree on the size of a state row");
+        const Weight &y = tensor_of(tensors, "y_proj.weight"), &x = tensor_of(tensors, "x_proj.weight");
+        in_ = Linear(concat_rows({y, x}, y.t.dtype == x.t.dtype ? y.t.dtype : FG_F32, rt.stream));
+        o_ = Linear(tensor_of(tensors, "o_proj.weight"));
+        in_b_ = f32_rows({flat(tensors, "y_proj.bias"), flat(tensors, "x_proj.bias")}, rt.stream);
+        conv_w_ = f32_rows({tensor_of(tensors, "conv.weight")}, rt.stream);
+        conv_b_ = f32_rows({tensor_of(tensors, "conv.bias")}, rt.stream);
+        lam_ = f32_rows({tensor_of(tensors, "lam")}, rt.stream);
+        // part by part: the rows of R, then those of I
+        const int64_t s = C_ / B_;
+        Weight r = tensor_of(tensors, "r_gate.weight"), i = tensor_of(tensors, "i_gate.weight");
+        if (r.t.dtype != i.t.dtype) { r = f32_rows({r}, rt.stream); i = f32_rows({i}, rt.stream); }
+        gates_ = by_part(r, i, s * s, r.t.dtype, rt.stream);
+        gates_.t.rows = 2 * C_; gates_.t.cols = s; gates_.t.ld = s;
+        gate_b_ = by_part(f32_rows({tensor_of(tensors, "r_gate.bias")}, rt.stream), f32_rows({tensor_of(tensors, "i_gate.bias")}, rt.stream), s, FG_F32, rt.stream);
+        if (rt.dtype == FG_BF16 && !rt.plain_kernels && gates_.t.dtype == FG_BF16 && s % 8 == 0) {
+            // the matrix three times side by side: it meets u as three bfloat16 numbers (rglru.cu)
+            wide_ = make_weight(2 * C_, 3 * s, FG_BF16, "gates of a recurrent unit");
+            for (int k = 0; k < 3; k++)
+                FG_CUDA(cudaMemcpy2DAsync((char *)wide_.t.data + (size_t)k * s * 2, (size_t)3 * s * 2, gates_.t.data, (size_t)s * 2, (size_t)s * 2, (size_t)2 * C_,
+                                          cudaMemcpyDeviceToDevice, rt.stream));
+        }
+        FG_CUDA(cudaStreamSynchronize(rt.stream));
+    }
+    DeferredNorm forward(Runtime &rt, const Tensor &xn, const DeferredNorm *deferred, const Batch &b, const LayerIO &io, Tensor &residual,
+                         Norm *emit_norm) override {
+        if (!io.state || io.state_bytes < state_bytes()) fail(FG_E_INTERNAL, "rglru: the schedule entry has no state rows");
+        const long long stride = (long long)(io.state_stride / (int64_t)sizeof(float));
+        const int s = C_ / B_;
+        float *state = (float *)io.state;
+        Tensor proj = in_.forward(rt, xn, deferred, Tensor(), FG_F32, false, nullptr, nullptr);
+        const int M = (int)proj.rows, ld = (int)proj.ld;
+        const float *in_b = in_b_.t.ptr<float>(), *conv_w = conv_w_.t.ptr<float>(), *conv_b = conv_b_.t.ptr<float>(), *gate_b = gate_b_.t.ptr<float>(),
+                    *lam = lam_.t.ptr<float>();
+        Tensor y = rt.arena->matrix(M, C_, rt.dtype);
+        if (b.single_token && FG_KERNEL("mix", fg_rglru_step_ok)(s)) {
+            FG_LAUNCH("mix", fg_rglru_step, proj.ptr<float>(), ld, in_b, conv_w, conv_b, taps_, gates_.t.data, gates_.t.dtype, gate_b, lam, gain_, b.positions,
+                      b.row_seq, b.slots, state, stride, y.data, y.dtype, (int)y.ld, M, C_, s, rt.stream);
+        } else {
+            Tensor u = rt.arena->matrix(M, C_, FG_F32), z;
+            long long z_row = 2 * C_, z_part = 2 * s;
+            const bool tc = wide_.t.defined() && !b.single_token && M >= tensor_cores_from_;
+            if (tc) {
+                Tensor pieces = rt.arena->matrix((int64_t)B_ * M, (int64_t)3 * s, FG_BF16);
+                z = rt.arena->matrix((int64_t)B_ * M, (int64_t)2 * s, FG_F32);
+                z_row = 2 * s; z_part = (long long)M * 2 * s;
+                const int bn = FG_KERNEL("tc", fg_gemm_tc_grouped_bn)(2 * s), n_tiles = FG_KERNEL("mix", fg_rglru_tiles)(M, C_, s, bn);
+                void *tiles = rt.arena->alloc((size_t)n_tiles * 4 * sizeof(int));
+                FG_LAUNCH("mix", fg_rglru_conv, proj.ptr<float>(), ld, in_b, conv_w, conv_b, taps_, state, stride, b.positions, b.row_seq, b.cu_rows, b.slots,
+                          u.ptr<float>(), (int)u.ld, pieces.data, tiles, bn, M, C_, s, rt.stream);
+                FG_LAUNCH("tc", fg_gemm_tc_grouped, pieces.data, (int)pieces.ld, (int)pieces.rows, wide_.t.data, (int)wide_.t.ld, (int)wide_.t.rows,
+                          z.ptr<float>(), (int)z.ld, 2 * s, 3 * s, tiles, n_tiles, rt.stream);
+            } else {
+                z = rt.arena->matrix(M, (int64_t)2 * C_, FG_F32);
+                FG_LAUNCH("mix", fg_rglru_conv, proj.ptr<float>(), ld, in_b, conv_w, conv_b, taps_, state, stride, b.positions, b.row_seq, b.cu_rows, b.slots,
+                          u.ptr<float>(), (int)u.ld, nullptr, nullptr, 0, M, C_, s, rt.stream);
+                FG_LAUNCH("mix", fg_head_gemm, u.data, FG_F32, (int)u.ld, s, gates_.t.data, gates_.t.dtype, s, 0, z.data, FG_F32, (int)z.ld, 2 * s, nullptr, 0, M,
+                          2 * s, s, B_, rt.stream);
+            }
+            FG_LAUNCH("mix", fg_rglru_scan, z.ptr<float>(), z_row, z_part, gate_b, u.ptr<float>(), (int)u.ld, lam, gain_, proj.ptr<float>(), ld, in_b, y.data,
+                      y.dtype, (int)y.ld, b.cu_rows, b.slots, b.positions, state, stride, b.n_seq, b.max_new, C_, s, taps_, rt.stream);
+        }
+        DeferredNorm started;
+        o_.forward(rt, y, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
+        return started;
+    }
+
+private:
+    static Weight flat(const std::map<std::string, Weight> &tensors, const char *name) {
+        Weight w = tensor_of(tensors, name);
+        w.t.rows = w.t.numel(); w.t.cols = 1; w.t.ld = 1;
+        return w;
+    }
+    // [parts][2][n]: part p of a, then part p of b
+    Weight by_part(const Weight &a, const Weight &b, int64_t n, int dtype, cudaStream_t st) const {
+        const size_t bytes = (size_t)n * elem_size(dtype);
+        Weight out = make_weight(2 * B_, n, dtype, "gates of a recurrent unit");
+        int at = 0;
+        for (const Weight *w : {&a, &b})
+            FG_CUDA(cudaMemcpy2DAsync((char *)out.t.data + bytes * at++, 2 * bytes, w->t.data, bytes, bytes, (size_t)B_, cudaMemcpyDeviceToDevice, st));
+        FG_CUDA(cudaStreamSynchronize(st));            // a and b may go away with the caller's expression
+        return out;
+    }
+    int E_ = 0, C_ = 0, B_ = 1, taps_ = 1;
+    int tensor_cores_from_ = 64;             // rows from which the gates run on the tensor cores
+    float gain_ = 8.f;
+    Linear in_, o_;
+    Weight in_b_, conv_w_, conv_b_, lam_, gates_, gate_b_, wide_;
+};
+
 void add_recurrent_kinds(std::map<std::string, PartFactory> &mixers) {
     mixers["gated_linear_attention"] = [](Runtime &, const Json &p, BuildContext &c) { return std::make_unique<GatedLinearAttention>(p, c); };
+    mixers["rglru"] = [](Runtime &, const Json &p, BuildContext &c) { return std::make_unique<RecurrentUnitMixer>(p, c); };
     mixers["retention"] = [](Runtime &, const Json &p, BuildContext &c) { return std::make_unique<RetentionMixer>(p, c); };
     mixers["state_space"] = [](Runtime &, const Json &p, BuildContext &c) { return std::make_unique<StateSpaceMixer>(p, c); };
     mixers["gated_delta"] = [](Runtime &, const Json &p, BuildContext &c) { return std::make_unique<GatedDeltaMixer>(p, c); };

@@ -1,0 +1,389 @@
+// The real-gated linear recurrent unit and what stands between its projections and its output projection.
+//
+// A recurrent block has two branches of C channels, y and x (both out of one contraction, float32, without their biases):
+//     u = conv_b + causal convolution over time per channel of (x + x_bias)      weights [C, taps], zeros before the sequence
+//     r = sigmoid(R u + r_bias), i = sigmoid(I u + i_bias)                       R, I block diagonal: `blocks` squares of C / blocks
+//     log a = -gain r softplus(lam);  S_t = a S_(t-1) + sqrt(1 - a^2) i u;       out = S gelu_tanh(y + y_bias)
+// Everything here is 32-bit in every engine dtype; only out takes the engine's.
+//
+// State row of a sequence: [a ring of `taps` convolution inputs, each C floats (none with one tap) | S, C floats].  The input of
+// position p lies at p mod taps, so a single-token step reads the entries of p - 1 .. p - taps + 1 and writes that of p, which is
+// none of them: one kernel does both, whatever order its blocks run in.
+//
+//   fg_rglru_step: a step of single tokens, all of it in ONE launch - a block per (16 channels of a part, 8 rows) forms u of the
+//     whole part in shared memory, its warps stream two channels' rows of R and I for the eight rows, and the lanes that end up
+//     with a (channel, row) finish it.
+//   fg_rglru_conv, the gates, fg_rglru_scan: prompts and portions.  The gates' contraction reads u in 32 bits; so that the tensor
+//     cores can run it, fg_rglru_conv also writes u as three bfloat16 numbers whose sum is u (8 + 8 + 8 bits of mantissa): with
+//     the matrix three times side by side along k, products of bfloat16 numbers are exact and the sum is a 32-bit one.
+//   fg_rglru_scan: the recurrence is linear with a diagonal matrix, so it is cut along time: a thread owns a channel and
+//     SCAN_T tokens, forms their (a, b) once in registers and composes them; the compositions of a block's warps meet in shared
+//     memory, those of a cluster's blocks in one another's, and every thread then walks its tokens from the right start.
+#include "common.cuh"
+
+#define SCAN_W 8                      // warps a block (a warp: 32 channels)
+#define SCAN_T 16                     // tokens a thread
+#define SCAN_MAX_CLUSTER 8
+#define STEP_ROWS 8                   // rows (sequences) a block of the single-token kernel serves
+#define STEP_CHANNELS 16              // channels it finishes, two a warp
+#define CONV_ROWS 8                   // rows a thread of the convolution walks
+
+__device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float rg_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float rg_gelu(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// a and the input term of one token: rate = gain * softplus(lam)
+__device__ __forceinline__ void rg_coefficients(float zr, float zi, float u, float rate, float &a, float &b) {
+    const float log_a = -rate * rg_sigmoid(zr);
+    a = expf(log_a);
+    b = sqrtf(-expm1f(2.0f * log_a)) * (rg_sigmoid(zi) * u);      // 1 - a^2 without cancellation where a is close to 1
+}
+
+// ------------------------------------------------------------------ convolution, prompts and portions
+// NC neighbouring channels a thread.  pieces (optional): [part][row][3][size of a part] bfloat16, see above.  tiles (optional): the
+// table of the grouped contraction that reads them - for each part, for each tile along its outputs, its rows in runs of 128.
+template <int NC>
+__global__ void __launch_bounds__(256)
+rglru_conv_kernel(const float *__restrict__ x, int ld, const float *__restrict__ x_bias, const float *__restrict__ w,
+                  const float *__restrict__ conv_b, int taps, const float *__restrict__ state, long long state_stride,
+                  const int *__restrict__ positions, const int *__restrict__ row_seq, const int *__restrict__ cu_rows,
+                  const int *__restrict__ slots, float *__restrict__ u, int ldu, bf16 *__restrict__ pieces, int4 *__restrict__ tiles,
+                  int n_tiles, int tiles_n, int M, int C, int part) {
+    pdl_wait();
+    if (tiles && blockIdx.x == 0 && blockIdx.y == 0) {
+        const int row_tiles = (M + 127) / 128;
+        for (int t = threadIdx.x; t < n_tiles; t += 256) {
+            const int b = t / (tiles_n * row_tiles), rest = t - b * tiles_n * row_tiles, qt = rest / row_tiles, rt = rest - qt * row_tiles;
+            tiles[t] = make_int4(b * M + rt * 128, (b + 1) * M, b * 2 * part, qt);
+        }
+    }
+    const int c = (blockIdx.y * 256 + threadIdx.x) * NC;
+    if (c >= C) return;
+    float xb[NC], cb[NC];
+#pragma unroll
+    for (int q = 0; q < NC; q++) { xb[q] = x_bias[c + q]; cb[q] = conv_b[c + q]; }
+    const int p = c / part, j0 = c - p * part;               // (NC channels of one part: a part is a multiple of NC)
+    for (int m = blockIdx.x * CONV_ROWS; m < min(M, (int)(blockIdx.x + 1) * CONV_ROWS); m++) {
+        const int s = row_seq[m], i = m - cu_rows[s], pos = positions[m];
+        const float *ring = state + (size_t)slots[s] * state_stride;
+        float acc[NC];
+#pragma unroll
+        for (int q = 0; q < NC; q++) acc[q] = cb[q];
+        for (int back = taps - 1; back >= 0; back--) {
+            float v[NC];
+            if (back <= i) {
+                const float *src = x + (size_t)(m - back) * ld + c;
+#pragma unroll
+                for (int q = 0; q < NC; q++) v[q] = src[q] + xb[q];
+            } else if (pos - back >= 0) {
+                const float *src = ring + (size_t)((pos - back) % taps) * C + c;
+#pragma unroll
+                for (int q = 0; q < NC; q++) v[q] = src[q];
+            } else continue;
+#pragma unroll
+            for (int q = 0; q < NC; q++) acc[q] = fmaf(w[(size_t)(c + q) * taps + taps - 1 - back], v[q], acc[q]);
+        }
+        if (NC == 2) *(float2 *)(u + (size_t)m * ldu + c) = make_float2(acc[0], acc[NC - 1]);
+        else u[(size_t)m * ldu + c] = acc[0];
+        if (pieces) {
+            bf16 *dst = pieces + ((size_t)p * M + m) * 3 * part + j0;
+            float rest[NC];
+#pragma unroll
+            for (int q = 0; q < NC; q++) rest[q] = acc[q];
+#pragma unroll
+            for (int e = 0; e < 3; e++, dst += part) {
+                bf16 h[NC];
+#pragma unroll
+                for (int q = 0; q < NC; q++) { h[q] = __float2bfloat16_rn(rest[q]); rest[q] -= __bfloat162float(h[q]); }
+                if (NC == 2) { __nv_bfloat162 two; two.x = h[0]; two.y = h[NC - 1]; *(__nv_bfloat162 *)dst = two; }
+                else dst[0] = h[0];
+            }
+        }
+    }
+}
+
+// ------------------------------------------------------------------ the recurrence over a portion
+__device__ __forceinline__ void rg_cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float rg_remote(const float *p, int rank) {
+    const uint32_t local = (uint32_t)__cvta_generic_to_shared(p);
+    uint32_t remote;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote) : "memory");
+    return v;
+}
+
+// z: the gates' raw numbers, row m of part p at z + m * z_row + p * z_part: [r: part | i: part]; gate_bias the same for one row.
+// grid (channel tiles of 32, sequences, blocks of the cluster): the cluster's blocks stand one after another along time.
+template <typename TO>
+__global__ void __launch_bounds__(SCAN_W * 32)
+rglru_scan_kernel(const float *__restrict__ z, long long z_row, long long z_part, const float *__restrict__ gate_bias,
+                  const float *__restrict__ u, int ldu, const float *__restrict__ lam, float gain, const float *__restrict__ proj, int ldp,
+                  const float *__restrict__ proj_bias, TO *__restrict__ out, int ldo, const int *__restrict__ cu_rows,
+                  const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ state, long long state_stride, int C,
+                  int part, int taps) {
+    __shared__ float agg_a[SCAN_W][32], agg_b[SCAN_W][32];
+    __shared__ float tot_a[2][32], tot_b[2][32];
+    pdl_wait();
+    const int seq = blockIdx.y, rank = blockIdx.z, CS = gridDim.z, warp = warp_index(), lane = threadIdx.x & 31;
+    const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1];
+    if (row1 <= row0) return;                                   // the whole cluster leaves
+    const int c = blockIdx.x * 32 + lane;
+    const bool live = c < C;
+    const int cc = live ? c : 0, p = cc / part, j = cc - p * part;
+    const float *zr = z + p * z_part + j, *zi = zr + part;
+    const float br = gate_bias[(size_t)p * 2 * part + j], bi = gate_bias[(size_t)p * 2 * part + part + j];
+    const float rate = gain * rg_softplus(lam[cc]), yb = proj_bias[cc];
+    float *ring = state + (size_t)slots[seq] * state_stride, *Sg = ring + (taps > 1 ? (size_t)taps * C : 0);
+    float carry = live ? Sg[c] : 0.f;
+    int it = 0;
+    for (int t0 = row0; t0 < row1; t0 += CS * SCAN_W * SCAN_T, it ^= 1) {
+        const int first = t0 + (rank * SCAN_W + warp) * SCAN_T;
+        const int n = live ? max(0, min(SCAN_T, row1 - first)) : 0;
+        float a[SCAN_T], b[SCAN_T];
+        {
+            float vr[SCAN_T], vi[SCAN_T], vu[SCAN_T];            // all loads on their way before the first is used
+#pragma unroll
+            for (int i = 0; i < SCAN_T; i++) {
+                const size_t m = (size_t)(first + i);
+                vr[i] = i < n ? zr[m * z_row] : 0.f;
+                vi[i] = i < n ? zi[m * z_row] : 0.f;
+                vu[i] = i < n ? u[m * ldu + c] : 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < SCAN_T; i++) {
+                a[i] = 1.f; b[i] = 0.f;
+                if (i < n) rg_coefficients(vr[i] + br, vi[i] + bi, vu[i], rate, a[i], b[i]);
+            }
+        }
+        float wa = 1.f, wb = 0.f;                               // this thread's tokens composed: S -> wa S + wb
+#pragma unroll
+        for (int i = 0; i < SCAN_T; i++) { wb = fmaf(a[i], wb, b[i]); wa *= a[i]; }
+        agg_a[warp][lane] = wa;
+        agg_b[warp][lane] = wb;
+        float y[SCAN_T];
+#pragma unroll
+        for (int i = 0; i < SCAN_T; i++) y[i] = i < n ? proj[(size_t)(first + i) * ldp + c] : 0.f;
+        __syncthreads();
+        float pa = 1.f, pb = 0.f, ta = 1.f, tb = 0.f;           // before this warp; the whole block
+#pragma unroll
+        for (int w = 0; w < SCAN_W; w++) {
+            if (w == warp) { pa = ta; pb = tb; }
+            tb = fmaf(agg_a[w][lane], tb, agg_b[w][lane]);
+            ta *= agg_a[w][lane];
+        }
+        float start = carry;
+        if (CS > 1) {
+            if (warp == 0) { tot_a[it][lane] = ta; tot_b[it][lane] = tb; }
+            rg_cluster_sync();                                  // (two sets of totals: the next but one iteration's writes come after everybody's reads)
+            float S = carry, ra[SCAN_MAX_CLUSTER], rb[SCAN_MAX_CLUSTER];
+#pragma unroll
+            for (int r = 0; r < SCAN_MAX_CLUSTER; r++) {
+                ra[r] = r < CS ? rg_remote(&tot_a[it][lane], r) : 1.f;
+                rb[r] = r < CS ? rg_remote(&tot_b[it][lane], r) : 0.f;
+            }
+#pragma unroll
+            for (int r = 0; r < SCAN_MAX_CLUSTER; r++) {
+                if (r == rank) start = S;
+                S = fmaf(ra[r], S, rb[r]);
+            }
+            carry = S;
+        } else {
+            carry = fmaf(ta, carry, tb);
+            __syncthreads();                                    // the compositions are read before the next ones are written
+        }
+        float S = fmaf(pa, start, pb);
+#pragma unroll
+        for (int i = 0; i < SCAN_T; i++) {
+            S = fmaf(a[i], S, b[i]);
+            if (i < n) out[(size_t)(first + i) * ldo + c] = from_f32<TO>(S * rg_gelu(y[i] + yb));
+        }
+    }
+    if (CS > 1) rg_cluster_sync();                              // nobody's totals go away while they are being read
+    if (rank != 0 || !live) return;
+    if (warp == 0) Sg[c] = carry;
+    else if (warp == 1 && taps > 1) {
+        // the portion's last inputs of the convolution to their places in the ring
+        const float xb = proj_bias[C + c];
+        const int n = row1 - row0, pos0 = positions[row0];
+        for (int i = max(0, n - (taps - 1)); i < n; i++) ring[(size_t)((pos0 + i) % taps) * C + c] = proj[(size_t)(row0 + i) * ldp + C + c] + xb;
+    }
+}
+
+// ------------------------------------------------------------------ a step of single tokens
+// W: [part][2 * size][size] rows of R, then of I.  grid (16 channels of a part, parts, 8 rows).
+template <typename TW, typename TO>
+__global__ void __launch_bounds__(256)
+rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ proj_bias, const float *__restrict__ conv_w,
+                  const float *__restrict__ conv_b, int taps, const TW *__restrict__ W, const float *__restrict__ gate_bias,
+                  const float *__restrict__ lam, float gain, const int *__restrict__ positions, const int *__restrict__ row_seq,
+                  const int *__restrict__ slots, float *__restrict__ state, long long state_stride, TO *__restrict__ out, int ldo, int M, int C,
+                  int part, int stride, int vec) {
+    extern __shared__ __align__(16) float us[];                 // [STEP_ROWS][stride] u of the part
+    constexpr int VEC = 16 / (int)sizeof(TW);
+    const int p = blockIdx.y, tid = threadIdx.x, warp = warp_index(), lane = tid & 31;
+    const int j0 = blockIdx.x * STEP_CHANNELS + warp * 2;       // the warp's channels j0, j0 + 1 of the part
+    // the warp's four rows: R of both channels, then I of both (channels beyond the part repeat its last one and are not stored)
+    const TW *wr[4];
+#pragma unroll
+    for (int q = 0; q < 4; q++) wr[q] = W + ((size_t)p * 2 * part + (q >> 1) * part + min(j0 + (q & 1), part - 1)) * part;
+    uint4 w4[4];
+    const bool have = vec && lane * VEC < part;
+    if (have) {                                                  // weights: before the wait on the contraction in front
+#pragma unroll
+        for (int q = 0; q < 4; q++) w4[q] = *(const uint4 *)(wr[q] + lane * VEC);
+    }
+    pdl_launch_dependents_small_step(M);
+    pdl_wait();
+    const int m0 = blockIdx.z * STEP_ROWS;
+    for (int e = tid; e < STEP_ROWS * stride; e += 256) {
+        const int row = e / stride, j = e - row * stride, m = m0 + row;
+        float acc = 0.f;
+        if (m < M && j < part) {
+            const int c = p * part + j, pos = positions[m];
+            float *ring = state + (size_t)slots[row_seq[m]] * state_stride;
+            const float now = proj[(size_t)m * ldp + C + c] + proj_bias[C + c];
+            acc = conv_b[c];
+            for (int back = taps - 1; back > 0; back--)
+                if (pos - back >= 0) acc = fmaf(conv_w[(size_t)c * taps + taps - 1 - back], ring[(size_t)((pos - back) % taps) * C + c], acc);
+            acc = fmaf(conv_w[(size_t)c * taps + taps - 1], now, acc);
+            if (taps > 1 && j / STEP_CHANNELS == blockIdx.x) ring[(size_t)(pos % taps) * C + c] = now;
+        }
+        us[e] = acc;
+    }
+    __syncthreads();
+    float v[4 * STEP_ROWS];                                      // [row of W][row of the step]
+#pragma unroll
+    for (int i = 0; i < 4 * STEP_ROWS; i++) v[i] = 0.f;
+    if (vec) {
+        for (int k = lane * VEC; k < part; k += 32 * VEC) {
+#pragma unroll
+            for (int q = 0; q < 4; q++)
+                if (k >= 32 * VEC) w4[q] = *(const uint4 *)(wr[q] + k);
+#pragma unroll
+            for (int row = 0; row < STEP_ROWS; row++) {
+                float x[VEC];
+#pragma unroll
+                for (int i = 0; i < VEC; i += 4) *(float4 *)(x + i) = *(const float4 *)(us + row * stride + k + i);
+#pragma unroll
+                for (int q = 0; q < 4; q++) {
+                    const TW *we = (const TW *)&w4[q];
+#pragma unroll
+                    for (int i = 0; i < VEC; i++) v[q * STEP_ROWS + row] = fmaf(x[i], to_f32<TW>(we[i]), v[q * STEP_ROWS + row]);
+                }
+            }
+        }
+    } else {
+        for (int k = lane; k < part; k += 32) {
+            float w[4];
+#pragma unroll
+            for (int q = 0; q < 4; q++) w[q] = to_f32<TW>(wr[q][k]);
+#pragma unroll
+            for (int row = 0; row < STEP_ROWS; row++) {
+                const float x = us[row * stride + k];
+#pragma unroll
+                for (int q = 0; q < 4; q++) v[q * STEP_ROWS + row] = fmaf(x, w[q], v[q * STEP_ROWS + row]);
+            }
+        }
+    }
+    // 32 sums over 32 lanes: at every exchange a lane keeps half of its numbers, and ends with sum number `lane`
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool up = (lane & o) != 0;
+#pragma unroll
+        for (int i = 0; i < o; i++) {
+            const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+    const float zi = __shfl_xor_sync(0xffffffffu, v[0], 16);     // lanes 0 .. 15: R u of (channel lane / 8, row lane % 8); I u from lane + 16
+    const int j = j0 + ((lane >> 3) & 1), row = lane & 7, m = m0 + row;
+    if (lane >= 16 || j >= part || m >= M) return;
+    const int c = p * part + j;
+    float a, b;
+    rg_coefficients(v[0] + gate_bias[(size_t)p * 2 * part + j], zi + gate_bias[(size_t)p * 2 * part + part + j], us[row * stride + j],
+                    gain * rg_softplus(lam[c]), a, b);
+    float *Sg = state + (size_t)slots[row_seq[m]] * state_stride + (taps > 1 ? (size_t)taps * C : 0);
+    const float S = fmaf(a, Sg[c], b);
+    Sg[c] = S;
+    out[(size_t)m * ldo + c] = from_f32<TO>(S * rg_gelu(proj[(size_t)m * ldp + c] + proj_bias[c]));
+}
+
+// ------------------------------------------------------------------ launchers
+// floats of a sequence's state row
+extern "C" long long fg_rglru_state_floats(int C, int taps) { return (long long)(taps > 1 ? taps + 1 : 1) * C; }
+
+// proj: [M, ldp] float32, columns [y: C | x: C] without their biases (proj_bias [2 C]); u: [M, ldu] float32.  pieces (or null):
+// [C / part][M][3 * part] bfloat16, tiles (with pieces): the grouped contraction's table for outputs of 2 * part in tiles of bn,
+// fg_rglru_tiles(M, C, part, bn) entries.
+extern "C" int fg_rglru_tiles(int M, int C, int part, int bn) { return (C / part) * ((2 * part + bn - 1) / bn) * ((M + 127) / 128); }
+
+extern "C" int fg_rglru_conv(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps,
+                             const float *state, long long state_stride, const int *positions, const int *row_seq, const int *cu_rows,
+                             const int *slots, float *u, int ldu, void *pieces, void *tiles, int bn, int M, int C, int part, cudaStream_t stream) {
+    if (M <= 0) return 0;
+    if (C <= 0 || part <= 0 || C % part || taps <= 0 || (pieces && (!tiles || bn <= 0))) return FG_ERR_BAD_SIZE;
+    const bool two = part % 2 == 0 && ldu % 2 == 0 && (((uintptr_t)u) & 7) == 0 && (((uintptr_t)pieces) & 3) == 0;
+    const int n_tiles = pieces ? fg_rglru_tiles(M, C, part, bn) : 0, tiles_n = pieces ? (2 * part + bn - 1) / bn : 0;
+    const int per = two ? 512 : 256;
+    const dim3 grid((M + CONV_ROWS - 1) / CONV_ROWS, (C + per - 1) / per);
+#define RG_CONV(NC) fg_launch(rglru_conv_kernel<NC>, grid, dim3(256), 0, stream, proj + C, ldp, proj_bias + C, conv_w, conv_b, taps, state, state_stride, \
+                              positions, row_seq, cu_rows, slots, u, ldu, (bf16 *)pieces, (int4 *)tiles, n_tiles, tiles_n, M, C, part)
+    return two ? RG_CONV(2) : RG_CONV(1);
+#undef RG_CONV
+}
+
+// z: the gates' raw numbers (row m of part p: [r | i] at z + m * z_row + p * z_part); gate_bias: [C / part][2 * part]; lam: [C];
+// out: [M, ldo] in out_dtype.  Brings the state rows up to date.  max_new: the longest portion of the step.
+extern "C" int fg_rglru_scan(const float *z, long long z_row, long long z_part, const float *gate_bias, const float *u, int ldu,
+                             const float *lam, float gain, const float *proj, int ldp, const float *proj_bias, void *out, int out_dtype, int ldo,
+                             const int *cu_rows, const int *slots, const int *positions, float *state, long long state_stride, int n_seq,
+                             int max_new, int C, int part, int taps, cudaStream_t stream) {
+    if (n_seq <= 0 || max_new <= 0) return 0;
+    if (C <= 0 || part <= 0 || C % part || taps <= 0 || n_seq > 65535) return FG_ERR_BAD_SIZE;
+    int cs = 1;
+    while (cs < SCAN_MAX_CLUSTER && cs * SCAN_W * SCAN_T < max_new) cs *= 2;
+    const dim3 grid((C + 31) / 32, n_seq, cs);
+    if (out_dtype == FG_F32)
+        return fg_launch_cluster(rglru_scan_kernel<float>, grid, dim3(SCAN_W * 32), 0, stream, cs, z, z_row, z_part, gate_bias, u, ldu, lam, gain, proj,
+                                 ldp, proj_bias, (float *)out, ldo, cu_rows, slots, positions, state, state_stride, C, part, taps);
+    if (out_dtype == FG_BF16)
+        return fg_launch_cluster(rglru_scan_kernel<bf16>, grid, dim3(SCAN_W * 32), 0, stream, cs, z, z_row, z_part, gate_bias, u, ldu, lam, gain, proj,
+                                 ldp, proj_bias, (bf16 *)out, ldo, cu_rows, slots, positions, state, state_stride, C, part, taps);
+    return FG_ERR_BAD_DTYPE;
+}
+
+// 1 if the single-token kernel holds a part of this size in shared memory
+extern "C" int fg_rglru_step_ok(int part) { return part > 0 && (size_t)STEP_ROWS * ((part + 3) / 4 * 4) * sizeof(float) <= 200 * 1024; }
+
+template <typename TW, typename TO>
+static int rglru_step_launch(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps, const void *W,
+                             const float *gate_bias, const float *lam, float gain, const int *positions, const int *row_seq, const int *slots,
+                             float *state, long long state_stride, void *out, int ldo, int M, int C, int part, cudaStream_t stream) {
+    static FgPerDevice setup;
+    if (fg_needs_setup(setup)) {
+        cudaError_t e = cudaFuncSetAttribute(rglru_step_kernel<TW, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return (int)e;
+    }
+    const int stride = (part + 3) / 4 * 4, vec = part % (16 / (int)sizeof(TW)) == 0 && (((uintptr_t)W) & 15) == 0;
+    const dim3 grid((part + STEP_CHANNELS - 1) / STEP_CHANNELS, C / part, (M + STEP_ROWS - 1) / STEP_ROWS);
+    return fg_launch(rglru_step_kernel<TW, TO>, grid, dim3(256), (size_t)STEP_ROWS * stride * sizeof(float), stream, proj, ldp, proj_bias, conv_w,
+                     conv_b, taps, (const TW *)W, gate_bias, lam, gain, positions, row_seq, slots, state, state_stride, (TO *)out, ldo, M, C, part, stride, vec);
+}
+
+// A step of single tokens (one row a sequence).  W: [C / part][2 * part][part] in w_dtype.
+extern "C" int fg_rglru_step(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps,
+                             const void *W, int w_dtype, const float *gate_bias, const float *lam, float gain, const int *positions,
+                             const int *row_seq, const int *slots, float *state, long long state_stride, void *out, int out_dtype, int ldo, int M,
+                             int C, int part, cudaStream_t stream) {
+    if (M <= 0) return 0;
+    if (C <= 0 || part <= 0 || C % part || taps <= 0 || C / part > 65535 || M > 65535 * STEP_ROWS || !fg_rglru_step_ok(part)) return FG_ERR_BAD_SIZE;
+#define RG_STEP(TW, TO) rglru_step_launch<TW, TO>(proj, ldp, proj_bias, conv_w, conv_b, taps, W, gate_bias, lam, gain, positions, row_seq, slots, state, \
+                                                  state_stride, out, ldo, M, C, part, stream)
+    if (w_dtype == FG_F32) return out_dtype == FG_F32 ? RG_STEP(float, float) : out_dtype == FG_BF16 ? RG_STEP(float, bf16) : FG_ERR_BAD_DTYPE;
+    if (w_dtype == FG_BF16) return out_dtype == FG_F32 ? RG_STEP(bf16, float) : out_dtype == FG_BF16 ? RG_STEP(bf16, bf16) : FG_ERR_BAD_DTYPE;
+#undef RG_STEP
+    return FG_ERR_BAD_DTYPE;
+}

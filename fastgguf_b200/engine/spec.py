@@ -44,7 +44,7 @@ class LayerSpec:
     block: str                     # arrangement kind, e.g. "prenorm", "sandwich"
     mixer: PartSpec
     feed_forward: Optional[PartSpec]           # None: a layer of a mixer alone
-    mixer_norm: PartSpec
+    mixer_norm: Optional[PartSpec]             # None: block "postnorm", whose sublayers read the stream itself
     feed_forward_norm: Optional[PartSpec]
     #: norms on a sublayer's output, before it joins the residual stream (block "sandwich")
     mixer_post_norm: Optional[PartSpec] = None
@@ -56,7 +56,7 @@ class LayerSpec:
         def opt(p):
             return p.to_json() if p is not None else None
         j = {"block": self.block, "mixer": self.mixer.to_json(), "feed_forward": opt(self.feed_forward),
-             "mixer_norm": self.mixer_norm.to_json(), "feed_forward_norm": opt(self.feed_forward_norm)}
+             "mixer_norm": opt(self.mixer_norm), "feed_forward_norm": opt(self.feed_forward_norm)}
         if self.mixer_post_norm is not None:
             j["mixer_post_norm"] = self.mixer_post_norm.to_json()
         if self.feed_forward_post_norm is not None:
@@ -113,7 +113,7 @@ class ModelSpec:
         return cls(
             hidden_size=j["hidden_size"], vocab_size=j["vocab_size"], max_positions=j["max_positions"],
             embedding=P(j["embedding"]), final_norm=P(j["final_norm"]), head=P(j["head"]),
-            layers=[LayerSpec(l["block"], P(l["mixer"]), O(l.get("feed_forward")), P(l["mixer_norm"]), O(l.get("feed_forward_norm")),
+            layers=[LayerSpec(l["block"], P(l["mixer"]), O(l.get("feed_forward")), O(l.get("mixer_norm")), O(l.get("feed_forward_norm")),
                               O(l.get("mixer_post_norm")), O(l.get("feed_forward_post_norm")), O(l.get("token_input"))) for l in j["layers"]],
             schedule=[RunSpec(r["layer"], r.get("cache_from"), bool(r.get("reenter", False))) for r in j["schedule"]],
             reentry=O(j.get("reentry")),

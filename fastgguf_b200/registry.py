@@ -20,9 +20,11 @@ from .config.zirivik import ZirivikConfig
 from .config.salulorn import SalulornConfig
 from .config.pirozen import PirozenConfig
 from .config.saluzen import SaluzenConfig
+from .config.zifelorn import ZifelornConfig
 from .engine.spec import ModelSpec
 
-_CLASSES = {"LlamaForCausalLM": LlamaConfig, "Zirivik": ZirivikConfig, "Salulorn": SalulornConfig, "Pirozen": PirozenConfig, "Saluzen": SaluzenConfig}
+_CLASSES = {"LlamaForCausalLM": LlamaConfig, "Zirivik": ZirivikConfig, "Salulorn": SalulornConfig, "Pirozen": PirozenConfig, "Saluzen": SaluzenConfig,
+            "Zifelorn": ZifelornConfig}
 _keep_alive = []
 
 
