@@ -218,9 +218,28 @@ def saluzen_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_f
     return {"architecture": "Saluzen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
 
 
-DESIGNS = {"zirivik": zirivik_config, "salulorn": salulorn_config, "pirozen": pirozen_config, "saluzen": saluzen_config}
+def zifelorn_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff, blocks=2):
+    """Layers of a real model's sizes in the pattern of ``zirivik_config``: recurrent block + dense, recurrent block + experts,
+    latent attention + dense, latent attention on the layer before's latents + experts; `blocks` times.  The recurrent blocks have
+    as many channels as the stream, in parts of 256, and four taps."""
+    del kv_heads, window
+    lat = {"heads": heads, "dim": 64, "rot_dim": 64, "vdim": head_dim, "kv_rank": 512, "q_rank": width * 3 // 4, "scale": 128 ** -0.5,
+           "rot": {"base": 10000.0, "dims": 64}}
+    rec = {"width": width, "blocks": width // 256, "conv": 4}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": 8, "top": 2}}
+    layers = []
+    for _ in range(blocks):
+        at = len(layers) + 2
+        layers += [{"type": "rglru", "mixer": rec, "mlp": dense}, {"type": "rglru", "mixer": rec, "mlp": moe},
+                   {"type": "latent_attention", "mixer": lat, "mlp": dense}, {"type": "latent_attention", "mixer": dict(lat, kv_from=at), "mlp": moe}]
+    return {"architecture": "Zifelorn", "vocab": vocab, "width": width, "embedding": {"scale": width ** 0.5}, "norm": {"eps": 1e-6},
+            "logit_scale": 0.25, "layers": layers}
+
+
+DESIGNS = {"zifelorn": zifelorn_config, "zirivik": zirivik_config, "salulorn": salulorn_config, "pirozen": pirozen_config, "saluzen": saluzen_config}
 #: the model a design stands beside, where that is not Llama
-COUNTERPARTS = {"pirozen": ("zirivik", zirivik_attention_config), "saluzen": ("salulorn", salulorn_config)}
+COUNTERPARTS = {"pirozen": ("zirivik", zirivik_attention_config), "saluzen": ("salulorn", salulorn_config), "zifelorn": ("zirivik", zirivik_config)}
 
 #: name -> (width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff)
 COMPARE_SIZES = {"s": (2048, 32, 8, 64, 8192, 32768, 1024, 2048), "m": (4096, 32, 8, 128, 14336, 32768, 2048, 4096)}
@@ -315,6 +334,10 @@ def compare_designs(args):
                                   "state_space": "%d heads of 64 with 128 state rows, 4 taps" % (width // 64),
                                   "delta_rule": "%d heads of 128 x 128 on %d key heads, 4 taps" % (width // 128, max(1, width // 256)),
                                   "chunk": window, "beside": "Salulorn: gla, windowed attention, gla, latent attention"})
+        elif design == "zifelorn":
+            row["config"].update({"latent": "rank 512 + 64 rotated, queries through %d, every second layer on the layer before's latents" % (width * 3 // 4),
+                                  "recurrent": "%d channels in parts of 256, 4 taps" % width, "experts": "8 of ff %d, 2 a row" % eff,
+                                  "beside": "Zirivik: retention, retention, windowed attention, attention on the layer before's keys; dense and experts alike"})
         else:
             row["config"].update({"gla": "%d heads of 64 x 128" % (width // 128), "latent": "rank 512 + 64 rotated, queries through %d" % (width * 3 // 4),
                                   "convolution": "4 taps", "loop": "all layers, once"})
