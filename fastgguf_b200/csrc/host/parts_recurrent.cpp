@@ -461,7 +461,12 @@ public:
         in_ = Linear(concat_rows({y, x}, y.t.dtype == x.t.dtype ? y.t.dtype : FG_F32, rt.stream));
         o_ = Linear(tensor_of(tensors, "o_proj.weight"));
         in_b_ = f32_rows({flat(tensors, "y_proj.bias"), flat(tensors, "x_proj.bias")}, rt.stream);
-        conv_w_ = f32_rows({tensor_of(tensors, "conv.weight")}, rt.stream);
+        // [C, taps] -> [taps][C], so that neighbouring channels' weights of a tap lie side by side
+        const Weight cw = f32_rows({tensor_of(tensors, "conv.weight")}, rt.stream);
+        conv_w_ = make_weight(taps_, C_, FG_F32, "convolution weights of a recurrent block");
+        for (int t = 0; t < taps_; t++)
+            FG_CUDA(cudaMemcpy2DAsync(conv_w_.t.ptr<float>() + (size_t)t * C_, sizeof(float), cw.t.ptr<float>() + t, (size_t)taps_ * sizeof(float), sizeof(float),
+                                      (size_t)C_, cudaMemcpyDeviceToDevice, rt.stream));
         conv_b_ = f32_rows({tensor_of(tensors, "conv.bias")}, rt.stream);
         lam_ = f32_rows({tensor_of(tensors, "lam")}, rt.stream);
         // part by part: the rows of R, then those of I

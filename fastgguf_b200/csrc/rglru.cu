@@ -1,7 +1,8 @@
 // The real-gated linear recurrent unit and what stands between its projections and its output projection.
 //
 // A recurrent block has two branches of C channels, y and x (both out of one contraction, float32, without their biases):
-//     u = conv_b + causal convolution over time per channel of (x + x_bias)      weights [C, taps], zeros before the sequence
+//     u = conv_b + causal convolution over time per channel of (x + x_bias)      weights [taps][C], the last for the
+//                                                                                token itself; zeros before the sequence
 //     r = sigmoid(R u + r_bias), i = sigmoid(I u + i_bias)                       R, I block diagonal: `blocks` squares of C / blocks
 //     log a = -gain r softplus(lam);  S_t = a S_(t-1) + sqrt(1 - a^2) i u;       out = S gelu_tanh(y + y_bias)
 // Everything here is 32-bit in every engine dtype; only out takes the engine's.
@@ -26,25 +27,67 @@
 #define SCAN_MAX_CLUSTER 8
 #define STEP_ROWS 8                   // rows (sequences) a block of the single-token kernel serves
 #define STEP_CHANNELS 16              // channels it finishes, two a warp
-#define CONV_ROWS 8                   // rows a thread of the convolution walks
+#define CONV_ROWS 8                   // rows a thread of the convolution takes
 
-__device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// exponential, division and square root on the special-function unit (each within 2 ulp, the exponential's argument rounded once)
+__device__ __forceinline__ float rg_sigmoid(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float rg_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float rg_gelu(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float rg_gelu(float z) { return z * rg_sigmoid(1.5957691216f * fmaf(0.044715f * z * z, z, z)); }   // 0.5 (1 + tanh(y)) = sigmoid(2 y)
+__device__ __forceinline__ float rg_sqrt(float x) {
+    float r;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
 // a and the input term of one token: rate = gain * softplus(lam)
 __device__ __forceinline__ void rg_coefficients(float zr, float zi, float u, float rate, float &a, float &b) {
     const float log_a = -rate * rg_sigmoid(zr);
-    a = expf(log_a);
-    b = sqrtf(-expm1f(2.0f * log_a)) * (rg_sigmoid(zi) * u);      // 1 - a^2 without cancellation where a is close to 1
+    a = __expf(log_a);
+    // 1 - a^2 = 1 - e^x, x = 2 log a <= 0: where a is close to one the series -x (1 + x/2 + x^2/6 + ...), so that nothing cancels
+    // (|x| < 1/4: the first term left out is below 2e-8 of the sum), else the difference
+    const float x = 2.0f * log_a;
+    float p = fmaf(x, 1.0f / 5040.0f, 1.0f / 720.0f);
+    p = fmaf(x, p, 1.0f / 120.0f);
+    p = fmaf(x, p, 1.0f / 24.0f);
+    p = fmaf(x, p, 1.0f / 6.0f);
+    p = fmaf(x, p, 0.5f);
+    p = fmaf(x, p, 1.0f);
+    const float rest = x > -0.25f ? -x * p : fmaf(-a, a, 1.0f);
+    b = rg_sqrt(rest) * (rg_sigmoid(zi) * u);
 }
 
 // ------------------------------------------------------------------ convolution, prompts and portions
-// NC neighbouring channels a thread.  pieces (optional): [part][row][3][size of a part] bfloat16, see above.  tiles (optional): the
-// table of the grouped contraction that reads them - for each part, for each tile along its outputs, its rows in runs of 128.
-template <int NC>
+// NC neighbouring channels (1 or 4) and CONV_ROWS rows a thread; TAPS > 0: that many, 0: `taps`.  Rows whose taps all lie in this
+// step are the common case: a thread's inputs are then fetched once, together.  pieces (optional): [part][row][3][size of a
+// part] bfloat16, see above.  tiles (optional): the table of the grouped contraction that reads them - for each part, for each tile
+// along its outputs, its rows in runs of 128.
+template <int NC> struct RgVec { float v[NC]; };
+template <int NC> __device__ __forceinline__ RgVec<NC> rg_load(const float *p) {
+    RgVec<NC> r;
+    if (NC == 4) { const float4 t = *(const float4 *)p; r.v[0] = t.x; r.v[NC > 1 ? 1 : 0] = t.y; r.v[NC > 2 ? 2 : 0] = t.z; r.v[NC > 3 ? 3 : 0] = t.w; }
+    else r.v[0] = *p;
+    return r;
+}
+template <int NC> __device__ __forceinline__ void rg_store_conv(const RgVec<NC> &acc, float *u, bf16 *dst, int part) {
+    if (NC == 4) *(float4 *)u = make_float4(acc.v[0], acc.v[NC > 1 ? 1 : 0], acc.v[NC > 2 ? 2 : 0], acc.v[NC > 3 ? 3 : 0]);
+    else *u = acc.v[0];
+    if (!dst) return;
+    float rest[NC];
+#pragma unroll
+    for (int q = 0; q < NC; q++) rest[q] = acc.v[q];
+#pragma unroll
+    for (int e = 0; e < 3; e++, dst += part) {
+        __align__(8) bf16 h[NC];
+#pragma unroll
+        for (int q = 0; q < NC; q++) { h[q] = __float2bfloat16_rn(rest[q]); rest[q] -= __bfloat162float(h[q]); }
+        if (NC == 4) *(uint2 *)dst = *(const uint2 *)h;
+        else dst[0] = h[0];
+    }
+}
+
+template <int NC, int TAPS>
 __global__ void __launch_bounds__(256)
 rglru_conv_kernel(const float *__restrict__ x, int ld, const float *__restrict__ x_bias, const float *__restrict__ w,
-                  const float *__restrict__ conv_b, int taps, const float *__restrict__ state, long long state_stride,
+                  const float *__restrict__ conv_b, int taps_, const float *__restrict__ state, long long state_stride,
                   const int *__restrict__ positions, const int *__restrict__ row_seq, const int *__restrict__ cu_rows,
                   const int *__restrict__ slots, float *__restrict__ u, int ldu, bf16 *__restrict__ pieces, int4 *__restrict__ tiles,
                   int n_tiles, int tiles_n, int M, int C, int part) {
@@ -56,48 +99,54 @@ rglru_conv_kernel(const float *__restrict__ x, int ld, const float *__restrict__
             tiles[t] = make_int4(b * M + rt * 128, (b + 1) * M, b * 2 * part, qt);
         }
     }
+    const int taps = TAPS > 0 ? TAPS : taps_;
     const int c = (blockIdx.y * 256 + threadIdx.x) * NC;
     if (c >= C) return;
-    float xb[NC], cb[NC];
+    const RgVec<NC> xb = rg_load<NC>(x_bias + c), cb = rg_load<NC>(conv_b + c);
+    const int p = c / part, j0 = c - p * part;               // (a part is a multiple of NC)
+    const int m0 = blockIdx.x * CONV_ROWS, m1 = min(M, m0 + CONV_ROWS);
+    bf16 *dst0 = pieces ? pieces + ((size_t)p * M) * 3 * part + j0 : nullptr;
+    if (TAPS > 0 && m1 - m0 == CONV_ROWS) {
+        const int s = row_seq[m0];
+        if (cu_rows[s] + TAPS - 1 <= m0 && row_seq[m1 - 1] == s) {
+            RgVec<NC> in[CONV_ROWS + (TAPS > 0 ? TAPS : 1) - 1], wt[TAPS > 0 ? TAPS : 1];
 #pragma unroll
-    for (int q = 0; q < NC; q++) { xb[q] = x_bias[c + q]; cb[q] = conv_b[c + q]; }
-    const int p = c / part, j0 = c - p * part;               // (NC channels of one part: a part is a multiple of NC)
-    for (int m = blockIdx.x * CONV_ROWS; m < min(M, (int)(blockIdx.x + 1) * CONV_ROWS); m++) {
+            for (int i = 0; i < CONV_ROWS + TAPS - 1; i++) in[i] = rg_load<NC>(x + (size_t)(m0 - (TAPS - 1) + i) * ld + c);
+#pragma unroll
+            for (int t = 0; t < TAPS; t++) wt[t] = rg_load<NC>(w + (size_t)t * C + c);
+#pragma unroll
+            for (int i = 0; i < CONV_ROWS + TAPS - 1; i++)
+#pragma unroll
+                for (int q = 0; q < NC; q++) in[i].v[q] += xb.v[q];
+#pragma unroll
+            for (int i = 0; i < CONV_ROWS; i++) {
+                RgVec<NC> acc = cb;
+#pragma unroll
+                for (int t = 0; t < TAPS; t++)
+#pragma unroll
+                    for (int q = 0; q < NC; q++) acc.v[q] = fmaf(wt[t].v[q], in[i + t].v[q], acc.v[q]);
+                rg_store_conv<NC>(acc, u + (size_t)(m0 + i) * ldu + c, dst0 ? dst0 + (size_t)(m0 + i) * 3 * part : nullptr, part);
+            }
+            return;
+        }
+    }
+    for (int m = m0; m < m1; m++) {
         const int s = row_seq[m], i = m - cu_rows[s], pos = positions[m];
         const float *ring = state + (size_t)slots[s] * state_stride;
-        float acc[NC];
-#pragma unroll
-        for (int q = 0; q < NC; q++) acc[q] = cb[q];
+        RgVec<NC> acc = cb;
         for (int back = taps - 1; back >= 0; back--) {
-            float v[NC];
+            RgVec<NC> v;
             if (back <= i) {
-                const float *src = x + (size_t)(m - back) * ld + c;
+                v = rg_load<NC>(x + (size_t)(m - back) * ld + c);
 #pragma unroll
-                for (int q = 0; q < NC; q++) v[q] = src[q] + xb[q];
-            } else if (pos - back >= 0) {
-                const float *src = ring + (size_t)((pos - back) % taps) * C + c;
+                for (int q = 0; q < NC; q++) v.v[q] += xb.v[q];
+            } else if (pos - back >= 0) v = rg_load<NC>(ring + (size_t)((pos - back) % taps) * C + c);
+            else continue;
+            const RgVec<NC> wt = rg_load<NC>(w + (size_t)(taps - 1 - back) * C + c);
 #pragma unroll
-                for (int q = 0; q < NC; q++) v[q] = src[q];
-            } else continue;
-#pragma unroll
-            for (int q = 0; q < NC; q++) acc[q] = fmaf(w[(size_t)(c + q) * taps + taps - 1 - back], v[q], acc[q]);
+            for (int q = 0; q < NC; q++) acc.v[q] = fmaf(wt.v[q], v.v[q], acc.v[q]);
         }
-        if (NC == 2) *(float2 *)(u + (size_t)m * ldu + c) = make_float2(acc[0], acc[NC - 1]);
-        else u[(size_t)m * ldu + c] = acc[0];
-        if (pieces) {
-            bf16 *dst = pieces + ((size_t)p * M + m) * 3 * part + j0;
-            float rest[NC];
-#pragma unroll
-            for (int q = 0; q < NC; q++) rest[q] = acc[q];
-#pragma unroll
-            for (int e = 0; e < 3; e++, dst += part) {
-                bf16 h[NC];
-#pragma unroll
-                for (int q = 0; q < NC; q++) { h[q] = __float2bfloat16_rn(rest[q]); rest[q] -= __bfloat162float(h[q]); }
-                if (NC == 2) { __nv_bfloat162 two; two.x = h[0]; two.y = h[NC - 1]; *(__nv_bfloat162 *)dst = two; }
-                else dst[0] = h[0];
-            }
-        }
+        rg_store_conv<NC>(acc, u + (size_t)m * ldu + c, dst0 ? dst0 + (size_t)m * 3 * part : nullptr, part);
     }
 }
 
@@ -220,10 +269,10 @@ rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restri
                   const float *__restrict__ conv_b, int taps, const TW *__restrict__ W, const float *__restrict__ gate_bias,
                   const float *__restrict__ lam, float gain, const int *__restrict__ positions, const int *__restrict__ row_seq,
                   const int *__restrict__ slots, float *__restrict__ state, long long state_stride, TO *__restrict__ out, int ldo, int M, int C,
-                  int part, int stride, int vec) {
+                  int part, int stride, int vec, int vec4) {
     extern __shared__ __align__(16) float us[];                 // [STEP_ROWS][stride] u of the part
     constexpr int VEC = 16 / (int)sizeof(TW);
-    const int p = blockIdx.y, tid = threadIdx.x, warp = warp_index(), lane = tid & 31;
+    const int p = blockIdx.y, warp = warp_index(), lane = threadIdx.x & 31;
     const int j0 = blockIdx.x * STEP_CHANNELS + warp * 2;       // the warp's channels j0, j0 + 1 of the part
     // the warp's four rows: R of both channels, then I of both (channels beyond the part repeat its last one and are not stored)
     const TW *wr[4];
@@ -235,23 +284,62 @@ rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restri
 #pragma unroll
         for (int q = 0; q < 4; q++) w4[q] = *(const uint4 *)(wr[q] + lane * VEC);
     }
+    // what the lanes that finish a (channel, row) need besides the sums: asked for early, used at the end
+    const int jf = j0 + ((lane >> 3) & 1), mf = blockIdx.z * STEP_ROWS + (lane & 7), cf = p * part + min(jf, part - 1);
+    const bool finish = lane < 16 && jf < part && mf < M;
+    const float br = gate_bias[(size_t)p * 2 * part + min(jf, part - 1)], bi = gate_bias[(size_t)p * 2 * part + part + min(jf, part - 1)];
+    const float lam_c = lam[cf], yb = proj_bias[cf];
     pdl_launch_dependents_small_step(M);
     pdl_wait();
-    const int m0 = blockIdx.z * STEP_ROWS;
-    for (int e = tid; e < STEP_ROWS * stride; e += 256) {
-        const int row = e / stride, j = e - row * stride, m = m0 + row;
-        float acc = 0.f;
-        if (m < M && j < part) {
-            const int c = p * part + j, pos = positions[m];
+    float *Sg = nullptr;
+    float S0 = 0.f, y0 = 0.f;
+    if (finish) {
+        y0 = proj[(size_t)mf * ldp + cf];
+        Sg = state + (size_t)slots[row_seq[mf]] * state_stride + (taps > 1 ? (size_t)taps * C : 0) + cf;
+        S0 = *Sg;
+    }
+    {
+        // u of the part: warp w the row m0 + w, its lanes NC channels at a time
+        const int m = blockIdx.z * STEP_ROWS + warp;
+        float *urow = us + warp * stride;
+        if (m < M) {
+            const int pos = positions[m];
             float *ring = state + (size_t)slots[row_seq[m]] * state_stride;
-            const float now = proj[(size_t)m * ldp + C + c] + proj_bias[C + c];
-            acc = conv_b[c];
-            for (int back = taps - 1; back > 0; back--)
-                if (pos - back >= 0) acc = fmaf(conv_w[(size_t)c * taps + taps - 1 - back], ring[(size_t)((pos - back) % taps) * C + c], acc);
-            acc = fmaf(conv_w[(size_t)c * taps + taps - 1], now, acc);
-            if (taps > 1 && j / STEP_CHANNELS == blockIdx.x) ring[(size_t)(pos % taps) * C + c] = now;
+            const float *now = proj + (size_t)m * ldp + C;
+            if (vec4) {
+                for (int j = lane * 4; j < part; j += 128) {
+                    const int c = p * part + j;
+                    RgVec<4> acc = rg_load<4>(conv_b + c), cur = rg_load<4>(now + c);
+                    const RgVec<4> xb = rg_load<4>(proj_bias + C + c), wl = rg_load<4>(conv_w + (size_t)(taps - 1) * C + c);
+#pragma unroll
+                    for (int q = 0; q < 4; q++) cur.v[q] += xb.v[q];
+#pragma unroll 4
+                    for (int back = 1; back < taps; back++) {
+                        if (pos - back < 0) break;
+                        const RgVec<4> old = rg_load<4>(ring + (size_t)((pos - back) % taps) * C + c), wt = rg_load<4>(conv_w + (size_t)(taps - 1 - back) * C + c);
+#pragma unroll
+                        for (int q = 0; q < 4; q++) acc.v[q] = fmaf(wt.v[q], old.v[q], acc.v[q]);
+                    }
+#pragma unroll
+                    for (int q = 0; q < 4; q++) acc.v[q] = fmaf(wl.v[q], cur.v[q], acc.v[q]);
+                    *(float4 *)(urow + j) = make_float4(acc.v[0], acc.v[1], acc.v[2], acc.v[3]);
+                    if (taps > 1 && j / STEP_CHANNELS == blockIdx.x)
+                        *(float4 *)(ring + (size_t)(pos % taps) * C + c) = make_float4(cur.v[0], cur.v[1], cur.v[2], cur.v[3]);
+                }
+            } else {
+                for (int j = lane; j < part; j += 32) {
+                    const int c = p * part + j;
+                    const float cur = now[c] + proj_bias[C + c];
+                    float acc = conv_b[c];
+                    for (int back = 1; back < taps; back++)
+                        if (pos - back >= 0) acc = fmaf(conv_w[(size_t)(taps - 1 - back) * C + c], ring[(size_t)((pos - back) % taps) * C + c], acc);
+                    urow[j] = fmaf(conv_w[(size_t)(taps - 1) * C + c], cur, acc);
+                    if (taps > 1 && j / STEP_CHANNELS == blockIdx.x) ring[(size_t)(pos % taps) * C + c] = cur;
+                }
+            }
+        } else {
+            for (int j = lane; j < part; j += 32) urow[j] = 0.f;
         }
-        us[e] = acc;
     }
     __syncthreads();
     float v[4 * STEP_ROWS];                                      // [row of W][row of the step]
@@ -299,16 +387,12 @@ rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restri
         }
     }
     const float zi = __shfl_xor_sync(0xffffffffu, v[0], 16);     // lanes 0 .. 15: R u of (channel lane / 8, row lane % 8); I u from lane + 16
-    const int j = j0 + ((lane >> 3) & 1), row = lane & 7, m = m0 + row;
-    if (lane >= 16 || j >= part || m >= M) return;
-    const int c = p * part + j;
+    if (!finish) return;
     float a, b;
-    rg_coefficients(v[0] + gate_bias[(size_t)p * 2 * part + j], zi + gate_bias[(size_t)p * 2 * part + part + j], us[row * stride + j],
-                    gain * rg_softplus(lam[c]), a, b);
-    float *Sg = state + (size_t)slots[row_seq[m]] * state_stride + (taps > 1 ? (size_t)taps * C : 0);
-    const float S = fmaf(a, Sg[c], b);
-    Sg[c] = S;
-    out[(size_t)m * ldo + c] = from_f32<TO>(S * rg_gelu(proj[(size_t)m * ldp + c] + proj_bias[c]));
+    rg_coefficients(v[0] + br, zi + bi, us[(lane & 7) * stride + jf], gain * rg_softplus(lam_c), a, b);
+    const float S = fmaf(a, S0, b);
+    *Sg = S;
+    out[(size_t)mf * ldo + cf] = from_f32<TO>(S * rg_gelu(y0 + yb));
 }
 
 // ------------------------------------------------------------------ launchers
@@ -325,13 +409,21 @@ extern "C" int fg_rglru_conv(const float *proj, int ldp, const float *proj_bias,
                              const int *slots, float *u, int ldu, void *pieces, void *tiles, int bn, int M, int C, int part, cudaStream_t stream) {
     if (M <= 0) return 0;
     if (C <= 0 || part <= 0 || C % part || taps <= 0 || (pieces && (!tiles || bn <= 0))) return FG_ERR_BAD_SIZE;
-    const bool two = part % 2 == 0 && ldu % 2 == 0 && (((uintptr_t)u) & 7) == 0 && (((uintptr_t)pieces) & 3) == 0;
+    const bool four = part % 4 == 0 && ldp % 4 == 0 && ldu % 4 == 0 &&
+                      ((((uintptr_t)proj) | ((uintptr_t)proj_bias) | ((uintptr_t)conv_w) | ((uintptr_t)conv_b) | ((uintptr_t)u)) & 15) == 0 &&
+                      (((uintptr_t)pieces) & 7) == 0 && (((uintptr_t)state) & 15) == 0 && state_stride % 4 == 0;
     const int n_tiles = pieces ? fg_rglru_tiles(M, C, part, bn) : 0, tiles_n = pieces ? (2 * part + bn - 1) / bn : 0;
-    const int per = two ? 512 : 256;
+    const int per = four ? 1024 : 256;
     const dim3 grid((M + CONV_ROWS - 1) / CONV_ROWS, (C + per - 1) / per);
-#define RG_CONV(NC) fg_launch(rglru_conv_kernel<NC>, grid, dim3(256), 0, stream, proj + C, ldp, proj_bias + C, conv_w, conv_b, taps, state, state_stride, \
-                              positions, row_seq, cu_rows, slots, u, ldu, (bf16 *)pieces, (int4 *)tiles, n_tiles, tiles_n, M, C, part)
-    return two ? RG_CONV(2) : RG_CONV(1);
+#define RG_CONV(NC, TAPS) fg_launch(rglru_conv_kernel<NC, TAPS>, grid, dim3(256), 0, stream, proj + C, ldp, proj_bias + C, conv_w, conv_b, taps, state, \
+                                    state_stride, positions, row_seq, cu_rows, slots, u, ldu, (bf16 *)pieces, (int4 *)tiles, n_tiles, tiles_n, M, C, part)
+    if (!four) return RG_CONV(1, 0);
+    switch (taps) {
+    case 2: return RG_CONV(4, 2);
+    case 3: return RG_CONV(4, 3);
+    case 4: return RG_CONV(4, 4);
+    default: return RG_CONV(4, 0);
+    }
 #undef RG_CONV
 }
 
@@ -368,9 +460,11 @@ static int rglru_step_launch(const float *proj, int ldp, const float *proj_bias,
         if (e != cudaSuccess) return (int)e;
     }
     const int stride = (part + 3) / 4 * 4, vec = part % (16 / (int)sizeof(TW)) == 0 && (((uintptr_t)W) & 15) == 0;
+    const int vec4 = part % 4 == 0 && ldp % 4 == 0 && state_stride % 4 == 0 &&
+                     ((((uintptr_t)proj) | ((uintptr_t)proj_bias) | ((uintptr_t)conv_w) | ((uintptr_t)conv_b) | ((uintptr_t)state)) & 15) == 0;
     const dim3 grid((part + STEP_CHANNELS - 1) / STEP_CHANNELS, C / part, (M + STEP_ROWS - 1) / STEP_ROWS);
     return fg_launch(rglru_step_kernel<TW, TO>, grid, dim3(256), (size_t)STEP_ROWS * stride * sizeof(float), stream, proj, ldp, proj_bias, conv_w,
-                     conv_b, taps, (const TW *)W, gate_bias, lam, gain, positions, row_seq, slots, state, state_stride, (TO *)out, ldo, M, C, part, stride, vec);
+                     conv_b, taps, (const TW *)W, gate_bias, lam, gain, positions, row_seq, slots, state, state_stride, (TO *)out, ldo, M, C, part, stride, vec, vec4);
 }
 
 // A step of single tokens (one row a sequence).  W: [C / part][2 * part][part] in w_dtype.
