@@ -20,6 +20,7 @@
 
 #define LAT_WARPS 8
 #define LAT_HG 8                      // heads a block serves
+#define LAT_MAX_SPLITS 32
 
 // four consecutive numbers of a cache row
 __device__ __forceinline__ void load4(const float *p, float (&v)[4]) { const float4 t = *(const float4 *)p; v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w; }
@@ -164,15 +165,29 @@ latent_decode_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, int 
 
 // ---------------------------------------------------------------------------------------------- the same on the tensor cores
 // bfloat16, pages of 64 positions, R a multiple of 64, DR a multiple of 16.  One block per (row, 16 heads, split of the
-// PAGES); per page: (1) S = Q K^T, warp w the page's keys 8 w .. 8 w + 7 as m16n8k16 MMAs whose B operand - a key's numbers
-// along k - is read straight from the cache rows; (2) the scores meet in shared memory, warp w runs the online softmax of
-// rows 2 w and 2 w + 1 (running maximum and sum per row in shared memory) and leaves bfloat16 weights there; (3) O += P V,
-// warp w the latent's columns w R / 8 .. , the B operand - two keys of one column - packed from 16-bit reads of the cache rows.
+// PAGES).  A page's rows [latent | rotated part] come to shared memory in 16-byte asynchronous copies, all of them in flight at
+// once (rows padded so that the eight rows of a matrix load hit different banks); with two buffers the next page travels while
+// this one is worked on.  Per page: (1) S = Q K^T, warp w the page's keys 8 w .. 8 w + 7 as m16n8k16 MMAs; (2) the scores meet in
+// shared memory, warp w runs the online softmax of rows 2 w and 2 w + 1 (running maximum and sum per row in shared memory) and
+// leaves bfloat16 weights there; (3) O += P V, warp w the latent's columns w R / 8 .. , the B operand - two keys of one column -
+// by transposed matrix loads of the same rows.
 #define LM_WARPS 8
 #define LM_HEADS 16
 __device__ __forceinline__ void lat_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+// four 8 x 8 matrices of 16-bit numbers; lane l gives the address of row l % 8 of matrix l / 8
+__device__ __forceinline__ void lat_ldm4(uint32_t (&v)[4], const bf16 *p) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void lat_ldm4_trans(uint32_t (&v)[4], const bf16 *p) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void lat_copy16(bf16 *dst, const bf16 *src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
 template <int NT>                     // n-tiles of 8 latent columns a warp owns: R = 64 NT
@@ -180,7 +195,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32)
 latent_decode_mma_kernel(const bf16 *__restrict__ q, int ldq, bf16 *__restrict__ out, int ldo, const int *__restrict__ positions,
                          const int *__restrict__ row_seq, const int *__restrict__ block_table, int table_width, const bf16 *__restrict__ k_pool,
                          const bf16 *__restrict__ v_pool, int H, int DR, float scale_log2, const float *__restrict__ sinks, int n_splits,
-                         float *__restrict__ part) {
+                         float *__restrict__ part, int stages) {
     constexpr int R = 64 * NT, PG = 64;
     extern __shared__ __align__(16) uint8_t lm_smem[];
     pdl_launch_dependents();
@@ -191,10 +206,24 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, int ldq, bf16 *__restrict__
     const int QD = R + DR, QS = QD + 8, PS = PG + 8;
     bf16 *Qs = (bf16 *)lm_smem;                                   // [16][QS]
     bf16 *Ps = Qs + LM_HEADS * QS;                                // [16][PS]
-    float *Ss = (float *)(Ps + LM_HEADS * PS);                    // [16][PG + 1]
+    bf16 *Ks = Ps + LM_HEADS * PS;                                // [stages][PG][QS] the pages' rows
+    float *Ss = (float *)(Ks + (size_t)stages * PG * QS);         // [16][PG + 1]
     float *m_s = Ss + LM_HEADS * (PG + 1), *l_s = m_s + LM_HEADS, *corr_s = l_s + LM_HEADS;
     const int pos = positions[m_row];
     const int *bt = block_table + (size_t)row_seq[m_row] * table_width;
+    const int last_page = pos / PG, chunks = QD / 8;
+    auto fetch = [&](int pg, int stage) {
+        if (pg <= last_page) {
+            const size_t base = (size_t)bt[pg] * PG;
+            bf16 *dst = Ks + (size_t)stage * PG * QS;
+            for (int e = threadIdx.x; e < PG * chunks; e += LM_WARPS * 32) {
+                const int row = e / chunks, d = (e - row * chunks) * 8;
+                lat_copy16(dst + row * QS + d, d < R ? v_pool + (base + row) * R + d : k_pool + (base + row) * DR + (d - R));
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");      // (an empty group behind the last page)
+    };
+    fetch(split, 0);
     for (int e = threadIdx.x; e < LM_HEADS * QD; e += LM_WARPS * 32) {
         const int hh = e / QD, d = e - hh * QD;
         Qs[hh * QS + d] = hh < nh ? q[(size_t)m_row * ldq + (size_t)(h0 + hh) * QD + d] : __float2bfloat16_rn(0.f);
@@ -204,26 +233,39 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, int ldq, bf16 *__restrict__
         m_s[threadIdx.x] = sink ? sinks[h0 + threadIdx.x] * 1.4426950408889634f : -INFINITY;
         l_s[threadIdx.x] = sink ? 1.f : 0.f;
     }
-    __syncthreads();
     float o[NT][4];
 #pragma unroll
     for (int nt = 0; nt < NT; nt++) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-    const int last_page = pos / PG;
+    int stage = 0;
     for (int pg = split; pg <= last_page; pg += n_splits) {
-        const size_t base = (size_t)bt[pg] * PG;
+        if (stages > 1) {
+            fetch(pg + n_splits, stage ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                          // everybody's copies have landed
+        const bf16 *Kp = Ks + (size_t)stage * PG * QS;
         // (1) scores of this warp's eight keys
         {
-            const size_t at = base + 8 * warp + r;
-            const bf16 *lat = v_pool + at * R, *rot = k_pool + at * DR;
-            float c[4] = {0.f, 0.f, 0.f, 0.f};
+            const bf16 *qa = Qs + (lane & 15) * QS + (lane >> 4) * 8, *kb = Kp + (8 * warp + (lane & 7)) * QS + (lane >> 3) * 8;
+            float c[4] = {0.f, 0.f, 0.f, 0.f}, c2[4] = {0.f, 0.f, 0.f, 0.f};
+            int kc = 0;
 #pragma unroll 4
-            for (int kc = 0; kc < QD; kc += 16) {
-                const bf16 *qa = Qs + r * QS + kc + cp;
-                const uint32_t a0 = *(const uint32_t *)qa, a1 = *(const uint32_t *)(qa + 8 * QS), a2 = *(const uint32_t *)(qa + 8),
-                               a3 = *(const uint32_t *)(qa + 8 * QS + 8);
-                const bf16 *kb = (kc < R ? lat + kc : rot + (kc - R)) + cp;
-                lat_mma(c, a0, a1, a2, a3, *(const uint32_t *)kb, *(const uint32_t *)(kb + 8));
+            for (; kc + 32 <= QD; kc += 32) {
+                uint32_t a[4], a2[4], b[4];
+                lat_ldm4(a, qa + kc);
+                lat_ldm4(a2, qa + kc + 16);
+                lat_ldm4(b, kb + kc);
+                lat_mma(c, a[0], a[1], a[2], a[3], b[0], b[1]);
+                lat_mma(c2, a2[0], a2[1], a2[2], a2[3], b[2], b[3]);
             }
+            if (kc < QD) {                                        // one step of sixteen is left (lanes 16 .. 31 repeat addresses)
+                uint32_t a[4], b[4];
+                lat_ldm4(a, qa + kc);
+                lat_ldm4(b, Kp + (8 * warp + (lane & 7)) * QS + ((lane >> 3) & 1) * 8 + kc);
+                lat_mma(c, a[0], a[1], a[2], a[3], b[0], b[1]);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; e++) c[e] += c2[e];
             const int col = 8 * warp + cp, key = pg * PG + col;
             Ss[r * (PG + 1) + col] = key <= pos ? c[0] * scale_log2 : -INFINITY;
             Ss[r * (PG + 1) + col + 1] = key + 1 <= pos ? c[1] * scale_log2 : -INFINITY;
@@ -255,21 +297,27 @@ latent_decode_mma_kernel(const bf16 *__restrict__ q, int ldq, bf16 *__restrict__
             const float c0 = corr_s[r], c1 = corr_s[r + 8];
 #pragma unroll
             for (int nt = 0; nt < NT; nt++) { o[nt][0] *= c0; o[nt][1] *= c0; o[nt][2] *= c1; o[nt][3] *= c1; }
-            const unsigned short *V = (const unsigned short *)(v_pool + base * R);
+            const bf16 *pa = Ps + (lane & 15) * PS + (lane >> 4) * 8;
+            const bf16 *vb = Kp + (lane & 15) * QS + warp * (R / 8) + (lane >> 4) * 8;
 #pragma unroll
             for (int ks = 0; ks < PG; ks += 16) {
-                const bf16 *pa = Ps + r * PS + ks + cp;
-                const uint32_t a0 = *(const uint32_t *)pa, a1 = *(const uint32_t *)(pa + 8 * PS), a2 = *(const uint32_t *)(pa + 8),
-                               a3 = *(const uint32_t *)(pa + 8 * PS + 8);
+                uint32_t a[4];
+                lat_ldm4(a, pa + ks);
 #pragma unroll
-                for (int nt = 0; nt < NT; nt++) {
-                    const unsigned short *vb = V + (size_t)(ks + cp) * R + warp * (R / 8) + nt * 8 + r;
-                    const uint32_t b0 = (uint32_t)vb[0] | ((uint32_t)vb[R] << 16), b1 = (uint32_t)vb[8 * R] | ((uint32_t)vb[9 * R] << 16);
-                    lat_mma(o[nt], a0, a1, a2, a3, b0, b1);
+                for (int nt = 0; nt < NT; nt += 2) {
+                    // the sixteen keys' rows of columns 8 nt .. and 8 (nt + 1) .. (an odd last tile: its own columns twice)
+                    uint32_t b[4];
+                    lat_ldm4_trans(b, vb + ks * QS + nt * 8 - ((nt + 1 < NT) ? 0 : (lane >> 4) * 8));
+                    lat_mma(o[nt], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    if (nt + 1 < NT) lat_mma(o[nt + 1 < NT ? nt + 1 : nt], a[0], a[1], a[2], a[3], b[2], b[3]);
                 }
             }
         }
+        __syncthreads();                                          // the page's buffer and the weights are free again
+        if (stages > 1) stage ^= 1;
+        else fetch(pg + n_splits, 0);
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < 2; k++) {
@@ -297,19 +345,23 @@ template <typename T>
 __global__ void latent_merge_kernel(const float *__restrict__ part, T *__restrict__ out, int ldo, int H, int R, int n_splits) {
     pdl_launch_dependents();
     pdl_wait();
+    __shared__ float w_s[LAT_MAX_SPLITS], inv_l;
     const int m_row = blockIdx.y, h = blockIdx.x;
     const float *pr = part + ((size_t)m_row * H + h) * n_splits * (R + 2);
-    float M = -INFINITY;
-    for (int s = 0; s < n_splits; s++) M = fmaxf(M, pr[(size_t)s * (R + 2) + R]);
+    if (threadIdx.x < 32) {                                  // the splits' weights once; up to 32 splits, a lane each
+        const int lane = threadIdx.x;
+        const float m = lane < n_splits ? pr[(size_t)lane * (R + 2) + R] : -INFINITY, l = lane < n_splits ? pr[(size_t)lane * (R + 2) + R + 1] : 0.f;
+        const float M = warp_max(m), w = m == -INFINITY ? 0.f : lat_ex2(m - M);          // maxima are in the base-2 domain
+        const float L = warp_sum(l * w);
+        w_s[lane] = w;
+        if (lane == 0) inv_l = L > 0.f ? 1.0f / L : 0.f;
+    }
+    __syncthreads();
     for (int d = threadIdx.x; d < R; d += blockDim.x) {
-        float L = 0.f, O = 0.f;
-        for (int s = 0; s < n_splits; s++) {                 // split order
-            const float *src = pr + (size_t)s * (R + 2);
-            const float wgt = src[R] == -INFINITY ? 0.f : lat_ex2(src[R] - M);       // maxima are in the base-2 domain
-            L = fmaf(src[R + 1], wgt, L);
-            O = fmaf(src[d], wgt, O);
-        }
-        out[(size_t)m_row * ldo + (size_t)h * R + d] = from_f32<T>(L > 0.f ? O / L : 0.f);
+        float O = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < n_splits; s++) O = fmaf(pr[(size_t)s * (R + 2) + d], w_s[s], O);                  // split order
+        out[(size_t)m_row * ldo + (size_t)h * R + d] = from_f32<T>(O * inv_l);
     }
 }
 
@@ -410,7 +462,7 @@ extern "C" int fg_latent_decode(const void *q, int ldq, void *out, int ldo, int 
                                 const int *block_table, int table_width, const void *k_pool, const void *v_pool, int M, int H, int R,
                                 int DR, int page_size, float scale, const float *sinks, int n_splits, float *part, cudaStream_t stream) {
     if (M <= 0) return 0;
-    if (H <= 0 || R <= 0 || R > 512 || R % 4 || DR <= 0 || DR > 128 || DR % 4 || n_splits < 1 || M > 65535 || n_splits > 65535) return FG_ERR_BAD_SIZE;
+    if (H <= 0 || R <= 0 || R > 512 || R % 4 || DR <= 0 || DR > 128 || DR % 4 || n_splits < 1 || M > 65535 || n_splits > LAT_MAX_SPLITS) return FG_ERR_BAD_SIZE;
     if (((uintptr_t)k_pool | (uintptr_t)v_pool) & 15) return FG_ERR_BAD_SIZE;
     if (n_splits > 1 && !part) return FG_ERR_BAD_SIZE;
     if (latent_smem(R, DR) > 200 * 1024) return FG_ERR_BAD_SIZE;
@@ -425,28 +477,35 @@ extern "C" int fg_latent_decode(const void *q, int ldq, void *out, int ldo, int 
     return FG_ERR_BAD_DTYPE;
 }
 
-static size_t latent_mma_smem(int R, int DR) {
-    return (size_t)LM_HEADS * (R + DR + 8) * 2 + (size_t)LM_HEADS * (64 + 8) * 2 + (size_t)LM_HEADS * 65 * 4 + 3 * LM_HEADS * 4;
+static size_t latent_mma_smem(int R, int DR, int stages) {
+    return (size_t)(LM_HEADS + stages * 64) * (R + DR + 8) * 2 + (size_t)LM_HEADS * (64 + 8) * 2 + (size_t)LM_HEADS * 65 * 4 + 3 * LM_HEADS * 4;
 }
 
 // 1 if the tensor-core form takes these sizes (bfloat16 only)
-extern "C" int fg_latent_decode_mma_ok(int R, int DR, int page_size) { return page_size == 64 && R % 64 == 0 && R >= 64 && R <= 512 && DR % 16 == 0 && DR > 0; }
+extern "C" int fg_latent_decode_mma_ok(int R, int DR, int page_size) { return page_size == 64 && R % 64 == 0 && R >= 64 && R <= 512 && DR % 16 == 0 && DR > 0 && latent_mma_smem(R, DR, 1) <= 224 * 1024; }
 
 // q: [M, H * (R + DR)], out: [M, H * R] bfloat16; n_splits over the PAGES of a sequence; part as for fg_latent_decode
 extern "C" int fg_latent_decode_mma(const void *q, int ldq, void *out, int ldo, const int *positions, const int *row_seq,
                                     const int *block_table, int table_width, const void *k_pool, const void *v_pool, int M, int H, int R,
                                     int DR, int page_size, float scale, const float *sinks, int n_splits, float *part, cudaStream_t stream) {
     if (M <= 0) return 0;
-    if (!fg_latent_decode_mma_ok(R, DR, page_size) || H <= 0 || n_splits < 1 || M > 65535 || n_splits > 65535) return FG_ERR_BAD_SIZE;
-    if ((n_splits > 1 && !part) || ldq % 2 || ldo % 2 || ((uintptr_t)q & 3) || ((uintptr_t)out & 3) || ((uintptr_t)k_pool & 3) || ((uintptr_t)v_pool & 3))
+    if (!fg_latent_decode_mma_ok(R, DR, page_size) || H <= 0 || n_splits < 1 || M > 65535 || n_splits > LAT_MAX_SPLITS) return FG_ERR_BAD_SIZE;
+    if ((n_splits > 1 && !part) || ldq % 2 || ldo % 2 || ((uintptr_t)q & 3) || ((uintptr_t)out & 3) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15))
         return FG_ERR_BAD_SIZE;
-    const size_t smem = latent_mma_smem(R, DR);
+    // two buffers where a block has several pages to walk and they fit an SM
+    const int stages = (long long)table_width > n_splits && latent_mma_smem(R, DR, 2) <= 224 * 1024 ? 2 : 1;
+    const size_t smem = latent_mma_smem(R, DR, stages);
     const dim3 grid((H + LM_HEADS - 1) / LM_HEADS, M, n_splits);
     const float scale_log2 = scale * 1.4426950408889634f;
     int code = FG_ERR_BAD_SIZE;
-#define LM_RUN(NT) code = fg_launch(latent_decode_mma_kernel<NT>, grid, dim3(LM_WARPS * 32), smem, stream, (const bf16 *)q, ldq, (bf16 *)out, ldo, \
+#define LM_RUN(NT)                                                                                                                       \
+    {                                                                                                                                    \
+        static FgPerDevice setup;                                                                                                        \
+        if (fg_needs_setup(setup)) cudaFuncSetAttribute(latent_decode_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024); \
+    }                                                                                                                                    \
+    code = fg_launch(latent_decode_mma_kernel<NT>, grid, dim3(LM_WARPS * 32), smem, stream, (const bf16 *)q, ldq, (bf16 *)out, ldo, \
                                     positions, row_seq, block_table, table_width, (const bf16 *)k_pool, (const bf16 *)v_pool, H, DR, scale_log2, sinks, \
-                                    n_splits, part)
+                                    n_splits, part, stages)
     switch (R / 64) {
         case 1: LM_RUN(1); break; case 2: LM_RUN(2); break; case 3: LM_RUN(3); break; case 4: LM_RUN(4); break;
         case 5: LM_RUN(5); break; case 6: LM_RUN(6); break; case 7: LM_RUN(7); break; case 8: LM_RUN(8); break;

@@ -239,70 +239,133 @@ head_gemm_kernel(const void *__restrict__ A, int a_dtype, int lda, int a_stride,
         }
 }
 
-// The same contraction for a few rows (a decode step): every weight is read once, 16-byte or coalesced, for all rows.
-// TRANSPOSED: a thread per output n (a stored row runs along n, so neighbouring threads read neighbouring numbers), sums along
-// k in order; else a warp per output n with its lanes along k (a stored row runs along k) and a shuffle tree at the end.
+// The same contraction for a few rows (a decode step): every weight is read once, in 16-byte or paired accesses, for all rows.
+// TRANSPOSED (a stored row runs along n): a thread owns two neighbouring outputs and, for bfloat16 weights, a quarter of the sum
+// over k, the four quarters being added in order in shared memory; for float32 weights the whole sum in order, as the tiled
+// kernel adds it.  Else (a stored row runs along k): a warp owns two outputs, its lanes lie along
+// k, and the sums meet in a shuffle tree.  RM: rows the registers hold (M <= RM).  vec: the sizes allow the wide accesses.
 #define HV_ROWS 16
-template <bool TRANSPOSED>
+#define HV_COLS 128                                     // outputs of 64 threads, transposed
+template <typename TW> struct HvPair;
+template <> struct HvPair<float> { static __device__ __forceinline__ float2 load(const float *p) { return *(const float2 *)p; } };
+template <> struct HvPair<bf16> { static __device__ __forceinline__ float2 load(const bf16 *p) { return __bfloat1622float2(*(const __nv_bfloat162 *)p); } };
+
+template <typename TW, bool TRANSPOSED, int RM>
 __global__ void __launch_bounds__(256)
-head_gemv_kernel(const void *__restrict__ A, int a_dtype, int lda, int a_stride, const void *__restrict__ W, int w_dtype, int ldw,
-                 void *__restrict__ Cm, int c_dtype, int ldc, int c_stride, const float *__restrict__ gate, int ldg, int M, int N, int K) {
-    extern __shared__ float as[];                       // [M][K]
+head_gemv_kernel(const void *__restrict__ A, int a_dtype, int lda, int a_stride, const TW *__restrict__ W, int ldw,
+                 void *__restrict__ Cm, int c_dtype, int ldc, int c_stride, const float *__restrict__ gate, int ldg, int M, int N, int K,
+                 int vec) {
+    extern __shared__ __align__(16) float as[];         // transposed: [K][RM], then the quarters' sums; else [RM][KP]
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.y;
-    for (int e = threadIdx.x; e < M * K; e += 256) {
+    const int h = blockIdx.y, tid = threadIdx.x, KP = (K + 3) / 4 * 4;
+    for (int e = tid; e < RM * K; e += 256) {
         const int m = e / K, k = e - m * K;
-        as[e] = load_as(A, a_dtype, (size_t)m * lda + (size_t)h * a_stride + k);
+        as[TRANSPOSED ? k * RM + m : m * KP + k] = m < M ? load_as(A, a_dtype, (size_t)m * lda + (size_t)h * a_stride + k) : 0.f;
     }
     __syncthreads();
-    float acc[HV_ROWS];
+    float acc[2][RM];
 #pragma unroll
-    for (int m = 0; m < HV_ROWS; m++) acc[m] = 0.f;
-    int n;
-    if (TRANSPOSED) {
-        n = blockIdx.x * 256 + threadIdx.x;
-        if (n >= N) return;
-        // sixteen weights are on their way before the first of them is used
-        for (int k0 = 0; k0 < K; k0 += 16) {
-            float w[16];
-#pragma unroll
-            for (int u = 0; u < 16; u++) w[u] = k0 + u < K ? load_as(W, w_dtype, ((size_t)h * K + k0 + u) * ldw + n) : 0.f;
-#pragma unroll
-            for (int u = 0; u < 16; u++) {
-                if (k0 + u >= K) break;
-#pragma unroll
-                for (int m = 0; m < HV_ROWS; m++)
-                    if (m < M) acc[m] = fmaf(as[m * K + k0 + u], w[u], acc[m]);
-            }
-        }
-    } else {
-        const int lane = threadIdx.x & 31;
-        n = blockIdx.x * 8 + (threadIdx.x >> 5);
-        if (n >= N) return;
-        for (int k0 = lane; k0 < K; k0 += 256) {
-            float w[8];
-#pragma unroll
-            for (int u = 0; u < 8; u++) w[u] = k0 + 32 * u < K ? load_as(W, w_dtype, ((size_t)h * N + n) * ldw + k0 + 32 * u) : 0.f;
-#pragma unroll
-            for (int u = 0; u < 8; u++) {
-                if (k0 + 32 * u >= K) break;
-#pragma unroll
-                for (int m = 0; m < HV_ROWS; m++)
-                    if (m < M) acc[m] = fmaf(as[m * K + k0 + 32 * u], w[u], acc[m]);
-            }
-        }
-#pragma unroll
-        for (int m = 0; m < HV_ROWS; m++)
-            if (m < M) acc[m] = warp_sum(acc[m]);
-        if (lane != 0) return;
-    }
-#pragma unroll
-    for (int m = 0; m < HV_ROWS; m++) {
-        if (m >= M) break;
-        float v = acc[m];
+    for (int m = 0; m < RM; m++) acc[0][m] = acc[1][m] = 0.f;
+    auto store = [&](int m, int n, float v) {
         if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)m * ldg + (size_t)h * N + n]));
         store_as(Cm, c_dtype, (size_t)m * ldc + (size_t)h * c_stride + n, v);
+    };
+    if (TRANSPOSED) {
+        constexpr bool QUARTERS = sizeof(TW) == 2;
+        const int grp = tid >> 6, n = (QUARTERS ? blockIdx.x : blockIdx.x * 4 + grp) * HV_COLS + 2 * (tid & 63), KQ = QUARTERS ? (K + 3) / 4 : K,
+                  k_begin = QUARTERS ? grp * KQ : 0, k_end = min(K, k_begin + KQ);
+        const TW *w0 = W + (size_t)h * K * ldw + n;
+        if (n < N) {
+            for (int k0 = k_begin; k0 < k_end; k0 += 8) {
+                float2 w[8];                                // eight weights' rows on their way before the first is used
+#pragma unroll
+                for (int u = 0; u < 8; u++) {
+                    const TW *p = w0 + (size_t)min(k0 + u, K - 1) * ldw;
+                    if (vec) w[u] = HvPair<TW>::load(p);
+                    else w[u] = make_float2(to_f32<TW>(p[0]), n + 1 < N ? to_f32<TW>(p[1]) : 0.f);
+                }
+#pragma unroll
+                for (int u = 0; u < 8; u++) {
+                    if (k0 + u >= k_end) break;
+                    const float4 *x4 = (const float4 *)(as + (size_t)(k0 + u) * RM);
+#pragma unroll
+                    for (int q = 0; q < RM / 4; q++) {
+                        const float4 x = x4[q];
+                        acc[0][4 * q] = fmaf(x.x, w[u].x, acc[0][4 * q]); acc[1][4 * q] = fmaf(x.x, w[u].y, acc[1][4 * q]);
+                        acc[0][4 * q + 1] = fmaf(x.y, w[u].x, acc[0][4 * q + 1]); acc[1][4 * q + 1] = fmaf(x.y, w[u].y, acc[1][4 * q + 1]);
+                        acc[0][4 * q + 2] = fmaf(x.z, w[u].x, acc[0][4 * q + 2]); acc[1][4 * q + 2] = fmaf(x.z, w[u].y, acc[1][4 * q + 2]);
+                        acc[0][4 * q + 3] = fmaf(x.w, w[u].x, acc[0][4 * q + 3]); acc[1][4 * q + 3] = fmaf(x.w, w[u].y, acc[1][4 * q + 3]);
+                    }
+                }
+            }
+        }
+        if (!QUARTERS) {
+#pragma unroll
+            for (int m = 0; m < RM; m++) {
+                if (m >= M || n >= N) break;
+                store(m, n, acc[0][m]);
+                if (n + 1 < N) store(m, n + 1, acc[1][m]);
+            }
+            return;
+        }
+        __syncthreads();                                    // the rows are read; their memory takes the sums [4][RM][HV_COLS]
+#pragma unroll
+        for (int m = 0; m < RM; m++) *(float2 *)(as + ((size_t)grp * RM + m) * HV_COLS + 2 * (tid & 63)) = make_float2(acc[0][m], acc[1][m]);
+        __syncthreads();
+        for (int e = tid; e < M * HV_COLS; e += 256) {
+            const int m = e / HV_COLS, c = e - m * HV_COLS, nn = blockIdx.x * HV_COLS + c;
+            if (nn >= N) continue;
+            float v = 0.f;
+#pragma unroll
+            for (int g = 0; g < 4; g++) v += as[((size_t)g * RM + m) * HV_COLS + c];
+            store(m, nn, v);
+        }
+    } else {
+        const int lane = tid & 31, n = (blockIdx.x * 8 + (tid >> 5)) * 2;
+        if (n >= N) return;
+        constexpr int VEC = 16 / (int)sizeof(TW);
+        const TW *w0 = W + ((size_t)h * N + n) * ldw, *w1 = n + 1 < N ? w0 + ldw : w0;
+        if (vec) {
+#pragma unroll 2
+            for (int k = lane * VEC; k < K; k += 32 * VEC) {
+                const uint4 r0 = *(const uint4 *)(w0 + k), r1 = *(const uint4 *)(w1 + k);
+                const TW *e0 = (const TW *)&r0, *e1 = (const TW *)&r1;
+#pragma unroll
+                for (int m = 0; m < RM; m++) {
+                    float x[VEC];
+#pragma unroll
+                    for (int i = 0; i < VEC; i += 4) *(float4 *)(x + i) = *(const float4 *)(as + m * KP + k + i);
+#pragma unroll
+                    for (int i = 0; i < VEC; i++) {
+                        acc[0][m] = fmaf(x[i], to_f32<TW>(e0[i]), acc[0][m]);
+                        acc[1][m] = fmaf(x[i], to_f32<TW>(e1[i]), acc[1][m]);
+                    }
+                }
+            }
+        } else {
+            for (int k = lane; k < K; k += 32) {
+                const float a = to_f32<TW>(w0[k]), b = to_f32<TW>(w1[k]);
+#pragma unroll
+                for (int m = 0; m < RM; m++) { acc[0][m] = fmaf(as[m * KP + k], a, acc[0][m]); acc[1][m] = fmaf(as[m * KP + k], b, acc[1][m]); }
+            }
+        }
+        // sums of 2 RM numbers: at every exchange a lane keeps half of them, and ends with one (RM = 16) or one twice over (RM = 8)
+        float v[2 * RM];
+#pragma unroll
+        for (int m = 0; m < RM; m++) { v[m] = acc[0][m]; v[RM + m] = acc[1][m]; }
+#pragma unroll
+        for (int o = RM; o > 0; o >>= 1) {
+            const bool up = (lane & o) != 0;
+#pragma unroll
+            for (int i = 0; i < o; i++) {
+                const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+        }
+        if (RM == 8) v[0] += __shfl_xor_sync(0xffffffffu, v[0], 16);
+        const int m = lane & (RM - 1), c = (lane / RM) & 1;
+        if (lane < 2 * RM && m < M && n + c < N) store(m, n + c, v[0]);
     }
 }
 
@@ -444,13 +507,22 @@ extern "C" int fg_head_gemm(const void *A, int a_dtype, int lda, int a_stride, c
     if (K <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
     for (int d : {a_dtype, w_dtype, c_dtype})
         if (d != FG_F32 && d != FG_BF16) return FG_ERR_BAD_DTYPE;
-    if (M <= HV_ROWS && (size_t)M * K * sizeof(float) <= 48 * 1024) {
-        const size_t smem = (size_t)M * K * sizeof(float);
-        if (transposed)
-            return fg_launch(head_gemv_kernel<true>, dim3((N + 255) / 256, H), dim3(256), smem, stream, A, a_dtype, lda, a_stride, W, w_dtype, ldw, C,
-                             c_dtype, ldc, c_stride, gate, ldg, M, N, K);
-        return fg_launch(head_gemv_kernel<false>, dim3((N + 7) / 8, H), dim3(256), smem, stream, A, a_dtype, lda, a_stride, W, w_dtype, ldw, C, c_dtype,
-                         ldc, c_stride, gate, ldg, M, N, K);
+    const int RM = M <= 8 ? 8 : HV_ROWS;
+    if (M <= HV_ROWS && (size_t)RM * (K + 3) * sizeof(float) <= 48 * 1024) {
+        const size_t rows = (size_t)RM * ((K + 3) / 4 * 4) * sizeof(float), sums = (size_t)4 * RM * HV_COLS * sizeof(float);
+        const size_t smem = transposed && sums > rows ? sums : rows;
+        const size_t es = w_dtype == FG_F32 ? 4 : 2;
+        const int vec = transposed ? (N % 2 == 0 && ldw % 2 == 0 && ((uintptr_t)W % (2 * es)) == 0)
+                                   : (K % (int)(16 / es) == 0 && ldw % (int)(16 / es) == 0 && ((uintptr_t)W & 15) == 0);
+        const int cols = w_dtype == FG_F32 ? 4 * HV_COLS : HV_COLS;
+        const dim3 grid(transposed ? (N + cols - 1) / cols : (N + 15) / 16, H);
+#define HV_LAUNCH(TW, TR, R_) fg_launch(head_gemv_kernel<TW, TR, R_>, grid, dim3(256), smem, stream, A, a_dtype, lda, a_stride, (const TW *)W, ldw, C, \
+                                        c_dtype, ldc, c_stride, gate, ldg, M, N, K, vec)
+#define HV_BY_ROWS(TW, TR) (RM == 8 ? HV_LAUNCH(TW, TR, 8) : HV_LAUNCH(TW, TR, 16))
+        if (w_dtype == FG_F32) return transposed ? HV_BY_ROWS(float, true) : HV_BY_ROWS(float, false);
+        return transposed ? HV_BY_ROWS(bf16, true) : HV_BY_ROWS(bf16, false);
+#undef HV_BY_ROWS
+#undef HV_LAUNCH
     }
     dim3 grid((N + HG_T - 1) / HG_T, (M + HG_T - 1) / HG_T, H);
     if (grid.y > 65535) return FG_ERR_BAD_SIZE;

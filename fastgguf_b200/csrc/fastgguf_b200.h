@@ -108,7 +108,7 @@ int fg_rglru_tiles(int M, int C, int part, int bn);
 int fg_rglru_conv(const float *proj, int ldp, const float *proj_bias, const float *conv_w, const float *conv_b, int taps, const float *state,
                   long long state_stride, const int *positions, const int *row_seq, const int *cu_rows, const int *slots, float *u, int ldu,
                   void *pieces, void *tiles, int bn, int M, int C, int part, cudaStream_t stream);
-int fg_rglru_scan(const float *z, long long z_row, long long z_part, const float *gate_bias, const float *u, int ldu, const float *lam, float gain,
+int fg_rglru_scan(const float *z, int z_row, long long z_part, const float *gate_bias, const float *u, int ldu, const float *lam, float gain,
                   const float *proj, int ldp, const float *proj_bias, void *out, int out_dtype, int ldo, const int *cu_rows, const int *slots,
                   const int *positions, float *state, long long state_stride, int n_seq, int max_new, int C, int part, int taps, cudaStream_t stream);
 int fg_rglru_step_ok(int part);

@@ -364,9 +364,9 @@ public:
             Tensor lat = rt.arena->matrix(M, (int64_t)H_ * r_, rt.dtype);
             if (b.single_token && M <= 65535 && !rt.plain_kernels && rt.dtype == FG_BF16 && io.cache_dtype == FG_BF16 &&
                 FG_KERNEL("mix", fg_latent_decode_mma_ok)(r_, dr_, io.page_size)) {
-                // tensor cores: a block per (row, 16 heads, split of the pages), enough blocks to fill the GPU
+                // tensor cores: a block per (row, 16 heads, split of the pages), as many as run at once (about one an SM)
                 const int blocks = M * ((H_ + 15) / 16), pages = b.max_len / io.page_size + 1;
-                int n_splits = std::max(1, std::min({(rt.n_sm + blocks - 1) / blocks, 32, pages}));
+                int n_splits = std::max(1, std::min({rt.n_sm / blocks, 32, pages}));
                 const long long floats = FG_KERNEL("mix", fg_latent_decode_scratch_floats)(M, H_, r_, n_splits);
                 float *part = floats > 0 ? (float *)rt.arena->alloc((size_t)floats * sizeof(float)) : nullptr;
                 FG_LAUNCH("mix", fg_latent_decode_mma, qf.data, (int)qf.ld, lat.data, (int)lat.ld, b.positions, b.row_seq, table, b.table_width, io.k_pool,

@@ -501,7 +501,8 @@ public:
                       b.row_seq, b.slots, state, stride, y.data, y.dtype, (int)y.ld, M, C_, s, rt.stream);
         } else {
             Tensor u = rt.arena->matrix(M, C_, FG_F32), z;
-            long long z_row = 2 * C_, z_part = 2 * s;
+            int z_row = 2 * C_;
+            long long z_part = 2 * s;
             const bool tc = wide_.t.defined() && !b.single_token && M >= tensor_cores_from_;
             if (tc) {
                 Tensor pieces = rt.arena->matrix((int64_t)B_ * M, (int64_t)3 * s, FG_BF16);

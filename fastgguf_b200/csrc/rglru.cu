@@ -168,7 +168,7 @@ __device__ __forceinline__ float rg_remote(const float *p, int rank) {
 // grid (channel tiles of 32, sequences, blocks of the cluster): the cluster's blocks stand one after another along time.
 template <typename TO>
 __global__ void __launch_bounds__(SCAN_W * 32)
-rglru_scan_kernel(const float *__restrict__ z, long long z_row, long long z_part, const float *__restrict__ gate_bias,
+rglru_scan_kernel(const float *__restrict__ z, int z_row, long long z_part, const float *__restrict__ gate_bias,
                   const float *__restrict__ u, int ldu, const float *__restrict__ lam, float gain, const float *__restrict__ proj, int ldp,
                   const float *__restrict__ proj_bias, TO *__restrict__ out, int ldo, const int *__restrict__ cu_rows,
                   const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ state, long long state_stride, int C,
@@ -191,20 +191,32 @@ rglru_scan_kernel(const float *__restrict__ z, long long z_row, long long z_part
     for (int t0 = row0; t0 < row1; t0 += CS * SCAN_W * SCAN_T, it ^= 1) {
         const int first = t0 + (rank * SCAN_W + warp) * SCAN_T;
         const int n = live ? max(0, min(SCAN_T, row1 - first)) : 0;
-        float a[SCAN_T], b[SCAN_T];
+        const bool full = __all_sync(0xffffffffu, n == SCAN_T);        // the common case has no predicates
+        float a[SCAN_T], b[SCAN_T], y[SCAN_T];
         {
             float vr[SCAN_T], vi[SCAN_T], vu[SCAN_T];            // all loads on their way before the first is used
+            const float *zrp = zr + (size_t)first * z_row, *zip = zi + (size_t)first * z_row, *up = u + (size_t)first * ldu + cc,
+                        *yp = proj + (size_t)first * ldp + cc;
+            if (full) {
 #pragma unroll
-            for (int i = 0; i < SCAN_T; i++) {
-                const size_t m = (size_t)(first + i);
-                vr[i] = i < n ? zr[m * z_row] : 0.f;
-                vi[i] = i < n ? zi[m * z_row] : 0.f;
-                vu[i] = i < n ? u[m * ldu + c] : 0.f;
-            }
+                for (int i = 0; i < SCAN_T; i++) { vr[i] = zrp[i * z_row]; vi[i] = zip[i * z_row]; vu[i] = up[i * ldu]; }
 #pragma unroll
-            for (int i = 0; i < SCAN_T; i++) {
-                a[i] = 1.f; b[i] = 0.f;
-                if (i < n) rg_coefficients(vr[i] + br, vi[i] + bi, vu[i], rate, a[i], b[i]);
+                for (int i = 0; i < SCAN_T; i++) y[i] = yp[i * ldp];
+#pragma unroll
+                for (int i = 0; i < SCAN_T; i++) rg_coefficients(vr[i] + br, vi[i] + bi, vu[i], rate, a[i], b[i]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < SCAN_T; i++) {
+                    vr[i] = i < n ? zrp[i * z_row] : 0.f;
+                    vi[i] = i < n ? zip[i * z_row] : 0.f;
+                    vu[i] = i < n ? up[i * ldu] : 0.f;
+                    y[i] = i < n ? yp[i * ldp] : 0.f;
+                }
+#pragma unroll
+                for (int i = 0; i < SCAN_T; i++) {
+                    rg_coefficients(vr[i] + br, vi[i] + bi, vu[i], rate, a[i], b[i]);
+                    if (i >= n) { a[i] = 1.f; b[i] = 0.f; }
+                }
             }
         }
         float wa = 1.f, wb = 0.f;                               // this thread's tokens composed: S -> wa S + wb
@@ -212,9 +224,6 @@ rglru_scan_kernel(const float *__restrict__ z, long long z_row, long long z_part
         for (int i = 0; i < SCAN_T; i++) { wb = fmaf(a[i], wb, b[i]); wa *= a[i]; }
         agg_a[warp][lane] = wa;
         agg_b[warp][lane] = wb;
-        float y[SCAN_T];
-#pragma unroll
-        for (int i = 0; i < SCAN_T; i++) y[i] = i < n ? proj[(size_t)(first + i) * ldp + c] : 0.f;
         __syncthreads();
         float pa = 1.f, pb = 0.f, ta = 1.f, tb = 0.f;           // before this warp; the whole block
 #pragma unroll
@@ -244,10 +253,19 @@ rglru_scan_kernel(const float *__restrict__ z, long long z_row, long long z_part
             __syncthreads();                                    // the compositions are read before the next ones are written
         }
         float S = fmaf(pa, start, pb);
+        TO *op = out + (size_t)first * ldo + cc;
+        if (full) {
 #pragma unroll
-        for (int i = 0; i < SCAN_T; i++) {
-            S = fmaf(a[i], S, b[i]);
-            if (i < n) out[(size_t)(first + i) * ldo + c] = from_f32<TO>(S * rg_gelu(y[i] + yb));
+            for (int i = 0; i < SCAN_T; i++) {
+                S = fmaf(a[i], S, b[i]);
+                op[i * ldo] = from_f32<TO>(S * rg_gelu(y[i] + yb));
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < SCAN_T; i++) {
+                S = fmaf(a[i], S, b[i]);
+                if (i < n) op[i * ldo] = from_f32<TO>(S * rg_gelu(y[i] + yb));
+            }
         }
     }
     if (CS > 1) rg_cluster_sync();                              // nobody's totals go away while they are being read
@@ -429,7 +447,7 @@ extern "C" int fg_rglru_conv(const float *proj, int ldp, const float *proj_bias,
 
 // z: the gates' raw numbers (row m of part p: [r | i] at z + m * z_row + p * z_part); gate_bias: [C / part][2 * part]; lam: [C];
 // out: [M, ldo] in out_dtype.  Brings the state rows up to date.  max_new: the longest portion of the step.
-extern "C" int fg_rglru_scan(const float *z, long long z_row, long long z_part, const float *gate_bias, const float *u, int ldu,
+extern "C" int fg_rglru_scan(const float *z, int z_row, long long z_part, const float *gate_bias, const float *u, int ldu,
                              const float *lam, float gain, const float *proj, int ldp, const float *proj_bias, void *out, int out_dtype, int ldo,
                              const int *cu_rows, const int *slots, const int *positions, float *state, long long state_stride, int n_seq,
                              int max_new, int C, int part, int taps, cudaStream_t stream) {
