@@ -18,8 +18,7 @@
 // depend on what else is in the step.
 //
 // Weights: w_in [X, 2F, E] (gate rows, then up rows, of each expert; [X, F, E] where an expert has no gate), w_out [X, E, F];
-// activations and weights share
-// the engine's dtype T, accumulation is float32.
+// activations and weights share the engine's dtype T, accumulation is float32.
 #include "common.cuh"
 
 #define MOE_MAX_EXPERTS 256
@@ -91,8 +90,9 @@ extern "C" int fg_moe_logits(const void *x, int ldx, const void *W, int ldw, int
 // One block.  logits: [M, X] float32, to which `bias` (a float per output, or null) is added first.  chosen_softmax: the weights
 // are the softmax over the chosen logits alone; else each choice weighs in with the sigmoid of its logit.
 __global__ void __launch_bounds__(1024)
-moe_route_kernel(const float *__restrict__ logits, const float *__restrict__ bias, int chosen_softmax, int M, int X, int top, int *__restrict__ pair_expert, float *__restrict__ pair_weight,
-                 int *__restrict__ offsets, int *__restrict__ order, int *__restrict__ slot_of) {
+moe_route_kernel(const float *__restrict__ logits, const float *__restrict__ bias, int chosen_softmax, int M, int X, int top,
+                 int *__restrict__ pair_expert, float *__restrict__ pair_weight, int *__restrict__ offsets, int *__restrict__ order,
+                 int *__restrict__ slot_of) {
     __shared__ int counts[MOE_MAX_EXPERTS], cursor[MOE_MAX_EXPERTS];
     pdl_launch_dependents();
     pdl_wait();
