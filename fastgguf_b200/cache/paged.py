@@ -27,18 +27,19 @@ __all__ = ["CacheError", "CacheFull", "CacheRequest", "PagedKVCache", "cache_byt
 class CacheRequest:
     """Keys and values a mixer keeps per position.  ``window`` None keeps every position; an integer keeps the
     last ``window`` positions and, with ``keep_first``, the sequence's first positions as well.  ``v_head_dim``: values
-    of another head size than the keys.  Requests that agree in all fields share a cache group."""
+    of another head size than the keys; ``n_v_heads``: fewer heads of values than of keys.  Requests that agree in all fields share a cache group."""
 
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None
     keep_first: int = 0
+    n_v_heads: Optional[int] = None
 
 
 def _requests_json(requests: Dict[int, CacheRequest]) -> bytes:
     return json.dumps([{"entry": int(e), "n_kv_heads": r.n_kv_heads, "head_dim": r.head_dim, "window": r.window,
-                        "v_head_dim": r.v_head_dim, "keep_first": int(r.keep_first)}
+                        "v_head_dim": r.v_head_dim, "keep_first": int(r.keep_first), "n_v_heads": r.n_v_heads}
                        for e, r in sorted(requests.items())]).encode("utf-8")
 
 

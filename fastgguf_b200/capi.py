@@ -266,8 +266,7 @@ def kernel_modules_for(spec_json, dtype_code: int) -> tuple:
         if role == "mixer" and part.get("kind") == "gqa_attention" and p.get("head_dim") in (64, 128) \
                 and p.get("v_head_dim", p.get("head_dim")) == p.get("head_dim"):
             fast_attention = True
-        if role == "mixer" and part.get("kind") == "sink_attention" and p.get("head_dim") in (64, 128) \
-                and p.get("v_head_dim", p.get("head_dim")) == p.get("head_dim"):
+        if role == "mixer" and part.get("kind") == "sink_attention" and (p.get("head_dim"), p.get("v_head_dim", p.get("head_dim"))) in ((64, 64), (64, 128), (128, 128)):
             fast_attention = True
         if role == "mixer" and part.get("kind") == "latent_attention" and p.get("head_dim", 0) + p.get("rot_dim", 0) in (64, 128) \
                 and p.get("v_head_dim", 0) <= p.get("head_dim", 0) + p.get("rot_dim", 0):

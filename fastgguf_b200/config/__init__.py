@@ -6,5 +6,6 @@ from .salulorn import SalulornConfig
 from .pirozen import PirozenConfig
 from .saluzen import SaluzenConfig
 from .zifelorn import ZifelornConfig
+from .buguzen import BuguzenConfig
 
-__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "ZirivikConfig", "SalulornConfig", "PirozenConfig", "SaluzenConfig", "ZifelornConfig", "architecture_name", "read_config_json"]
+__all__ = ["ConfigError", "ModelConfig", "LlamaConfig", "ZirivikConfig", "SalulornConfig", "PirozenConfig", "SaluzenConfig", "ZifelornConfig", "BuguzenConfig", "architecture_name", "read_config_json"]

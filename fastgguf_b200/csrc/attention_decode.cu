@@ -4,6 +4,9 @@
 // of one KV head share every K/V load (the reference's "up to 4 query rows sharing one KV head",
 // :3268-3272).  Formulas as in attention_generic.cu.
 //
+// Values may be wider than keys (HV = 128 beside HD = 64), v_share neighbouring key heads may read one value head, and the output
+// may be float32 (what maps of a differential attention are subtracted in).
+//
 // Grid (split, kv head x head chunk, sequence).  The pages of a sequence are divided evenly
 // among `n_splits` CTAs, so one long sequence fills the GPU as well as many short ones; inside a
 // CTA four warps take pages round-robin, each with K and V buffers of its own (one K and one V
@@ -12,7 +15,7 @@
 // splits) and merge their partial (O, max, sum) through distributed shared memory, or (more
 // splits, very long contexts) write them to scratch memory for a second kernel to merge.
 //
-// The merge inside a cluster: CTA r owns the slice [r * HD / S, (r + 1) * HD / S) of the head dimension.  Every
+// The merge inside a cluster: CTA r owns the slice [r * HV / S, (r + 1) * HV / S) of the value dimension.  Every
 // warp that read pages pushes its running (max, sum) to all CTAs and the slices of its O to their owners
 // (st.shared::cluster), one cluster barrier makes the pushes visible, and each owner combines the up to 4 S
 // partial results of its slice in (split, warp) order from its own shared memory and writes the output.
@@ -45,22 +48,31 @@ struct RopeArgs {
     int keep_first;                  // with a window: the sequence's first keys stay visible (both forms of the kernel)
     float softcap;                   // > 0: capped scores (both forms)
     const float *sinks;              // or null: a float per query head that joins the softmax's denominator once
+    int v_share;                     // key heads that share a value head (1: each has its own)
+    int out_f32;                     // float32 output
 };
 
-template <int HD, bool CLUSTER, bool FUSE>
+__device__ __forceinline__ void store_out(void *out, int out_f32, size_t at, float v) {
+    if (out_f32) ((float *)out)[at] = v;
+    else ((bf16 *)out)[at] = __float2bfloat16_rn(v);
+}
+
+template <int HD, int HV, bool CLUSTER, bool FUSE>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ positions,
                    const int *__restrict__ block_table, int table_width,
                    const bf16 *__restrict__ k_pool, const bf16 *__restrict__ v_pool,
                    int KV, int G, float scale, int window, int n_splits,
                    float *__restrict__ part_o, float *__restrict__ part_ml,
-                   bf16 *__restrict__ out, int ldo, RopeArgs rope) {
+                   void *__restrict__ out, int ldo, RopeArgs rope) {
+    static_assert(!FUSE || HV == HD, "the fused form takes values of the keys' size");
     extern __shared__ __align__(128) uint8_t smem[];
-    constexpr int TILE_BYTES = PAGE * HD * 2;
+    constexpr int K_BYTES = PAGE * HD * 2, V_BYTES = PAGE * HV * 2, KV_BYTES = K_BYTES + V_BYTES;
     const int warp = warp_index(), lane = threadIdx.x & 31;
     const int chunks = (G + 15) / 16;
     const int kvh = blockIdx.y / chunks, g0 = (blockIdx.y % chunks) * 16;
     const int rows = min(16, G - g0);
+    const int VH = KV / rope.v_share, vh = kvh / rope.v_share;      // value heads in the pool, and this one
     const int b = blockIdx.z, split = blockIdx.x;
     if (CLUSTER && n_splits > 1) cluster_arrive_relaxed();       // matched before the first push: every CTA runs
     pdl_launch_dependents();
@@ -82,12 +94,12 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
     const int *bt = block_table + (size_t)b * table_width;
     auto page_of = [&](int i) { return i < n_kept ? i : first_page + (i - n_kept); };
 
-    uint8_t *kbuf = smem + (size_t)warp * 2 * TILE_BYTES, *vbuf = kbuf + TILE_BYTES;
+    uint8_t *kbuf = smem + (size_t)warp * KV_BYTES, *vbuf = kbuf + K_BYTES;
     const uint32_t ks = smem_addr(kbuf), vs = smem_addr(vbuf);
 
-    float o[HD / 8][4];
+    float o[HV / 8][4];
 #pragma unroll
-    for (int d = 0; d < HD / 8; d++) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    for (int d = 0; d < HV / 8; d++) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     const int lo[2] = {lo_key, lo_key}, hi[2] = {pos, pos};
     if (rope.sinks && split == 0 && warp == 0) {
@@ -103,10 +115,10 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
 
     int p = p_begin + warp;
     if (p < p_end) {
-        size_t base = ((size_t)bt[page_of(p)] * KV + kvh) * PAGE * HD;
-        load_page_warp<HD>(ks, k_pool + base, lane);
+        const size_t page = (size_t)bt[page_of(p)];
+        load_page_warp<HD>(ks, k_pool + (page * KV + kvh) * PAGE * HD, lane);
         cp_async_commit();
-        load_page_warp<HD>(vs, v_pool + base, lane);
+        load_page_warp<HV>(vs, v_pool + (page * VH + vh) * PAGE * HV, lane);
         cp_async_commit();
     }
     if (FUSE) pdl_wait();                      // q, k, v of the new token come from the kernel before
@@ -152,7 +164,7 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
     }
     for (; p < p_end; p += DEC_WARPS) {
         const int pn = p + DEC_WARPS;
-        const size_t nbase = pn < p_end ? ((size_t)bt[page_of(pn)] * KV + kvh) * PAGE * HD : 0;
+        const size_t npage = pn < p_end ? (size_t)bt[page_of(pn)] : 0;
         const int rp = page_of(p);             // the page of the sequence this step works on
         cp_async_wait<1>();                    // K of this page has landed (V may still be in flight)
         __syncwarp();
@@ -191,12 +203,12 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
         for (int j = 0; j < 8; j++) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
         qk_page<HD>(s, qf, ks, lane);
         __syncwarp();
-        if (pn < p_end) load_page_warp<HD>(ks, k_pool + nbase, lane);
+        if (pn < p_end) load_page_warp<HD>(ks, k_pool + (npage * KV + kvh) * PAGE * HD, lane);
         cp_async_commit();                     // (possibly empty) group: keeps the wait counts uniform
         if (rp * PAGE + PAGE - 1 <= pos && rp * PAGE >= lo_key)
-            softmax_update<HD / 8, false>(s, o, m, l, scale * LOG2E, rp * PAGE, lo, hi, lane, 0, cap_log2, cap_in);
+            softmax_update<HV / 8, false>(s, o, m, l, scale * LOG2E, rp * PAGE, lo, hi, lane, 0, cap_log2, cap_in);
         else
-            softmax_update<HD / 8, true>(s, o, m, l, scale * LOG2E, rp * PAGE, lo, hi, lane, keep, cap_log2, cap_in);
+            softmax_update<HV / 8, true>(s, o, m, l, scale * LOG2E, rp * PAGE, lo, hi, lane, keep, cap_log2, cap_in);
         cp_async_wait<1>();                    // V of this page has landed
         __syncwarp();
         if (newest) {
@@ -209,22 +221,22 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
             }
             __syncwarp();
         }
-        pv_page<HD>(o, s, vs, lane);
+        pv_page<HV>(o, s, vs, lane);
         __syncwarp();
-        if (pn < p_end) load_page_warp<HD>(vs, v_pool + nbase, lane);
+        if (pn < p_end) load_page_warp<HV>(vs, v_pool + (npage * VH + vh) * PAGE * HV, lane);
         cp_async_commit();
     }
     cp_async_wait<0>();
     if (CLUSTER) {
         // ---- every warp's partial result goes to the owners of its slices; see the head of this file
-        const int S = n_splits, dsl = HD / S, dsl_log = __ffs(dsl) - 1;          // HD and S are powers of two
-        float *recv_o = (float *)(smem + (size_t)DEC_WARPS * 2 * TILE_BYTES);     // [4 S][rows][dsl]
-        float *recv_ml = recv_o + DEC_WARPS * rows * HD;                           // [4 S][16][2]
+        const int S = n_splits, dsl = HV / S, dsl_log = __ffs(dsl) - 1;          // HV and S are powers of two
+        float *recv_o = (float *)(smem + (size_t)DEC_WARPS * KV_BYTES);     // [4 S][rows][dsl]
+        float *recv_ml = recv_o + DEC_WARPS * rows * HV;                           // [4 S][16][2]
         if (S > 1) cluster_wait();                                                // the phase opened at the top
         if (p_begin + warp < p_end) {                                             // this warp read at least one page
             const int slot = split * DEC_WARPS + warp, r0 = lane >> 2, c = (lane & 3) * 2;
 #pragma unroll
-            for (int d = 0; d < HD / 8; d++) {
+            for (int d = 0; d < HV / 8; d++) {
                 const int col = d * 8 + c, owner = col >> dsl_log, cc = col & (dsl - 1);
                 if (r0 < rows) st_dsmem2(&recv_o[(slot * rows + r0) * dsl + cc], owner, o[d][0], o[d][1]);
                 if (r0 + 8 < rows) st_dsmem2(&recv_o[(slot * rows + r0 + 8) * dsl + cc], owner, o[d][2], o[d][3]);
@@ -271,21 +283,22 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
                     L += wgt * lw[w];
                 }
             }
-            out[(size_t)b * ldo + (size_t)(kvh * G + g0 + r) * HD + split * dsl + cc] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+            store_out(out, rope.out_f32, (size_t)b * ldo + (size_t)(kvh * G + g0 + r) * HV + split * dsl + cc, L > 0.f ? O / L : 0.f);
         }
         return;
     }
     __syncthreads();
 
-    // ---- scratch path: merge the four warps, each leaves (m, l) and O[16][HD] in its own buffer
-    float *wo = (float *)kbuf;                 // 16 * HD floats <= TILE_BYTES
+    // ---- scratch path: merge the four warps, each leaves (m, l) and O[16][HV] in its own buffer
+    static_assert(16 * HV * 4 <= K_BYTES, "a warp's partial result fits its K tile");
+    float *wo = (float *)kbuf;                 // 16 * HV floats
     float *wml = (float *)vbuf;                // 16 * 2 floats
     {
         const int r0 = lane >> 2, c = (lane & 3) * 2;
 #pragma unroll
-        for (int d = 0; d < HD / 8; d++) {
-            wo[r0 * HD + d * 8 + c] = o[d][0];       wo[r0 * HD + d * 8 + c + 1] = o[d][1];
-            wo[(r0 + 8) * HD + d * 8 + c] = o[d][2]; wo[(r0 + 8) * HD + d * 8 + c + 1] = o[d][3];
+        for (int d = 0; d < HV / 8; d++) {
+            wo[r0 * HV + d * 8 + c] = o[d][0];       wo[r0 * HV + d * 8 + c + 1] = o[d][1];
+            wo[(r0 + 8) * HV + d * 8 + c] = o[d][2]; wo[(r0 + 8) * HV + d * 8 + c + 1] = o[d][3];
         }
         if ((lane & 3) == 0) {
             wml[r0 * 2] = m[0]; wml[r0 * 2 + 1] = l[0];
@@ -293,36 +306,36 @@ attn_decode_kernel(const bf16 *__restrict__ q, int ldq, const int *__restrict__ 
         }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < rows * HD; i += DEC_WARPS * 32) {
-        int r = i / HD, d = i % HD;
+    for (int i = threadIdx.x; i < rows * HV; i += DEC_WARPS * 32) {
+        int r = i / HV, d = i % HV;
         float M = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < DEC_WARPS; w++) M = fmaxf(M, ((float *)(smem + (size_t)w * 2 * TILE_BYTES + TILE_BYTES))[r * 2]);
+        for (int w = 0; w < DEC_WARPS; w++) M = fmaxf(M, ((float *)(smem + (size_t)w * KV_BYTES + K_BYTES))[r * 2]);
         float O = 0.f, L = 0.f;
 #pragma unroll
         for (int w = 0; w < DEC_WARPS; w++) {
-            const float *pml = (const float *)(smem + (size_t)w * 2 * TILE_BYTES + TILE_BYTES);
-            const float *po = (const float *)(smem + (size_t)w * 2 * TILE_BYTES);
+            const float *pml = (const float *)(smem + (size_t)w * KV_BYTES + K_BYTES);
+            const float *po = (const float *)(smem + (size_t)w * KV_BYTES);
             float mw = pml[r * 2];
             float wgt = mw == -INFINITY ? 0.f : ex2(mw - M);
-            O += wgt * po[r * HD + d];
+            O += wgt * po[r * HV + d];
             L += wgt * pml[r * 2 + 1];
         }
         int h = kvh * G + g0 + r;
         if (n_splits == 1) {
-            out[(size_t)b * ldo + (size_t)h * HD + d] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+            store_out(out, rope.out_f32, (size_t)b * ldo + (size_t)h * HV + d, L > 0.f ? O / L : 0.f);
         } else {
             size_t prow = ((size_t)b * KV * G + h) * n_splits + split;
-            part_o[prow * HD + d] = O;
+            part_o[prow * HV + d] = O;
             if (d == 0) { part_ml[prow * 2] = M; part_ml[prow * 2 + 1] = L; }
         }
     }
 }
 
 // merge the splits of one (sequence, head) in split order
-template <int HD>
+template <int HV>
 __global__ void attn_decode_merge_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml,
-                                         int n_splits, int H, bf16 *__restrict__ out, int ldo) {
+                                         int n_splits, int H, void *__restrict__ out, int ldo, int out_f32) {
     const int b = blockIdx.y, h = blockIdx.x, d = threadIdx.x;
     pdl_launch_dependents();
     pdl_wait();
@@ -333,21 +346,21 @@ __global__ void attn_decode_merge_kernel(const float *__restrict__ part_o, const
     for (int s = 0; s < n_splits; s++) {
         float ms = part_ml[(prow0 + s) * 2];
         float wgt = ms == -INFINITY ? 0.f : ex2(ms - M);
-        O += wgt * part_o[(prow0 + s) * HD + d];
+        O += wgt * part_o[(prow0 + s) * HV + d];
         L += wgt * part_ml[(prow0 + s) * 2 + 1];
     }
-    out[(size_t)b * ldo + (size_t)h * HD + d] = __float2bfloat16_rn(L > 0.f ? O / L : 0.f);
+    store_out(out, out_f32, (size_t)b * ldo + (size_t)h * HV + d, L > 0.f ? O / L : 0.f);
 }
 
-template <int HD, bool CLUSTER, bool FUSE = false>
+template <int HD, int HV, bool CLUSTER, bool FUSE = false>
 static int launch_decode_kernel(dim3 grid, int cluster_x, cudaStream_t stream, const void *q, int ldq, void *out, int ldo,
                                 const int *positions, const int *block_table, int table_width, const void *k_pool,
                                 const void *v_pool, int KV, int G, float scale, int window, int n_splits,
-                                float *part_o, float *part_ml, RopeArgs rope = RopeArgs{}) {
-    // behind the page buffers: the cluster merge receives 4 S partial slices [rows][HD / S] and (max, sum) pairs
-    constexpr int smem_max = DEC_WARPS * 2 * PAGE * HD * 2 + (CLUSTER ? DEC_WARPS * 16 * HD * 4 + DEC_WARPS * 8 * 16 * 2 * 4 : 0);
+                                float *part_o, float *part_ml, RopeArgs rope) {
+    // behind the page buffers: the cluster merge receives 4 S partial slices [rows][HV / S] and (max, sum) pairs
+    constexpr int smem_max = DEC_WARPS * PAGE * (HD + HV) * 2 + (CLUSTER ? DEC_WARPS * 16 * HV * 4 + DEC_WARPS * 8 * 16 * 2 * 4 : 0);
     const int rows_cap = G < 16 ? G : 16;
-    const int smem = DEC_WARPS * 2 * PAGE * HD * 2 + (CLUSTER ? DEC_WARPS * rows_cap * HD * 4 + DEC_WARPS * n_splits * 16 * 2 * 4 : 0);
+    const int smem = DEC_WARPS * PAGE * (HD + HV) * 2 + (CLUSTER ? DEC_WARPS * rows_cap * HV * 4 + DEC_WARPS * n_splits * 16 * 2 * 4 : 0);
     // the attribute belongs to the function on ONE device: set it once on every device that launches
     static bool configured[64] = {false};
     int dev = 0;
@@ -355,7 +368,7 @@ static int launch_decode_kernel(dim3 grid, int cluster_x, cudaStream_t stream, c
     if (ed != cudaSuccess) return (int)ed;
     if (dev < 0 || dev >= 64) return FG_ERR_BAD_SIZE;
     if (!configured[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD, CLUSTER, FUSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max);
+        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD, HV, CLUSTER, FUSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max);
         if (e != cudaSuccess) return (int)e;
         configured[dev] = true;
     }
@@ -374,53 +387,59 @@ static int launch_decode_kernel(dim3 grid, int cluster_x, cudaStream_t stream, c
         n++;
     }
     cfg.attrs = attr; cfg.numAttrs = n;
-    return (int)cudaLaunchKernelEx(&cfg, attn_decode_kernel<HD, CLUSTER, FUSE>, (const bf16 *)q, ldq, positions, block_table,
+    return (int)cudaLaunchKernelEx(&cfg, attn_decode_kernel<HD, HV, CLUSTER, FUSE>, (const bf16 *)q, ldq, positions, block_table,
                                    table_width, (const bf16 *)k_pool, (const bf16 *)v_pool, KV, G, scale, window, n_splits,
-                                   part_o, part_ml, (bf16 *)out, ldo, rope);
+                                   part_o, part_ml, out, ldo, rope);
 }
 
-template <int HD>
+template <int HD, int HV>
 static int launch_decode(const void *q, int ldq, void *out, int ldo, const int *positions, const int *block_table,
                          int table_width, const void *k_pool, const void *v_pool, int B, int H, int KV, float scale,
                          int window, int keep_first, int n_splits, float *part_o, float *part_ml, cudaStream_t stream,
-                         float softcap = 0.f, const float *sinks = nullptr) {
+                         float softcap, const float *sinks, int v_share, int out_f32) {
     int G = H / KV;
     dim3 grid(n_splits, KV * ((G + 15) / 16), B);
     RopeArgs extra{};
     extra.keep_first = keep_first;
     extra.softcap = softcap;
     extra.sinks = sinks;
+    extra.v_share = v_share;
+    extra.out_f32 = out_f32;
     // 2, 4 or 8 splits without scratch memory: merged inside a cluster
     bool cluster = !part_o && (n_splits == 2 || n_splits == 4 || n_splits == 8);
     if (n_splits == 1 || cluster)
-        return launch_decode_kernel<HD, true>(grid, cluster ? n_splits : 1, stream, q, ldq, out, ldo, positions, block_table,
+        return launch_decode_kernel<HD, HV, true>(grid, cluster ? n_splits : 1, stream, q, ldq, out, ldo, positions, block_table,
                                               table_width, k_pool, v_pool, KV, G, scale, window, n_splits, nullptr, nullptr, extra);
-    int e = launch_decode_kernel<HD, false>(grid, 1, stream, q, ldq, out, ldo, positions, block_table, table_width, k_pool,
+    int e = launch_decode_kernel<HD, HV, false>(grid, 1, stream, q, ldq, out, ldo, positions, block_table, table_width, k_pool,
                                             v_pool, KV, G, scale, window, n_splits, part_o, part_ml, extra);
     if (e) return e;
-    return fg_launch(attn_decode_merge_kernel<HD>, dim3(H, B), dim3(HD), 0, stream, (const float *)part_o,
-                     (const float *)part_ml, n_splits, H, (bf16 *)out, ldo);
+    return fg_launch(attn_decode_merge_kernel<HV>, dim3(H, B), dim3(HV), 0, stream, (const float *)part_o,
+                     (const float *)part_ml, n_splits, H, out, ldo, out_f32);
 }
 
 // q: [B, ldq] bf16, one row per sequence, heads first in the row; positions[b] is the position of
 // that row (its key and value are already in the cache); pools [pages, KV, 64, HD] bf16.
 // part_o: [B, H, n_splits, HD] f32 and part_ml: [B, H, n_splits, 2] f32 scratch for the two-kernel
 // path; pass null pointers with n_splits 1, 2, 4 or 8 for the path that needs no scratch.
-// Takes HD 64 and 128 and pages of 64; anything else returns FG_ERR_BAD_SIZE.
+// Takes HD 64 and 128 (values hdv of the same size, or 128 beside 64) and pages of 64; anything else returns FG_ERR_BAD_SIZE.
 // keep_first (with a window): the first keep_first keys of the sequence stay visible.
 // softcap > 0: capped scores; sinks (or null): a float per query head that joins the softmax's denominator.
 extern "C" int fg_attention_decode_ext(const void *q, int ldq, void *out, int ldo, const int *positions,
                                         const int *block_table, int table_width, const void *k_pool, const void *v_pool,
                                         int B, int H, int KV, int hd, int page_size, float scale, int window, int keep_first,
-                                        int n_splits, float *part_o, float *part_ml, float softcap, const float *sinks,
-                                        cudaStream_t stream) {
+                                        int n_splits, float *part_o, float *part_ml, float softcap, const float *sinks, int hdv,
+                                        int v_share, int out_f32, cudaStream_t stream) {
     if (B <= 0) return 0;
-    if (KV <= 0 || H <= 0 || keep_first < 0 || softcap < 0.f) return FG_ERR_BAD_SIZE;
+    if (KV <= 0 || H <= 0 || keep_first < 0 || softcap < 0.f || v_share <= 0 || KV % v_share) return FG_ERR_BAD_SIZE;
     if (page_size != PAGE || H % KV || n_splits < 1 || B > 65535 || ldq % 2 || ((uintptr_t)q & 3)) return FG_ERR_BAD_SIZE;
     if ((part_o == nullptr) != (part_ml == nullptr)) return FG_ERR_BAD_SIZE;
     if (!part_o && n_splits != 1 && n_splits != 2 && n_splits != 4 && n_splits != 8) return FG_ERR_BAD_SIZE;
-    if (hd == 64) return launch_decode<64>(q, ldq, out, ldo, positions, block_table, table_width, k_pool, v_pool, B, H, KV, scale, window, keep_first, n_splits, part_o, part_ml, stream, softcap, sinks);
-    if (hd == 128) return launch_decode<128>(q, ldq, out, ldo, positions, block_table, table_width, k_pool, v_pool, B, H, KV, scale, window, keep_first, n_splits, part_o, part_ml, stream, softcap, sinks);
+#define DEC_RUN(HD, HV) launch_decode<HD, HV>(q, ldq, out, ldo, positions, block_table, table_width, k_pool, v_pool, B, H, KV, scale, window, keep_first, \
+                                              n_splits, part_o, part_ml, stream, softcap, sinks, v_share, out_f32)
+    if (hd == 64 && hdv == 64) return DEC_RUN(64, 64);
+    if (hd == 64 && hdv == 128) return DEC_RUN(64, 128);
+    if (hd == 128 && hdv == 128) return DEC_RUN(128, 128);
+#undef DEC_RUN
     return FG_ERR_BAD_SIZE;
 }
 
@@ -429,7 +448,7 @@ extern "C" int fg_attention_decode_kept(const void *q, int ldq, void *out, int l
                                         int B, int H, int KV, int hd, int page_size, float scale, int window, int keep_first,
                                         int n_splits, float *part_o, float *part_ml, cudaStream_t stream) {
     return fg_attention_decode_ext(q, ldq, out, ldo, positions, block_table, table_width, k_pool, v_pool, B, H, KV, hd, page_size, scale,
-                                   window, keep_first, n_splits, part_o, part_ml, 0.f, nullptr, stream);
+                                   window, keep_first, n_splits, part_o, part_ml, 0.f, nullptr, hd, 1, 0, stream);
 }
 
 extern "C" int fg_attention_decode(const void *q, int ldq, void *out, int ldo, const int *positions,
@@ -455,13 +474,13 @@ extern "C" int fg_attention_decode_fused_kept(const void *qkv, int ldq, void *ou
         return FG_ERR_BAD_SIZE;
     int G = H / KV;
     dim3 grid(n_splits, KV * ((G + 15) / 16), B);
-    RopeArgs rope{cos_t, sin_t, (bf16 *)k_pool, (bf16 *)v_pool, H, keep_first};
+    RopeArgs rope{cos_t, sin_t, (bf16 *)k_pool, (bf16 *)v_pool, H, keep_first, 0.f, nullptr, 1, 0};
     if (hd == 64)
-        return launch_decode_kernel<64, true, true>(grid, n_splits, stream, qkv, ldq, out, ldo, positions, block_table,
+        return launch_decode_kernel<64, 64, true, true>(grid, n_splits, stream, qkv, ldq, out, ldo, positions, block_table,
                                                     table_width, k_pool, v_pool, KV, G, scale, window, n_splits, nullptr,
                                                     nullptr, rope);
     if (hd == 128)
-        return launch_decode_kernel<128, true, true>(grid, n_splits, stream, qkv, ldq, out, ldo, positions, block_table,
+        return launch_decode_kernel<128, 128, true, true>(grid, n_splits, stream, qkv, ldq, out, ldo, positions, block_table,
                                                      table_width, k_pool, v_pool, KV, G, scale, window, n_splits, nullptr,
                                                      nullptr, rope);
     return FG_ERR_BAD_SIZE;
@@ -517,12 +536,14 @@ extern "C" int fg_attention_decode_noalloc(const void *q, int ldq, void *out, in
     if (page_size != PAGE || H % KV || B > 65535 || ldq % 2 || ((uintptr_t)q & 3)) return FG_ERR_BAD_SIZE;
     int G = H / KV;
     dim3 grid(n_splits, KV * ((G + 15) / 16), B);
+    RopeArgs plain{};
+    plain.v_share = 1;
 #define NOALLOC_RUN(HD) do { \
-        e = launch_decode_kernel<HD, false>(grid, 1, stream, q, ldq, out, ldo, positions, block_table, table_width, \
-                                            k_pool, v_pool, KV, G, scale, window, n_splits, part_o, part_ml); \
+        e = launch_decode_kernel<HD, HD, false>(grid, 1, stream, q, ldq, out, ldo, positions, block_table, table_width, \
+                                            k_pool, v_pool, KV, G, scale, window, n_splits, part_o, part_ml, plain); \
         if (e || n_splits == 1) return e;      /* one split writes the output itself */ \
         return fg_launch(attn_decode_merge_kernel<HD>, dim3(H, B), dim3(HD), 0, stream, (const float *)part_o, \
-                         (const float *)part_ml, n_splits, H, (bf16 *)out, ldo); } while (0)
+                         (const float *)part_ml, n_splits, H, out, ldo, 0); } while (0)
     if (hd == 64) NOALLOC_RUN(64);
     if (hd == 128) NOALLOC_RUN(128);
 #undef NOALLOC_RUN

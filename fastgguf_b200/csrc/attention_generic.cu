@@ -15,6 +15,8 @@
 // well) and a rotated key part in k_pool (hd numbers); a query row then has hdv + hd numbers a head, and a score is
 // q[0:hdv] . latent + q[hdv:] . rotated part.  This is attention over keys and values that are linear maps of the
 // latent, with the key map folded into the query and the value map applied to the output by the caller.
+// v_share: that many neighbouring key heads read the same value head (the pool of values then has KV / v_share heads).
+// out_f32: the output is float32 whatever T is.
 //
 // Keys are visited in chunks of CHUNK visible keys, the kept first ones and then the window from lo, with a running maximum and
 // sum in f32 (online softmax).  Within a chunk a thread scores whole keys; for the weighted sum of
@@ -31,12 +33,12 @@
 
 template <typename T, int DPL>          // DPL: output dimensions a lane owns (32 * DPL >= head size)
 __global__ void __launch_bounds__(ATT_THREADS)
-attention_generic_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, int ldo,
+attention_generic_kernel(const T *__restrict__ q, int ldq, void *__restrict__ out, int ldo,
                          const int *__restrict__ positions, const int *__restrict__ row_seq,
                          const int *__restrict__ block_table, int table_width,
                          const T *__restrict__ k_pool, const T *__restrict__ v_pool,
                          int H, int KV, int hd, int hdv, int page_size, float scale, int window, int keep_first,
-                         float softcap, const float *__restrict__ sinks, int latent) {
+                         float softcap, const float *__restrict__ sinks, int latent, int v_share, int out_f32) {
     extern __shared__ float smem[];
     const int qd = latent ? hdv + hd : hd;      // numbers a query head holds
     float *qs = smem;                 // [qd]
@@ -44,6 +46,7 @@ attention_generic_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, 
     __shared__ float scratch[32];
     int m = blockIdx.x, h = blockIdx.y;
     int kvh = h / (H / KV);
+    const int VH = KV / v_share, vh = kvh / v_share;    // value heads in the pool, and this one
     int pos = positions[m];
     int lo = first_visible_key(pos, window);
     const int n_first = min(keep_first, lo);          // kept first keys that lie in front of the window
@@ -80,7 +83,7 @@ attention_generic_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, 
                 for (int d = 0; d < hd; d++) s = fmaf(qk[d], to_f32<T>(kr[d]), s);
             }
             if (latent) {
-                const T *lr = v_pool + (((size_t)bt[p / page_size] * KV + kvh) * page_size + p % page_size) * hdv;
+                const T *lr = v_pool + (((size_t)bt[p / page_size] * VH + vh) * page_size + p % page_size) * hdv;
                 for (int d = 0; d < hdv; d++) s = fmaf(qs[d], to_f32<T>(lr[d]), s);
             }
             s *= scale;
@@ -110,7 +113,7 @@ attention_generic_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, 
             const int p = vi < n_first ? vi : lo + (vi - n_first), off = p % page_size;
             // a run of keys within one page, and within the kept first keys or within the window
             const int cnt = min(min(page_size - off, i_end - i), vi < n_first ? n_first - vi : i_end - i);
-            const T *vr = v_pool + (((size_t)bt[p / page_size] * KV + kvh) * page_size + off) * hdv;
+            const T *vr = v_pool + (((size_t)bt[p / page_size] * VH + vh) * page_size + off) * hdv;
             for (int u0 = 0; u0 < cnt; u0 += 8) {
                 float v[8][DPL];
 #pragma unroll
@@ -148,11 +151,14 @@ attention_generic_kernel(const T *__restrict__ q, int ldq, T *__restrict__ out, 
         __syncthreads();                   // sc[] and part[] are rewritten by the next chunk
     }
     if (warp == 0) {
-        T *orow = out + (size_t)m * ldo + (size_t)h * hdv;
+        const size_t at = (size_t)m * ldo + (size_t)h * hdv;
         const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
 #pragma unroll
         for (int j = 0; j < DPL; j++)
-            if (lane + 32 * j < hdv) orow[lane + 32 * j] = from_f32<T>(acc[j] * inv);
+            if (lane + 32 * j < hdv) {
+                if (out_f32) ((float *)out)[at + lane + 32 * j] = acc[j] * inv;
+                else ((T *)out)[at + lane + 32 * j] = from_f32<T>(acc[j] * inv);
+            }
     }
 }
 
@@ -160,15 +166,17 @@ extern "C" int fg_attention_generic_ext(const void *q, int ldq, void *out, int l
                                         const int *positions, const int *row_seq, const int *block_table,
                                         int table_width, const void *k_pool, const void *v_pool,
                                         int M, int H, int KV, int hd, int hdv, int page_size, float scale, int window,
-                                        int keep_first, float softcap, const float *sinks, int latent, cudaStream_t stream) {
+                                        int keep_first, float softcap, const float *sinks, int latent, int v_share, int out_f32,
+                                        cudaStream_t stream) {
     if (M <= 0) return 0;
-    if (hdv > 32 * MAX_DPL || hd <= 0 || hdv <= 0 || H % KV != 0 || H > 65535 || keep_first < 0 || softcap < 0.f) return FG_ERR_BAD_SIZE;
+    if (hdv > 32 * MAX_DPL || hd <= 0 || hdv <= 0 || H % KV != 0 || H > 65535 || keep_first < 0 || softcap < 0.f || v_share <= 0 || KV % v_share)
+        return FG_ERR_BAD_SIZE;
     dim3 grid(M, H);
     size_t smem = (size_t)((latent ? hd + hdv : hd) + CHUNK + ATT_WARPS * hdv) * sizeof(float);
     if (smem > 48 * 1024) return FG_ERR_BAD_SIZE;
-#define ATT_LAUNCH(T, DPL) attention_generic_kernel<T, DPL><<<grid, ATT_THREADS, smem, stream>>>((const T *)q, ldq, (T *)out, ldo, \
+#define ATT_LAUNCH(T, DPL) attention_generic_kernel<T, DPL><<<grid, ATT_THREADS, smem, stream>>>((const T *)q, ldq, out, ldo, \
         positions, row_seq, block_table, table_width, (const T *)k_pool, (const T *)v_pool, H, KV, hd, hdv, page_size, scale, window, \
-        window > 0 ? keep_first : 0, softcap, sinks, latent)
+        window > 0 ? keep_first : 0, softcap, sinks, latent, v_share, out_f32)
 #define ATT_BY_SIZE(T) do { if (hdv <= 64) ATT_LAUNCH(T, 2); else if (hdv <= 128) ATT_LAUNCH(T, 4); else if (hdv <= 256) ATT_LAUNCH(T, 8); \
                             else ATT_LAUNCH(T, 16); } while (0)
     if (dtype == FG_F32) ATT_BY_SIZE(float);
@@ -186,7 +194,7 @@ extern "C" int fg_attention_generic_kept(const void *q, int ldq, void *out, int 
                                          int keep_first, cudaStream_t stream) {
     if (hd > 256 || hdv > 256) return FG_ERR_BAD_SIZE;
     return fg_attention_generic_ext(q, ldq, out, ldo, dtype, positions, row_seq, block_table, table_width, k_pool, v_pool, M, H, KV,
-                                    hd, hdv, page_size, scale, window, keep_first, 0.f, nullptr, 0, stream);
+                                    hd, hdv, page_size, scale, window, keep_first, 0.f, nullptr, 0, 1, 0, stream);
 }
 
 extern "C" int fg_attention_generic(const void *q, int ldq, void *out, int ldo, int dtype,

@@ -31,7 +31,8 @@
 //                      (tcgen05.ld / st), after the MMAs before have finished.  At the end the row is read
 //                      once, divided by the sum and stored.
 //
-// Every mbarrier wait is bounded (error flag, tensor memory freed, copies in flight awaited).
+// Values may be wider than keys (HV = 128 beside HD = 64), v_share neighbouring key heads may read one value head, and the output
+// may be float32.  Every mbarrier wait is bounded (error flag, tensor memory freed, copies in flight awaited).
 #include <cuda.h>
 #include <climits>
 #include "common.cuh"
@@ -211,20 +212,22 @@ __device__ __forceinline__ void softmax_chunk(const float (&v)[32], int key, int
 // of its own, so that nothing orders the softmax of one iteration behind the one before it; the two partial results
 // of a row (O, maximum, sum) are combined at the end.  Four softmax streams an SM instead of two keep the exponential
 // unit busier.
-template <int HD, bool PIPE, bool PP>
+template <int HD, int HV, bool PIPE, bool PP>
 __global__ void __launch_bounds__(ATT_THREADS(PP), 2)              // two CTAs share an SM and overlap
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                       const bf16 *__restrict__ q, int ldq, bf16 *__restrict__ out, int ldo,
+                       const bf16 *__restrict__ q, int ldq, void *__restrict__ out, int ldo,
                        const int *__restrict__ cu_rows, const int *__restrict__ seq_start,
                        const int *__restrict__ block_table, int table_width, int KV, int G, float scale_log2, int window,
-                       int keep_first, int test_skip_copy, float cap_log2, float cap_in, const float *__restrict__ sinks) {
-    constexpr int CH = HD / 64;                        // 64-wide chunks of the head dimension
-    constexpr int KEYS = PIPE ? 64 : (HD > 64 ? 64 : 128), NPG = KEYS / PAGE;      // keys and pages per iteration
+                       int keep_first, int test_skip_copy, float cap_log2, float cap_in, const float *__restrict__ sinks,
+                       int v_share, int out_f32) {
+    constexpr int CH = HD / 64, CHV = HV / 64;         // 64-wide chunks of a key and of a value
+    constexpr int KEYS = PIPE ? 64 : (HV > 64 ? 64 : 128), NPG = KEYS / PAGE;      // keys and pages per iteration
     constexpr int NS = PIPE ? 2 : 1;                   // score tiles in tensor memory, P tiles in shared memory
-    constexpr int Q_BYTES = ROWS * HD * 2, KV_TILE = KEYS * HD * 2, P_TILE = ROWS * KEYS * 2;
-    constexpr uint32_t TMEM_COLS = 256;                // S tiles: columns 0..NS*KEYS-1, O: the HD columns after them (PP: twice)
+    constexpr int Q_BYTES = ROWS * HD * 2, K_TILE = KEYS * HD * 2, V_TILE = KEYS * HV * 2, P_TILE = ROWS * KEYS * 2;
+    constexpr uint32_t TMEM_COLS = 256;                // S tiles: columns 0..NS*KEYS-1, O: the HV columns after them (PP: twice)
     constexpr uint32_t O_COL = NS * KEYS;
-    static_assert(!PP || (PIPE && O_COL + 2 * HD <= TMEM_COLS), "two accumulators need two score tiles and head size 64");
+    static_assert(O_COL + HV <= TMEM_COLS && HV >= HD, "the accumulator fits behind the score tiles");
+    static_assert(!PP || (PIPE && O_COL + 2 * HV <= TMEM_COLS), "two accumulators need two score tiles and head size 64");
 
     extern __shared__ uint8_t smem_raw[];
     uint8_t *smem = (uint8_t *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -236,7 +239,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     const int Gc = G < 16 ? G : 16, TQ = ROWS / Gc, chunks = (G + Gc - 1) / Gc;
     const int kvh = blockIdx.x / chunks, g0 = (blockIdx.x % chunks) * Gc;
     const int b = blockIdx.z;
-    const uint32_t qs = smem_u32(smem), kt = qs + Q_BYTES, vt = kt + KV_TILE, ps = vt + KV_TILE;
+    const int VH = KV / v_share, vh = kvh / v_share;   // value heads in the pool, and this one
+    const uint32_t qs = smem_u32(smem), kt = qs + Q_BYTES, vt = kt + K_TILE, ps = vt + V_TILE;
     const uint32_t k_full = smem_u32(&bars[0]), k_empty = smem_u32(&bars[1]);
     const uint32_t v_full = smem_u32(&bars[2]), v_empty = smem_u32(&bars[3]);
     const uint32_t s_full = smem_u32(&bars[4]), p_full = smem_u32(&bars[6]), o_full = smem_u32(&bars[8]);     // s_full, p_full: one per tile
@@ -305,16 +309,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         // order: K(0), then for every iteration K(j + 1) before V(j) - K(j + 1) may go as soon as S(j) has read the K
         // tile, V(j) only when P V of iteration j - 1 has read the V tile, which is later
         int k_issued = 0, v_issued = 0;
-        auto page_rows = [&](int j, int (&y)[NPG]) {
+        auto page_rows = [&](int j, int (&y)[NPG], int heads, int head) {
             for (int h = 0; h < NPG; h++)
-                y[h] = (bt[min(first_page_of(j) + h, p_end - 1)] * KV + kvh) * PAGE;   // a page past the end is masked anyway
+                y[h] = (bt[min(first_page_of(j) + h, p_end - 1)] * heads + head) * PAGE;   // a page past the end is masked anyway
         };
         auto load_k = [&](int j) {
             int y[NPG];
-            page_rows(j, y);
+            page_rows(j, y, KV, kvh);
             if (!__all_sync(0xffffffffu, mbar_wait(k_empty, (j & 1) ^ 1))) { raise_error(1); return false; }
             if (elect_one()) {
-                mbar_expect_tx(k_full, KV_TILE);
+                mbar_expect_tx(k_full, K_TILE);
                 // (a test may ask for the first K tile to stay incomplete: its barrier never fires and every wait runs out)
                 if (!(test_skip_copy && j == 0))
                     for (int h = 0; h < NPG; h++)
@@ -328,12 +332,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         for (int j = 0; j < n_iter && ok; j++) {
             if (j + 1 < n_iter && !load_k(j + 1)) break;
             int y[NPG];
-            page_rows(j, y);
+            page_rows(j, y, VH, vh);
             if (!__all_sync(0xffffffffu, mbar_wait(v_empty, (j & 1) ^ 1))) { raise_error(1); break; }
             if (elect_one()) {
-                mbar_expect_tx(v_full, KV_TILE);
+                mbar_expect_tx(v_full, V_TILE);
                 for (int h = 0; h < NPG; h++)
-                    for (int c = 0; c < CH; c++) tma_load_2d(vt + c * (KEYS * 128) + h * (PAGE * 128), &tmV, c * 64, y[h], v_full);
+                    for (int c = 0; c < CHV; c++) tma_load_2d(vt + c * (KEYS * 128) + h * (PAGE * 128), &tmV, c * 64, y[h], v_full);
             }
             __syncwarp();
             v_issued = j + 1;
@@ -344,7 +348,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         // ------------------------------------------------------------ MMA issuer
         // the whole warp walks the iterations and waits; one elected lane issues
         if (n_iter > 0) {
-            const uint32_t idesc_s = make_idesc(ROWS, KEYS, 0), idesc_o = make_idesc(ROWS, HD, 1);
+            const uint32_t idesc_s = make_idesc(ROWS, KEYS, 0), idesc_o = make_idesc(ROWS, HV, 1);
             auto issue_s = [&](int j) {
                 if (!__all_sync(0xffffffffu, mbar_wait(k_full, j & 1))) { raise_error(2); return false; }
                 tc_fence_after();
@@ -374,7 +378,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
                         uint64_t adesc = desc_k_major(ps + tile_of(j) * P_TILE + (ks >> 2) * (ROWS * 128) + (ks & 3) * 32);
                         uint64_t bdesc = desc_mn_major(vt + ks * 2048, KEYS * 128);
                         // O accumulates over the iterations (PP: over those of the iteration's set, in that set's columns)
-                        if (PP) tc_mma_bf16(tmem_base + O_COL + (j & 1) * HD, adesc, bdesc, idesc_o, ((j >> 1) | ks) != 0);
+                        if (PP) tc_mma_bf16(tmem_base + O_COL + (j & 1) * HV, adesc, bdesc, idesc_o, ((j >> 1) | ks) != 0);
                         else tc_mma_bf16(tmem_base + O_COL, adesc, bdesc, idesc_o, (j | ks) != 0);
                     }
                     tc_commit(PP ? o_full + 8 * (j & 1) : o_full);
@@ -390,7 +394,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         const int lg = warp & 3, r = lg * 32 + lane, set = PP ? (warp - 2) >> 2 : 0;
         const int step = PP ? 2 : 1;                    // this thread's iterations: set, set + step, ...
         const uint32_t trow = tmem_base + ((uint32_t)(lg * 32) << 16);
-        const uint32_t ocol = O_COL + set * HD, my_o_full = o_full + 8 * set;
+        const uint32_t ocol = O_COL + set * HV, my_o_full = o_full + 8 * set;
         // the wait for the P V of this thread's previous iteration names a phase by its parity: PP counts the set's own
         auto o_parity = [&](int j_prev) { return (uint32_t)((PP ? j_prev >> 1 : j_prev) & 1); };
         float m = -INFINITY, l = 0.f;
@@ -498,7 +502,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
                 if (!PIPE && !mbar_wait(my_o_full, o_parity(j_last))) { raise_error(5); ok = false; break; }
                 tc_fence_after();
 #pragma unroll 1
-                for (int c = 0; c < HD / 32; c++) {
+                for (int c = 0; c < HV / 32; c++) {
                     float v[32];
                     tc_ld32(trow + ocol + c * 32, v);
 #pragma unroll
@@ -528,21 +532,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         tc_fence_after();
         if (n_iter > 0 && __all_sync(0xffffffffu, ok)) {           // the tensor-memory loads are warp-wide: every lane takes part
             const float inv = l > 0.f ? 1.0f / l : 0.f;
-            bf16 *dst = out + (size_t)(row0 + q0 + t_row) * ldo + (size_t)(kvh * G + g_row) * HD;
+            const size_t at = (size_t)(row0 + q0 + t_row) * ldo + (size_t)(kvh * G + g_row) * HV;
             // (PP: each set stores half of the row's columns, from both accumulators)
 #pragma unroll 1
-            for (int c = PP ? set * (HD / 64) : 0; c < (PP ? (set + 1) * (HD / 64) : HD / 32); c++) {
+            for (int c = PP ? set * (HV / 64) : 0; c < (PP ? (set + 1) * (HV / 64) : HV / 32); c++) {
                 float v[32];
                 if (!PP) tc_ld32(trow + O_COL + c * 32, v);
                 else {
                     float a[32], b2[32];
-                    tc_ld32(trow + O_COL + set * HD + c * 32, a);              // this set's accumulator (set 0 always has one)
+                    tc_ld32(trow + O_COL + set * HV + c * 32, a);              // this set's accumulator (set 0 always has one)
                     const bool have_own = set == 0 || n_iter > 1, have_other = n_other > 0;
-                    if (have_other) tc_ld32(trow + O_COL + (set ^ 1) * HD + c * 32, b2);
+                    if (have_other) tc_ld32(trow + O_COL + (set ^ 1) * HV + c * 32, b2);
 #pragma unroll
                     for (int i = 0; i < 32; i++) v[i] = (have_own ? a[i] * w_own : 0.f) + (have_other ? b2[i] * w_other : 0.f);
                 }
                 if (!valid) continue;
+                if (out_f32) {
+#pragma unroll
+                    for (int k4 = 0; k4 < 8; k4++)
+                        *(float4 *)((float *)out + at + c * 32 + k4 * 4) = make_float4(v[4 * k4] * inv, v[4 * k4 + 1] * inv, v[4 * k4 + 2] * inv, v[4 * k4 + 3] * inv);
+                    continue;
+                }
 #pragma unroll
                 for (int k8 = 0; k8 < 4; k8++) {
                     uint32_t w[4];
@@ -551,7 +561,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
                         __nv_bfloat162 t = __floats2bfloat162_rn(v[k8 * 8 + 2 * k] * inv, v[k8 * 8 + 2 * k + 1] * inv);
                         w[k] = *(uint32_t *)&t;
                     }
-                    *(uint4 *)(dst + c * 32 + k8 * 8) = make_uint4(w[0], w[1], w[2], w[3]);
+                    *(uint4 *)((bf16 *)out + at + c * 32 + k8 * 8) = make_uint4(w[0], w[1], w[2], w[3]);
                 }
             }
         }
@@ -595,47 +605,48 @@ static int pool_map(CUtensorMap *map, const void *pool, long long rows, int hd) 
     return r == CUDA_SUCCESS ? 0 : FG_ERR_TENSORMAP;
 }
 
-template <int HD, bool PIPE, bool PP>
+template <int HD, int HV, bool PIPE, bool PP>
 static int launch_tc(const CUtensorMap &tmK, const CUtensorMap &tmV, const void *q, int ldq, void *out, int ldo,
                      const int *cu_rows, const int *seq_start, const int *block_table, int table_width, int n_seq,
                      int max_new, int H, int KV, float scale, int window, int keep_first, float softcap, const float *sinks,
-                     cudaStream_t stream) {
-    constexpr int KEYS = PIPE ? 64 : (HD > 64 ? 64 : 128);
-    constexpr int smem = ROWS * HD * 2 + 2 * KEYS * HD * 2 + (PIPE ? 2 : 1) * ROWS * KEYS * 2 + 1024;
+                     int v_share, int out_f32, cudaStream_t stream) {
+    constexpr int KEYS = PIPE ? 64 : (HV > 64 ? 64 : 128);
+    constexpr int smem = ROWS * HD * 2 + KEYS * (HD + HV) * 2 + (PIPE ? 2 : 1) * ROWS * KEYS * 2 + 1024;
     // the attributes belong to the function on ONE device: set them once on every device that launches
     static bool configured[64] = {false};
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return FG_ERR_BAD_SIZE;
     if (!configured[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, PIPE, PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, HV, PIPE, PP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
-        cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, PIPE, PP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+        cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, HV, PIPE, PP>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
         configured[dev] = true;
     }
     int G = H / KV, Gc = G < 16 ? G : 16, TQ = ROWS / Gc;
     dim3 grid(KV * ((G + Gc - 1) / Gc), (max_new + TQ - 1) / TQ, n_seq);
-    return fg_launch(attn_prefill_tc_kernel<HD, PIPE, PP>, grid, dim3(ATT_THREADS(PP)), (size_t)smem, stream, tmK, tmV, (const bf16 *)q, ldq,
-                     (bf16 *)out, ldo, cu_rows, seq_start, block_table, table_width, KV, G, scale * LOG2E, window, keep_first, g_test_skip_copy,
-                     softcap > 0.f ? softcap * LOG2E : 0.f, softcap > 0.f ? scale / softcap : 0.f, sinks);
+    return fg_launch(attn_prefill_tc_kernel<HD, HV, PIPE, PP>, grid, dim3(ATT_THREADS(PP)), (size_t)smem, stream, tmK, tmV, (const bf16 *)q, ldq,
+                     out, ldo, cu_rows, seq_start, block_table, table_width, KV, G, scale * LOG2E, window, keep_first, g_test_skip_copy,
+                     softcap > 0.f ? softcap * LOG2E : 0.f, softcap > 0.f ? scale / softcap : 0.f, sinks, v_share, out_f32);
 }
 
-// Arguments as fg_attention_prefill_kept, plus the number of pages in the pools.  Takes HD 64 and 128.
+// Arguments as fg_attention_prefill_kept, plus the number of pages in the pools.  Takes HD 64 and 128, values hdv of the same
+// size or 128 beside 64 (v_share key heads to a value head; out_f32: float32 output).
 // softcap > 0: capped scores; sinks (or null): a float per query head that joins the softmax's denominator.
 extern "C" int fg_attention_prefill_tc_ext(const void *q, int ldq, void *out, int ldo, const int *cu_rows,
                                            const int *seq_start, const int *block_table, int table_width,
                                            const void *k_pool, const void *v_pool, int n_pages, int n_seq, int max_new,
                                            int H, int KV, int hd, int page_size, float scale, int window, int keep_first,
-                                           float softcap, const float *sinks, cudaStream_t stream) {
+                                           float softcap, const float *sinks, int hdv, int v_share, int out_f32,
+                                           cudaStream_t stream) {
     if (n_seq <= 0 || max_new <= 0) return 0;
-    if (softcap < 0.f) return FG_ERR_BAD_SIZE;
+    if (softcap < 0.f || v_share <= 0 || KV % v_share || (hdv != hd && !(hd == 64 && hdv == 128))) return FG_ERR_BAD_SIZE;
     if (keep_first < 0 || page_size != PAGE || H % KV || n_seq > 65535 || ldq % 8 || ldo % 8 || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
         ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || (hd != 64 && hd != 128))
         return FG_ERR_BAD_SIZE;
     CUtensorMap tmK, tmV;
-    long long rows = (long long)n_pages * KV * PAGE;
-    int e = pool_map(&tmK, k_pool, rows, hd);
+    int e = pool_map(&tmK, k_pool, (long long)n_pages * KV * PAGE, hd);
     if (e) return e;
-    e = pool_map(&tmV, v_pool, rows, hd);
+    e = pool_map(&tmV, v_pool, (long long)n_pages * (KV / v_share) * PAGE, hdv);
     if (e) return e;
     // Which form runs.  Two score tiles (S of iteration j + 1 under the softmax of iteration j, P V of iteration j under
     // the softmax of j + 1): always - at head size 128 it took a fifth off the kernel (3B shapes, 2,048 tokens: 81 -> 62
@@ -647,10 +658,11 @@ extern "C" int fg_attention_prefill_tc_ext(const void *q, int ldq, void *out, in
     if (g_variant == -2) { const char *e = getenv("FASTGGUF_ATTN_PIPE"); g_variant = e ? atoi(e) : -1; }
     const bool pipe = g_variant >= 0 ? ((g_variant >> (hd == 64 ? 0 : 1)) & 1) != 0 : true;
     const bool pp = hd == 64 && pipe && (g_variant >= 0 ? (g_variant & 4) != 0 : (long long)n_seq * max_new >= 3072);
-#define TC_RUN(HD, PIPE, PP) launch_tc<HD, PIPE, PP>(tmK, tmV, q, ldq, out, ldo, cu_rows, seq_start, block_table, table_width, \
-                                                     n_seq, max_new, H, KV, scale, window, keep_first, softcap, sinks, stream)
-    if (hd == 64) return pipe ? (pp ? TC_RUN(64, true, true) : TC_RUN(64, true, false)) : TC_RUN(64, false, false);
-    return pipe ? TC_RUN(128, true, false) : TC_RUN(128, false, false);
+#define TC_RUN(HD, HV, PIPE, PP) launch_tc<HD, HV, PIPE, PP>(tmK, tmV, q, ldq, out, ldo, cu_rows, seq_start, block_table, table_width, \
+                                                     n_seq, max_new, H, KV, scale, window, keep_first, softcap, sinks, v_share, out_f32, stream)
+    if (hd == 64 && hdv == 128) return TC_RUN(64, 128, true, false);
+    if (hd == 64) return pipe ? (pp ? TC_RUN(64, 64, true, true) : TC_RUN(64, 64, true, false)) : TC_RUN(64, 64, false, false);
+    return pipe ? TC_RUN(128, 128, true, false) : TC_RUN(128, 128, false, false);
 #undef TC_RUN
 }
 
@@ -660,7 +672,7 @@ extern "C" int fg_attention_prefill_tc_kept(const void *q, int ldq, void *out, i
                                             int H, int KV, int hd, int page_size, float scale, int window, int keep_first,
                                             cudaStream_t stream) {
     return fg_attention_prefill_tc_ext(q, ldq, out, ldo, cu_rows, seq_start, block_table, table_width, k_pool, v_pool, n_pages, n_seq,
-                                       max_new, H, KV, hd, page_size, scale, window, keep_first, 0.f, nullptr, stream);
+                                       max_new, H, KV, hd, page_size, scale, window, keep_first, 0.f, nullptr, hd, 1, 0, stream);
 }
 
 extern "C" int fg_attention_prefill_tc(const void *q, int ldq, void *out, int ldo, const int *cu_rows,

@@ -23,14 +23,14 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
                    const float *__restrict__ cos_t, const float *__restrict__ sin_t, int tbl_half, int rot_dims,
                    const int *__restrict__ positions, const int *__restrict__ row_seq, const int *__restrict__ cu_rows,
                    const int *__restrict__ slots, const int *__restrict__ block_table, int table_width, T *__restrict__ q_out, int ldq,
-                   T *__restrict__ k_pool, T *__restrict__ v_pool, int H, int KV, int hd, int hdv, int page_size, int norm_per_head,
-                   int rot_halves) {
+                   T *__restrict__ k_pool, T *__restrict__ v_pool, int H, int KV, int VH, int hd, int hdv, int page_size, int norm_per_head,
+                   int rot_halves, int v_from_k) {
     extern __shared__ float row[];
     __shared__ float scratch[32];
     pdl_launch_dependents_small_step(gridDim.x);
     pdl_wait();
     const int m = blockIdx.x, tid = threadIdx.x, nthr = blockDim.x;
-    const int Cq = H * hd, Ck = KV * hd, C = Cq + Ck + KV * hdv;
+    const int Cq = H * hd, Ck = KV * hd, C = Cq + Ck + (v_from_k ? 0 : VH * hdv);
     const int seq = row_seq[m], pos = positions[m];
     const int i_step = m - cu_rows[seq];                 // the token's index among the step's tokens of its sequence
     const float *mine = proj + (size_t)m * ld;
@@ -52,6 +52,15 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
         for (int c = tid; c < C; c += nthr) row[c] = mine[c] + (bias ? bias[c] : 0.f);
     }
     __syncthreads();
+    if (v_from_k && v_pool) {
+        // the values are the keys as projected (bias included), before norm and rotation
+        const int page = block_table[(size_t)seq * table_width + pos / page_size], off = pos % page_size;
+        for (int c = tid; c < Ck; c += nthr) {
+            const int vh = c / hdv, d = c - vh * hdv;
+            v_pool[(((size_t)page * VH + vh) * page_size + off) * hdv + d] = from_f32<T>(row[Cq + c]);
+        }
+        __syncthreads();
+    }
     if (qn_w && norm_per_head) {
         // every head of q and of k by itself: x / sqrt(mean(x^2) + eps) * w with ONE weight vector [hd] for all heads of q and
         // one for all heads of k; a warp takes a head, its lanes the head's numbers, the sum by a shuffle tree
@@ -98,9 +107,9 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
             const int kvh = c / hd, d = c - kvh * hd;
             k_pool[(((size_t)page * KV + kvh) * page_size + off) * hd + d] = from_f32<T>(row[Cq + c]);
         }
-        for (int c = tid; c < KV * hdv; c += nthr) {
-            const int kvh = c / hdv, d = c - kvh * hdv;
-            v_pool[(((size_t)page * KV + kvh) * page_size + off) * hdv + d] = from_f32<T>(row[Cq + Ck + c]);
+        for (int c = tid; c < (v_from_k ? 0 : VH * hdv); c += nthr) {
+            const int vh = c / hdv, d = c - vh * hdv;
+            v_pool[(((size_t)page * VH + vh) * page_size + off) * hdv + d] = from_f32<T>(row[Cq + Ck + c]);
         }
     }
 }
@@ -370,17 +379,22 @@ head_gemv_kernel(const void *__restrict__ A, int a_dtype, int lda, int a_stride,
 }
 
 // norm_per_head: the norm weights are [hd] and every head of q and of k is normalised by itself (else: [H * hd] / [KV * hd], the
-// whole of q and of k at once); rot_halves: a rotated pair is (i, i + rot_dims / 2) of a head (else (2i, 2i + 1))
+// whole of q and of k at once); rot_halves: a rotated pair is (i, i + rot_dims / 2) of a head (else (2i, 2i + 1)); v_heads (0: KV):
+// heads of values, where several key heads share one; v_from_k: there is no value projection, the values are the keys as projected
 extern "C" int fg_qkv_prepare_ext(const float *proj, int ld, const float *bias, const float *conv_w, int taps, const float *conv_state,
                                   const float *qn_w, const float *kn_w, float eps, const float *cos_t, const float *sin_t, int tbl_half,
                                   int rot_dims, const int *positions, const int *row_seq, const int *cu_rows, const int *slots,
                                   const int *block_table, int table_width, void *q_out, int ldq, void *k_pool, void *v_pool, int dtype, int M,
-                                  int H, int KV, int hd, int hdv, int page_size, int norm_per_head, int rot_halves, cudaStream_t stream) {
+                                  int H, int KV, int hd, int hdv, int page_size, int norm_per_head, int rot_halves, int v_heads, int v_from_k,
+                                  cudaStream_t stream) {
     if (M <= 0) return 0;
+    const int VH = v_heads > 0 ? v_heads : KV;
+    if (v_from_k && (conv_w || VH != KV || hdv != hd)) return FG_ERR_BAD_SIZE;
     if (H <= 0 || KV <= 0 || hd <= 0 || hdv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > hd || rot_dims / 2 > tbl_half) return FG_ERR_BAD_SIZE;
     if (conv_w && (taps < 1 || (taps > 1 && !conv_state))) return FG_ERR_BAD_SIZE;
     if ((qn_w == nullptr) != (kn_w == nullptr)) return FG_ERR_BAD_SIZE;
-    const size_t smem = ((size_t)H * hd + (size_t)KV * (hd + hdv)) * sizeof(float);
+    const int C_all = H * hd + KV * hd + (v_from_k ? 0 : VH * hdv);
+    const size_t smem = (size_t)C_all * sizeof(float);
     if (smem > 200 * 1024) return FG_ERR_BAD_SIZE;
     static FgPerDevice setup[2];
     if (smem > 48 * 1024 && fg_needs_setup(setup[dtype == FG_F32 ? 0 : 1])) {
@@ -389,16 +403,15 @@ extern "C" int fg_qkv_prepare_ext(const float *proj, int ld, const float *bias, 
         if (e != cudaSuccess) return (int)e;
     }
     // few rows (a decode step) leave most of the GPU idle: a row's channels are then spread over more threads
-    const int C_all = H * hd + KV * (hd + hdv);
     const int threads = (M < 64 && C_all >= 2048) ? 1024 : PREP_THREADS;
     if (dtype == FG_F32)
         return fg_launch(qkv_prepare_kernel<float>, dim3(M), dim3(threads), smem, stream, proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w,
                          eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq, cu_rows, slots, block_table, table_width, (float *)q_out,
-                         ldq, (float *)k_pool, (float *)v_pool, H, KV, hd, hdv, page_size, norm_per_head, rot_halves);
+                         ldq, (float *)k_pool, (float *)v_pool, H, KV, VH, hd, hdv, page_size, norm_per_head, rot_halves, v_from_k);
     if (dtype == FG_BF16)
         return fg_launch(qkv_prepare_kernel<bf16>, dim3(M), dim3(threads), smem, stream, proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w,
                          eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq, cu_rows, slots, block_table, table_width, (bf16 *)q_out, ldq,
-                         (bf16 *)k_pool, (bf16 *)v_pool, H, KV, hd, hdv, page_size, norm_per_head, rot_halves);
+                         (bf16 *)k_pool, (bf16 *)v_pool, H, KV, VH, hd, hdv, page_size, norm_per_head, rot_halves, v_from_k);
     return FG_ERR_BAD_DTYPE;
 }
 
@@ -408,7 +421,62 @@ extern "C" int fg_qkv_prepare(const float *proj, int ld, const float *bias, cons
                               const int *block_table, int table_width, void *q_out, int ldq, void *k_pool, void *v_pool, int dtype, int M,
                               int H, int KV, int hd, int hdv, int page_size, cudaStream_t stream) {
     return fg_qkv_prepare_ext(proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w, eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq,
-                              cu_rows, slots, block_table, table_width, q_out, ldq, k_pool, v_pool, dtype, M, H, KV, hd, hdv, page_size, 0, 0, stream);
+                              cu_rows, slots, block_table, table_width, q_out, ldq, k_pool, v_pool, dtype, M, H, KV, hd, hdv, page_size, 0, 0, 0, 0, stream);
+}
+
+// ------------------------------------------------------------------ the difference of two maps' outputs
+// maps [M, 2 H * dv] float32, heads in the order [key head g][map][head i of the group]: with a1, a2 the two maps' outputs of a head,
+// o = a1 - lambda a2, out = o / sqrt(mean(o^2) + eps) * gain over the head's dv values; out's heads are g * R + i.  A warp a head.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(PREP_THREADS)
+differential_combine_kernel(const float *__restrict__ maps, int ld, T *__restrict__ out, int ldo, int H, int R, int dv, float lambda, float eps,
+                            float gain) {
+    pdl_launch_dependents_small_step(gridDim.x);
+    pdl_wait();
+    const int m = blockIdx.x, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    for (int h = blockIdx.y * n_warps + (threadIdx.x >> 5); h < H; h += gridDim.y * n_warps) {
+        const int g = h / R, i = h - g * R;
+        const float *a1 = maps + (size_t)m * ld + (size_t)(2 * g * R + i) * dv, *a2 = a1 + (size_t)R * dv;
+        T *o = out + (size_t)m * ldo + (size_t)h * dv;
+        float ss = 0.f;
+        if (VEC) {
+            for (int d = lane * 4; d < dv; d += 128) {
+                const float4 x = *(const float4 *)(a1 + d), y = *(const float4 *)(a2 + d);
+                const float p = fmaf(-lambda, y.x, x.x), q = fmaf(-lambda, y.y, x.y), r = fmaf(-lambda, y.z, x.z), s = fmaf(-lambda, y.w, x.w);
+                ss += p * p; ss += q * q; ss += r * r; ss += s * s;
+            }
+        } else {
+            for (int d = lane; d < dv; d += 32) { const float p = fmaf(-lambda, a2[d], a1[d]); ss += p * p; }
+        }
+        const float inv = gain / sqrtf(warp_sum(ss) / (float)dv + eps);
+        if (VEC) {
+            for (int d = lane * 4; d < dv; d += 128) {
+                const float4 x = *(const float4 *)(a1 + d), y = *(const float4 *)(a2 + d);
+                const float p = fmaf(-lambda, y.x, x.x) * inv, q = fmaf(-lambda, y.y, x.y) * inv, r = fmaf(-lambda, y.z, x.z) * inv, s = fmaf(-lambda, y.w, x.w) * inv;
+                if (sizeof(T) == 4) *(float4 *)(o + d) = make_float4(p, q, r, s);
+                else {
+                    __nv_bfloat162 lo = __floats2bfloat162_rn(p, q), hi = __floats2bfloat162_rn(r, s);
+                    *(uint2 *)(o + d) = make_uint2(*(uint32_t *)&lo, *(uint32_t *)&hi);
+                }
+            }
+        } else {
+            for (int d = lane; d < dv; d += 32) o[d] = from_f32<T>(fmaf(-lambda, a2[d], a1[d]) * inv);
+        }
+    }
+}
+
+extern "C" int fg_differential_combine(const float *maps, int ld, void *out, int out_dtype, int ldo, int M, int H, int KV, int dv, float lambda,
+                                       float eps, float gain, cudaStream_t stream) {
+    if (M <= 0) return 0;
+    if (H <= 0 || KV <= 0 || H % KV || dv <= 0) return FG_ERR_BAD_SIZE;
+    const bool vec = dv % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && ((((uintptr_t)maps) | ((uintptr_t)out)) & 15) == 0;
+    const dim3 grid(M, (H + 7) / 8);
+#define DIFF_LAUNCH(T, VEC) fg_launch(differential_combine_kernel<T, VEC>, grid, dim3(PREP_THREADS), 0, stream, maps, ld, (T *)out, ldo, H, H / KV, dv, lambda, \
+                                      eps, gain)
+    if (out_dtype == FG_F32) return vec ? DIFF_LAUNCH(float, true) : DIFF_LAUNCH(float, false);
+    if (out_dtype == FG_BF16) return vec ? DIFF_LAUNCH(bf16, true) : DIFF_LAUNCH(bf16, false);
+#undef DIFF_LAUNCH
+    return FG_ERR_BAD_DTYPE;
 }
 
 // ------------------------------------------------------------------ a gate per head on the heads' outputs

@@ -11,27 +11,33 @@
 
 // ------------------------------------------------------------------ embedding gather
 template <typename TW>
-__global__ void embed_gather_kernel(const TW *__restrict__ table, const int *__restrict__ tokens,
+__global__ void embed_gather_kernel(const TW *__restrict__ table, const int *__restrict__ tokens, const float *__restrict__ add_row,
                                     float *__restrict__ x, int E, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     int m = blockIdx.x;
     const TW *row = table + (size_t)tokens[m] * E;
     float *out = x + (size_t)m * E;
-    for (int i = threadIdx.x; i < E; i += blockDim.x) out[i] = to_f32<TW>(row[i]) * scale;
+    for (int i = threadIdx.x; i < E; i += blockDim.x) out[i] = to_f32<TW>(row[i]) * scale + (add_row ? add_row[i] : 0.f);
 }
 
 // x = table[token] * scale (embd_scale of the reference, fastgguf.c:4652; 1 for most models)
-extern "C" int fg_embed_gather_scaled(const void *table, int table_dtype, const int *tokens, float *x,
-                                      int M, int E, float scale, cudaStream_t stream) {
+// add_row ([E] or null): added to every row
+extern "C" int fg_embed_gather_row(const void *table, int table_dtype, const int *tokens, const float *add_row, float *x,
+                                   int M, int E, float scale, cudaStream_t stream) {
     if (M <= 0) return 0;
     int threads = E >= 1024 ? 256 : 128;
     if (table_dtype == FG_F32)
-        return fg_launch(embed_gather_kernel<float>, dim3(M), dim3(threads), 0, stream, (const float *)table, tokens, x, E, scale);
+        return fg_launch(embed_gather_kernel<float>, dim3(M), dim3(threads), 0, stream, (const float *)table, tokens, add_row, x, E, scale);
     else if (table_dtype == FG_BF16)
-        return fg_launch(embed_gather_kernel<bf16>, dim3(M), dim3(threads), 0, stream, (const bf16 *)table, tokens, x, E, scale);
+        return fg_launch(embed_gather_kernel<bf16>, dim3(M), dim3(threads), 0, stream, (const bf16 *)table, tokens, add_row, x, E, scale);
     else return FG_ERR_BAD_DTYPE;
     return FG_LAUNCH_CHECK();
+}
+
+extern "C" int fg_embed_gather_scaled(const void *table, int table_dtype, const int *tokens, float *x,
+                                      int M, int E, float scale, cudaStream_t stream) {
+    return fg_embed_gather_row(table, table_dtype, tokens, nullptr, x, M, E, scale, stream);
 }
 
 extern "C" int fg_embed_gather(const void *table, int table_dtype, const int *tokens, float *x,
@@ -42,7 +48,7 @@ extern "C" int fg_embed_gather(const void *table, int table_dtype, const int *to
 // The same gather that also starts a deferred RMSNorm: xw = bf16(x * norm_w) and the row's sum of squares
 // (one "tile"), for a contraction that applies 1/rms in its epilogue.
 template <typename TW>
-__global__ void embed_gather_norm_kernel(const TW *__restrict__ table, const int *__restrict__ tokens,
+__global__ void embed_gather_norm_kernel(const TW *__restrict__ table, const int *__restrict__ tokens, const float *__restrict__ add_row,
                                          float *__restrict__ x, const float *__restrict__ norm_w,
                                          bf16 *__restrict__ xw, float *__restrict__ ss, int E) {
     __shared__ float scratch[32];
@@ -52,7 +58,7 @@ __global__ void embed_gather_norm_kernel(const TW *__restrict__ table, const int
     const TW *row = table + (size_t)tokens[m] * E;
     float acc = 0.f;
     for (int i = threadIdx.x; i < E; i += blockDim.x) {
-        float v = to_f32<TW>(row[i]);
+        float v = to_f32<TW>(row[i]) + (add_row ? add_row[i] : 0.f);
         x[(size_t)m * E + i] = v;
         xw[(size_t)m * E + i] = __float2bfloat16_rn(v * norm_w[i]);
         acc += v * v;
@@ -61,17 +67,36 @@ __global__ void embed_gather_norm_kernel(const TW *__restrict__ table, const int
     if (threadIdx.x == 0) ss[m] = acc;
 }
 
-extern "C" int fg_embed_gather_norm(const void *table, int table_dtype, const int *tokens, float *x,
-                                    const float *norm_w, void *xw, float *ss, int M, int E, cudaStream_t stream) {
+extern "C" int fg_embed_gather_norm_row(const void *table, int table_dtype, const int *tokens, const float *add_row, float *x,
+                                        const float *norm_w, void *xw, float *ss, int M, int E, cudaStream_t stream) {
     if (M <= 0) return 0;
     int threads = E >= 1024 ? 256 : 128;
     if (table_dtype == FG_F32)
-        return fg_launch(embed_gather_norm_kernel<float>, dim3(M), dim3(threads), 0, stream, (const float *)table, tokens, x,
+        return fg_launch(embed_gather_norm_kernel<float>, dim3(M), dim3(threads), 0, stream, (const float *)table, tokens, add_row, x,
                          norm_w, (bf16 *)xw, ss, E);
     if (table_dtype == FG_BF16)
-        return fg_launch(embed_gather_norm_kernel<bf16>, dim3(M), dim3(threads), 0, stream, (const bf16 *)table, tokens, x,
+        return fg_launch(embed_gather_norm_kernel<bf16>, dim3(M), dim3(threads), 0, stream, (const bf16 *)table, tokens, add_row, x,
                          norm_w, (bf16 *)xw, ss, E);
     return FG_ERR_BAD_DTYPE;
+}
+
+extern "C" int fg_embed_gather_norm(const void *table, int table_dtype, const int *tokens, float *x,
+                                    const float *norm_w, void *xw, float *ss, int M, int E, cudaStream_t stream) {
+    return fg_embed_gather_norm_row(table, table_dtype, tokens, nullptr, x, norm_w, xw, ss, M, E, stream);
+}
+
+// ------------------------------------------------------------------ one vector for every row
+// x[m, :] += row: the stream in front of a pass of a looped span
+__global__ void add_row_kernel(float *__restrict__ x, const float *__restrict__ row, int E) {
+    pdl_launch_dependents_small_step(gridDim.x);
+    pdl_wait();
+    float *xi = x + (size_t)blockIdx.x * E;
+    for (int i = threadIdx.x; i < E; i += blockDim.x) xi[i] += row[i];
+}
+
+extern "C" int fg_add_row(float *x, const float *row, int M, int E, cudaStream_t stream) {
+    if (M <= 0 || E <= 0) return 0;
+    return fg_launch(add_row_kernel, dim3(M), dim3(E >= 1024 ? 256 : 128), 0, stream, x, row, E);
 }
 
 // ------------------------------------------------------------------ RMSNorm
@@ -295,9 +320,10 @@ extern "C" int fg_kv_append(const void *qkv, int dtype, int ld, int k_off, const
 // when w_next is given, out[m] = x[m] / rms(x[m]) * w_next for the sublayer that reads x next - one pass over
 // the row instead of three kernels.  Statistics and the sum are 32-bit; one block a row, fixed reduction order.
 // Without w_next, out (when given) receives the updated x[m] itself: the input of a sublayer that reads the stream as it is.
+// add_row ([E] or null) joins every row of x in the same sum.
 // VEC: rows are read and written four elements at a time (E % 4 == 0, 16-byte aligned rows)
 template <typename TO, bool VEC>
-__global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *__restrict__ w_post, float *__restrict__ x,
+__global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *__restrict__ w_post, const float *__restrict__ add_row, float *__restrict__ x,
                                      const float *__restrict__ w_next, TO *__restrict__ out, int E, float eps_post,
                                      float eps_next) {
     __shared__ float scratch[32];
@@ -321,6 +347,7 @@ __global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *_
         for (int i = threadIdx.x; i < E / 4; i += blockDim.x) {
             float4 a = t4[i], g = w4[i], v = x4[i];
             v.x += a.x * inv * g.x; v.y += a.y * inv * g.y; v.z += a.z * inv * g.z; v.w += a.w * inv * g.w;
+            if (add_row) { const float4 b = ((const float4 *)add_row)[i]; v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
             x4[i] = v;
             if (w_next) { r4[i] = v; ss2 += v.x * v.x; ss2 += v.y * v.y; ss2 += v.z * v.z; ss2 += v.w * v.w; }
             else if (out) store4<TO>(out + base + 4 * i, v.x, v.y, v.z, v.w);
@@ -328,6 +355,7 @@ __global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *_
     } else {
         for (int i = threadIdx.x; i < E; i += blockDim.x) {
             float v = x[base + i] + t[base + i] * inv * w_post[i];
+            if (add_row) v += add_row[i];
             x[base + i] = v;
             if (w_next) { row[i] = v; ss2 += v * v; }
             else if (out) out[base + i] = from_f32<TO>(v);
@@ -347,21 +375,26 @@ __global__ void norm_add_norm_kernel(const float *__restrict__ t, const float *_
     }
 }
 
-extern "C" int fg_norm_add_norm(const float *t, const float *w_post, float *x, const float *w_next, void *out, int out_dtype,
-                                int M, int E, float eps_post, float eps_next, cudaStream_t stream) {
+extern "C" int fg_norm_add_norm_row(const float *t, const float *w_post, const float *add_row, float *x, const float *w_next, void *out, int out_dtype,
+                                    int M, int E, float eps_post, float eps_next, cudaStream_t stream) {
     if (M <= 0) return 0;
     size_t smem = w_next ? (size_t)E * sizeof(float) : 0;
     if (smem > 48 * 1024) return FG_ERR_BAD_SIZE;
-    const bool vec = E % 4 == 0 && ((((uintptr_t)t) | ((uintptr_t)w_post) | ((uintptr_t)x) | ((uintptr_t)w_next) | ((uintptr_t)out)) & 15) == 0;
+    const bool vec = E % 4 == 0 && ((((uintptr_t)t) | ((uintptr_t)w_post) | ((uintptr_t)x) | ((uintptr_t)w_next) | ((uintptr_t)out) | ((uintptr_t)add_row)) & 15) == 0;
     int per = vec ? E / 4 : E;
     int threads = per >= 1024 ? 256 : (per >= 256 ? 128 : 64);
     const bool wide = out_dtype == FG_F32 || (!w_next && !out);
     if (!wide && out_dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
-#define NAN_LAUNCH(TO, VEC) fg_launch(norm_add_norm_kernel<TO, VEC>, dim3(M), dim3(threads), smem, stream, t, w_post, x, w_next, (TO *)out, E, \
+#define NAN_LAUNCH(TO, VEC) fg_launch(norm_add_norm_kernel<TO, VEC>, dim3(M), dim3(threads), smem, stream, t, w_post, add_row, x, w_next, (TO *)out, E, \
                                       eps_post, eps_next)
     if (wide) return vec ? NAN_LAUNCH(float, true) : NAN_LAUNCH(float, false);
     return vec ? NAN_LAUNCH(bf16, true) : NAN_LAUNCH(bf16, false);
 #undef NAN_LAUNCH
+}
+
+extern "C" int fg_norm_add_norm(const float *t, const float *w_post, float *x, const float *w_next, void *out, int out_dtype,
+                                int M, int E, float eps_post, float eps_next, cudaStream_t stream) {
+    return fg_norm_add_norm_row(t, w_post, nullptr, x, w_next, out, out_dtype, M, E, eps_post, eps_next, stream);
 }
 
 // ------------------------------------------------------------------ two mixers side by side
@@ -448,12 +481,12 @@ extern "C" int fg_softcap(float *logits, int R, int V, int ld, float cap, cudaSt
 }
 
 // ------------------------------------------------------------------ act(g) * u
-// gu: [M, 2F] rows of (gate | up); out: [M, F].  act: SiLU, or the tanh form of gelu.
+// gu: [M, 2F] rows of (gate | up); out: [M, F].  act: SiLU (0), the tanh form of gelu (1), or max(., 0) (2).
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-template <typename T, bool GELU>
+template <typename T, int ACT>
 __global__ void gated_mul_kernel(const T *__restrict__ gu, T *__restrict__ out, size_t total, int F) {
     pdl_launch_dependents();
     pdl_wait();
@@ -463,11 +496,11 @@ __global__ void gated_mul_kernel(const T *__restrict__ gu, T *__restrict__ out, 
         size_t m = i / F;
         int f = (int)(i - m * F);
         float g = to_f32<T>(gu[m * 2 * F + f]), u = to_f32<T>(gu[m * 2 * F + F + f]);
-        out[i] = from_f32<T>(GELU ? gelu_tanh_f32(g) * u : g / (1.0f + expf(-g)) * u);
+        out[i] = from_f32<T>(ACT == 2 ? fmaxf(g, 0.f) * u : ACT == 1 ? gelu_tanh_f32(g) * u : g / (1.0f + expf(-g)) * u);
     }
 }
 
-template <bool GELU>
+template <int ACT>
 static int gated_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) {
     size_t total = (size_t)M * F;
     if (total == 0) return 0;
@@ -475,14 +508,15 @@ static int gated_mul(const void *gu, void *out, int dtype, int M, int F, cudaStr
     size_t want = (total + threads - 1) / threads;
     int blocks = (int)(want > 148 * 16 ? 148 * 16 : want);
     if (dtype == FG_F32)
-        return fg_launch(gated_mul_kernel<float, GELU>, dim3(blocks), dim3(threads), 0, stream, (const float *)gu, (float *)out, total, F);
+        return fg_launch(gated_mul_kernel<float, ACT>, dim3(blocks), dim3(threads), 0, stream, (const float *)gu, (float *)out, total, F);
     if (dtype == FG_BF16)
-        return fg_launch(gated_mul_kernel<bf16, GELU>, dim3(blocks), dim3(threads), 0, stream, (const bf16 *)gu, (bf16 *)out, total, F);
+        return fg_launch(gated_mul_kernel<bf16, ACT>, dim3(blocks), dim3(threads), 0, stream, (const bf16 *)gu, (bf16 *)out, total, F);
     return FG_ERR_BAD_DTYPE;
 }
 
-extern "C" int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<false>(gu, out, dtype, M, F, stream); }
-extern "C" int fg_gelu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<true>(gu, out, dtype, M, F, stream); }
+extern "C" int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<0>(gu, out, dtype, M, F, stream); }
+extern "C" int fg_gelu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<1>(gu, out, dtype, M, F, stream); }
+extern "C" int fg_relu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream) { return gated_mul<2>(gu, out, dtype, M, F, stream); }
 
 // ------------------------------------------------------------------ decode feedback
 // After a decode step of a fixed-shape (graph-replayed) batch: the sampled token of every row

@@ -24,6 +24,12 @@ extern "C" {
 int fg_embed_gather(const void *table, int table_dtype, const int *tokens, float *x, int M, int E, cudaStream_t stream);
 int fg_embed_gather_scaled(const void *table, int table_dtype, const int *tokens, float *x, int M, int E, float scale,
                            cudaStream_t stream);
+/* add_row: a vector [E] (or null) added to every row */
+int fg_embed_gather_row(const void *table, int table_dtype, const int *tokens, const float *add_row, float *x, int M, int E, float scale,
+                        cudaStream_t stream);
+int fg_embed_gather_norm_row(const void *table, int table_dtype, const int *tokens, const float *add_row, float *x, const float *norm_w,
+                             void *xw, float *ss, int M, int E, cudaStream_t stream);
+int fg_add_row(float *x, const float *row, int M, int E, cudaStream_t stream);
 int fg_embed_gather_norm(const void *table, int table_dtype, const int *tokens, float *x, const float *norm_w,
                          void *xw, float *ss, int M, int E, cudaStream_t stream);
 int fg_rmsnorm(const float *x, const float *w, const int *rows, void *out, int out_dtype, int R, int E, float eps,
@@ -36,6 +42,8 @@ int fg_kv_append(const void *qkv, int dtype, int ld, int k_off, const int *posit
                  const int *block_table, int table_width, void *k_pool, void *v_pool, int M, int KV, int hd, int hdv,
                  int page_size, cudaStream_t stream);
 /* x += t / rms(t) * w_post; with w_next also out = x / rms(x) * w_next (out_dtype) */
+int fg_norm_add_norm_row(const float *t, const float *w_post, const float *add_row, float *x, const float *w_next, void *out, int out_dtype,
+                         int M, int E, float eps_post, float eps_next, cudaStream_t stream);
 int fg_norm_add_norm(const float *t, const float *w_post, float *x, const float *w_next, void *out, int out_dtype,
                      int M, int E, float eps_post, float eps_next, cudaStream_t stream);
 int fg_activation(void *z, int dtype, long long total, int kind /* 0: relu(z)^2 */, cudaStream_t stream);
@@ -44,6 +52,7 @@ int fg_concat2(const float *a, int lda, const float *b, int ldb, void *out, int 
                cudaStream_t stream);
 int fg_silu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream);
 int fg_gelu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream);      /* the tanh form of gelu instead */
+int fg_relu_mul(const void *gu, void *out, int dtype, int M, int F, cudaStream_t stream);      /* max(gate, 0) * up */
 /* out (+)= scale_a * f_a(a) + scale_b * f_b(b) over float32 rows [M, E]; f(t) = t / rms(t) * w with a weight, t itself without */
 int fg_pair_combine(const float *a, const float *b, const float *w_a, const float *w_b, float scale_a, float scale_b, float eps,
                     float *out, int M, int E, int accumulate, cudaStream_t stream);
@@ -65,11 +74,12 @@ int fg_attention_generic(const void *q, int ldq, void *out, int ldo, int dtype, 
 /* the same with values of head size hdv and, with a window, the sequence's first keep_first keys visible as well */
 /* softcap > 0: scores capped by softcap * tanh(score / softcap); sinks: a float per query head that joins the softmax's denominator;
    latent: the cache holds a latent (v_pool, hdv numbers, also the value) and a rotated key part (k_pool, hd numbers) a position,
-   and a query head has hdv + hd numbers */
+   and a query head has hdv + hd numbers; v_share: that many neighbouring key heads share a value head; out_f32: float32 output */
 int fg_attention_generic_ext(const void *q, int ldq, void *out, int ldo, int dtype, const int *positions,
                              const int *row_seq, const int *block_table, int table_width, const void *k_pool,
                              const void *v_pool, int M, int H, int KV, int hd, int hdv, int page_size, float scale,
-                             int window, int keep_first, float softcap, const float *sinks, int latent, cudaStream_t stream);
+                             int window, int keep_first, float softcap, const float *sinks, int latent, int v_share, int out_f32,
+                             cudaStream_t stream);
 int fg_attention_generic_kept(const void *q, int ldq, void *out, int ldo, int dtype, const int *positions,
                               const int *row_seq, const int *block_table, int table_width, const void *k_pool,
                               const void *v_pool, int M, int H, int KV, int hd, int hdv, int page_size, float scale,
@@ -81,16 +91,17 @@ int fg_sample(float *logits, int B, int V, int ldl, float temp, int top_k, float
 int fg_argmax(const float *logits, int B, int V, int ldl, int *out, cudaStream_t stream);
 
 /* ---- libfg_mix: retention (linear attention with a fixed decay per head) and the mixture of experts */
-/* proj rows: q [H, dk] | k [H, dk] | v [H, dv] | g [H, dv] float32; state [slots, H, dk, dv] float32; out [M, H * dv] */
+/* proj rows: q [H, dk] | k [H, dk] | v [H, dv] | g [H, dv] float32; state [slots, H, dk, dv] float32; out [M, H * dv].  cos_t null: no
+   rotation; opts: 1 = silu on q, k and v, 2 = the sums o themselves, without unit norm and gate */
 int fg_retention(const float *proj, int ld, void *out, int out_dtype, int ldo, const int *positions, const int *cu_rows,
                  const int *slots, const float *cos_t, const float *sin_t, const float *decay, float *state, int n_seq,
-                 int H, int dk, int dv, float k_scale, float eps, cudaStream_t stream);
+                 int H, int dk, int dv, float k_scale, float eps, int opts, cudaStream_t stream);
 int fg_retention_chunk_tokens(void);
 int fg_retention_chunked_ok(int dk, int dv);
 int fg_retention_chunked(const float *proj, int ld, void *out, int out_dtype, int ldo, const int *positions,
                          const int *cu_rows, const int *slots, const float *cos_t, const float *sin_t,
                          const float *decay, float *state, int *plan, float *U, int n_seq, int n_chunks, int H, int dk,
-                         int dv, float k_scale, float eps, cudaStream_t stream);
+                         int dv, float k_scale, float eps, int opts, cudaStream_t stream);
 /* gated linear attention (gla.cu): proj rows q [H, dk] | k [H, dk] | v [H, dv] | g [H, dv] float32, z rows [H, dk] decay logits
    without their bias; state [slots, H, dk, dv] float32; out [M, H * dv] */
 int fg_gla(const float *proj, int ld, const float *z, int ldz, const float *z_bias, const float *norm_w, void *out, int out_dtype,
@@ -135,9 +146,10 @@ int fg_conv1d_state(const float *in, int ld, int taps, float *state, long long s
 int fg_decay_gates(const float *a_raw, int lda, const float *b_raw, int ldb, const float *A_log, const float *dt_bias, int mode,
                    float *decay, float *step, int M, int H, cudaStream_t stream);
 int fg_unit_heads(float *x, int ld, int n_heads, int d, float eps, float scale, int M, cudaStream_t stream);
-/* gate_first: t = y silu(g), out = t / rms(t) * w over groups of `group` channels; else out = y / rms(y) * w[c % w_period] * silu(g) */
+/* gate_first: t = y silu(g), out = t / rms(t) * w over groups of `group` channels; else out = y / rms(y) * w[c % w_period] * silu(g);
+   sigmoid_gate: sigmoid(g) for silu(g) */
 int fg_gated_group_norm(const float *y, int ldy, const float *g, int ldg, const float *w, int w_period, void *out, int out_dtype,
-                        int ldo, int M, int C, int group, float eps, int gate_first, cudaStream_t stream);
+                        int ldo, int M, int C, int group, float eps, int gate_first, int sigmoid_gate, cudaStream_t stream);
 /* between an attention mixer's projections and its attention kernel (attention_prep.cu) */
 int fg_qkv_prepare(const float *proj, int ld, const float *bias, const float *conv_w, int taps, const float *conv_state,
                    const float *qn_w, const float *kn_w, float eps, const float *cos_t, const float *sin_t, int tbl_half,
@@ -145,12 +157,16 @@ int fg_qkv_prepare(const float *proj, int ld, const float *bias, const float *co
                    const int *block_table, int table_width, void *q_out, int ldq, void *k_pool, void *v_pool, int dtype, int M,
                    int H, int KV, int hd, int hdv, int page_size, cudaStream_t stream);
 /* the same with the norm per head (weights [hd]) instead of over the whole of q and of k, and with rotated pairs
-   (i, i + rot_dims / 2) instead of (2i, 2i + 1) */
+   (i, i + rot_dims / 2) instead of (2i, 2i + 1); v_heads (0: KV) heads of values; v_from_k: the values are the keys as projected */
 int fg_qkv_prepare_ext(const float *proj, int ld, const float *bias, const float *conv_w, int taps, const float *conv_state,
                        const float *qn_w, const float *kn_w, float eps, const float *cos_t, const float *sin_t, int tbl_half,
                        int rot_dims, const int *positions, const int *row_seq, const int *cu_rows, const int *slots,
                        const int *block_table, int table_width, void *q_out, int ldq, void *k_pool, void *v_pool, int dtype, int M,
-                       int H, int KV, int hd, int hdv, int page_size, int norm_per_head, int rot_halves, cudaStream_t stream);
+                       int H, int KV, int hd, int hdv, int page_size, int norm_per_head, int rot_halves, int v_heads, int v_from_k,
+                       cudaStream_t stream);
+/* out = (a1 - lambda a2) / rms * gain per head, maps rows [key head][map][head of the group][dv] float32 */
+int fg_differential_combine(const float *maps, int ld, void *out, int out_dtype, int ldo, int M, int H, int KV, int dv, float lambda, float eps,
+                            float gain, cudaStream_t stream);
 /* x[m, h * DV + j] *= sigmoid(gate[m, h]) in place (gate null: none); `pad` columns behind the heads become (1, 0, 0, ...) */
 int fg_head_gate(void *x, int ldx, int dtype, const float *gate, int ldg, int M, int H, int DV, int pad, cudaStream_t stream);
 int fg_conv_state_update(const float *proj, int ld, const float *bias, int taps, float *conv_state, const int *cu_rows,
@@ -219,7 +235,7 @@ int fg_moe_combine_weighted(const float *slot_out, int ld, const int *slot_of, c
 
 /* ---- libfg_tc: bf16 contraction on tcgen05 / TMA / tensor memory
  * epi: 0 bf16 out, 1 f32 out, 2 f32 out += (residual add), 3 silu(gate) * up on interleaved rows, 4 bf16 out of max(x, 0)^2,
- * 5 gelu_tanh(gate) * up on interleaved rows */
+ * 5 gelu_tanh(gate) * up on interleaved rows, 6 max(gate, 0) * up on interleaved rows */
 int fg_gemm_tc(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int epi, int M, int N, int K,
                int force_splits, const float *ss_in, int ss_tiles, int ss_size, float ss_eps, const float *norm_w,
                void *xw_out, float *ss_out, int *ss_tiles_out /* host */, cudaStream_t stream);
@@ -254,19 +270,21 @@ int fg_attention_prefill(const void *q, int ldq, void *out, int ldo, const int *
                          const int *block_table, int table_width, const void *k_pool, const void *v_pool, int n_seq,
                          int max_new, int H, int KV, int hd, int page_size, float scale, int window, cudaStream_t stream);
 /* the three above with the first keep_first keys of a sequence visible in front of a window */
-/* the same with capped scores (softcap > 0) and a sink per query head (sinks, or null) */
+/* the same with capped scores (softcap > 0) and a sink per query head (sinks, or null); values of head size hdv (hd, or 128 beside
+   keys of 64), v_share neighbouring key heads to a value head; out_f32: float32 output instead of bfloat16 */
 int fg_attention_decode_ext(const void *q, int ldq, void *out, int ldo, const int *positions, const int *block_table,
                             int table_width, const void *k_pool, const void *v_pool, int B, int H, int KV, int hd,
                             int page_size, float scale, int window, int keep_first, int n_splits, float *part_o,
-                            float *part_ml, float softcap, const float *sinks, cudaStream_t stream);
+                            float *part_ml, float softcap, const float *sinks, int hdv, int v_share, int out_f32, cudaStream_t stream);
 int fg_attention_prefill_ext(const void *q, int ldq, void *out, int ldo, const int *cu_rows, const int *seq_start,
                              const int *block_table, int table_width, const void *k_pool, const void *v_pool, int n_seq,
                              int max_new, int H, int KV, int hd, int page_size, float scale, int window, int keep_first,
-                             float softcap, const float *sinks, cudaStream_t stream);
+                             float softcap, const float *sinks, int hdv, int v_share, int out_f32, cudaStream_t stream);
 int fg_attention_prefill_tc_ext(const void *q, int ldq, void *out, int ldo, const int *cu_rows, const int *seq_start,
                                 const int *block_table, int table_width, const void *k_pool, const void *v_pool,
                                 int n_pool_pages, int n_seq, int max_new, int H, int KV, int hd, int page_size, float scale,
-                                int window, int keep_first, float softcap, const float *sinks, cudaStream_t stream);
+                                int window, int keep_first, float softcap, const float *sinks, int hdv, int v_share, int out_f32,
+                                cudaStream_t stream);
 int fg_attention_decode_kept(const void *q, int ldq, void *out, int ldo, const int *positions, const int *block_table,
                              int table_width, const void *k_pool, const void *v_pool, int B, int H, int KV, int hd,
                              int page_size, float scale, int window, int keep_first, int n_splits, float *part_o,

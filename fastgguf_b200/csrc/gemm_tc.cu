@@ -22,7 +22,7 @@
 //               kernel (weights are never written), so weight traffic overlaps that kernel's tail.
 //   warp 1      MMA issuer (the same way): tcgen05.mma 128 x BN x 16; its commit frees the stage.
 //   warps 2-5   epilogue: tcgen05.ld of the f32 tile, then one of
-//               store bf16 | store f32 | add into f32 (residual) | silu(gate) * up -> bf16 (or gelu(gate) * up)
+//               store bf16 | store f32 | add into f32 (residual) | silu(gate) * up -> bf16 (or gelu(gate) * up, max(gate, 0) * up)
 //               (the decode kernel has eight epilogue warps, 2-9: two per lane group of tensor memory)
 //
 // The silu epilogue expects the gate and up matrices interleaved in blocks of 64 rows
@@ -48,7 +48,7 @@
 #define WAIT_SHORT_CYCLES 1000000ll
 
 enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_RELU2_BF16 = 4 /* launcher only: EPI_BF16 + act */,
-       EPI_GELU_MUL = 5 /* launcher only: EPI_SILU_MUL + act */ };
+       EPI_GELU_MUL = 5 /* launcher only: EPI_SILU_MUL + act 1 */, EPI_RELU_MUL = 6 /* launcher only: EPI_SILU_MUL + act 2 */ };
 
 __device__ int g_gemm_error = 0;      // 0, or (code << 8 | role) of the first wait that ran out
 // How long a wait may last, in SM cycles (about a second).  A variable, so that a test can make a wait run out within a
@@ -182,8 +182,10 @@ __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.w
 // silu(g) * u in f32 with the fast exponential and division (2 ulp each): the result is rounded to bfloat16
 // (8 bits of mantissa) right after, and the precise forms made the epilogue of a 64-token tile several us long
 // gelu: g * u with the tanh form of gelu instead; 0.5 (1 + tanh(y)) = sigmoid(2 y), so it is the same form on another argument
-__device__ __forceinline__ float gated_mul(float g, float u, int gelu) {
-    const float z = gelu ? g * fmaf(0.07135481627f, g * g, 1.5957691216f) : g;       // 2 sqrt(2 / pi) (g + 0.044715 g^3)
+// (act: 0 SiLU, 1 gelu, 2 max(g, 0) * u)
+__device__ __forceinline__ float gated_mul(float g, float u, int act) {
+    if (act == 2) return fmaxf(g, 0.f) * u;
+    const float z = act ? g * fmaf(0.07135481627f, g * g, 1.5957691216f) : g;       // 2 sqrt(2 / pi) (g + 0.044715 g^3)
     return __fdividef(g, 1.0f + __expf(-z)) * u;
 }
 
@@ -208,7 +210,7 @@ struct GemmArgs {
     int epi, stages;      // decode kernel: epilogue and ring depth are run-time values
     int test_skip_copy;   // tests only: the decode kernel's producer omits the activation copy of its first stage
     int splits;           // prefill kernel: > 1 = partial products of `kb_per_split` K-blocks each into out[split][M][ldc]
-    int act;              // bf16 epilogue: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward); gated epilogue: 1 = gelu, not SiLU
+    int act;              // bf16 epilogue: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward); gated epilogue: 1 = gelu, 2 = relu, not SiLU
     // prefill kernel, grouped contraction (rows in runs, each run with a weight matrix of its own out of a stack): tile t
     // is tiles[t] = {first row, end of its run, first row of the run's matrix in W, tile index along N}; null: one matrix
     const int4 *tiles;
@@ -1310,7 +1312,7 @@ static int sm_count() {
 static int prefill_splits(int M, int N, int K, int epi, int *kb_per_split) {
     static int off = -1;                           // FASTGGUF_SPLITK=0: never (the prefill kernels as they were without it)
     if (off < 0) { const char *e = getenv("FASTGGUF_SPLITK"); off = (e && e[0] == '0') ? 1 : 0; }
-    if (off || M <= 128 || epi == EPI_SILU_MUL || epi == EPI_GELU_MUL) return 0;
+    if (off || M <= 128 || epi == EPI_SILU_MUL || epi == EPI_GELU_MUL || epi == EPI_RELU_MUL) return 0;
     const int total_kb = (K + BK - 1) / BK, sms = sm_count();
     const long long tiles = (long long)((M + BM - 1) / BM) * ((N + 127) / 128);
     if (tiles * 2 > sms || total_kb < 16) return 0;
@@ -1355,9 +1357,9 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return FG_ERR_BAD_SIZE;
     // epilogue code 4: bfloat16 output of max(x, 0)^2 - the bf16 epilogue with its activation flag set
-    // epilogue code 5: the gated epilogue with the tanh form of gelu on the gate
-    const int act = (epi == EPI_RELU2_BF16 || epi == EPI_GELU_MUL) ? 1 : 0;
-    if (act) epi = epi == EPI_GELU_MUL ? EPI_SILU_MUL : EPI_BF16;
+    // epilogue codes 5, 6: the gated epilogue with the tanh form of gelu, or max(., 0), on the gate
+    const int act = epi == EPI_RELU_MUL ? 2 : (epi == EPI_RELU2_BF16 || epi == EPI_GELU_MUL) ? 1 : 0;
+    if (act) epi = epi == EPI_RELU2_BF16 ? EPI_BF16 : EPI_SILU_MUL;
     if (epi == EPI_SILU_MUL && N % 128) return FG_ERR_BAD_SIZE;
     // Up to 128 rows the weights stream through the decode kernel, in blocks of 64 tokens whose CTAs run side by side
     // and share each weight tile through L2; beyond that the prefill kernel is faster (measured: 56.6 against 45.5 k tok/s

@@ -788,7 +788,7 @@ int fg_part_run(int role, const char *kind, const char *params_json, int dtype, 
             FG_CUDA(cudaMemcpy(tok, tokens, (size_t)M * 4, cudaMemcpyHostToDevice));
             batch.tokens = tok;
             Tensor xs = upload(x, M, cols_in, FG_F32);
-            dynamic_cast<TokenInput &>(*part).forward(rt, batch, xs);
+            dynamic_cast<TokenInput &>(*part).forward(rt, batch, xs, DeferredNorm(), nullptr, nullptr);
             download(xs, out);
         } else {
             fail(FG_E_USAGE, std::string("fg_part_run cannot run a ") + role_name(role) + " alone");

@@ -51,7 +51,7 @@ PagedKVCache::~PagedKVCache() {
 }
 
 static int64_t pool_elems(const CacheGroup &g, int page_size, bool values) {
-    return (int64_t)g.n_pages * g.request.n_kv_heads * page_size * (values ? g.request.value_dim() : g.request.head_dim);
+    return (int64_t)g.n_pages * page_size * (values ? (int64_t)g.request.value_heads() * g.request.value_dim() : (int64_t)g.request.n_kv_heads * g.request.head_dim);
 }
 static int64_t pool_bytes_of(const CacheGroup &g, int page_size, int dtype, bool values) {
     return (pool_elems(g, page_size, values) * elem_size(dtype) + 255) / 256 * 256;
@@ -68,7 +68,7 @@ int64_t PagedKVCache::pool_bytes(int dtype) const {
 int64_t PagedKVCache::bytes_per_token(int dtype) const {
     int64_t b = 0;
     for (auto &g : groups)
-        b += (int64_t)g.request.n_kv_heads * (g.request.head_dim + g.request.value_dim()) * elem_size(dtype) * (int64_t)g.entries.size();
+        b += ((int64_t)g.request.n_kv_heads * g.request.head_dim + (int64_t)g.request.value_heads() * g.request.value_dim()) * elem_size(dtype) * (int64_t)g.entries.size();
     return b;
 }
 
@@ -270,6 +270,7 @@ Json PagedKVCache::info() const {
         o.set("head_dim", g.request.head_dim);
         o.set("window", g.request.window > 0 ? Json(g.request.window) : Json());
         o.set("v_head_dim", g.request.value_dim());
+        o.set("n_v_heads", g.request.value_heads());
         o.set("keep_first", g.request.window > 0 ? g.request.keep_first : 0);
         Json es = Json::array();
         for (int e : g.entries) es.push(Json(e));
@@ -336,6 +337,7 @@ std::map<int, CacheRequest> cache_requests_from_json(const Json &j) {
         c.head_dim = (int)r.get("head_dim").as_int();
         c.window = r.get("window").is_int() ? (int)r.get("window").as_int() : 0;
         c.v_head_dim = r.get("v_head_dim").is_int() ? (int)r.get("v_head_dim").as_int() : 0;
+        c.n_v_heads = r.get("n_v_heads").is_int() ? (int)r.get("n_v_heads").as_int() : 0;
         c.keep_first = r.get("keep_first").is_int() ? (int)r.get("keep_first").as_int() : 0;
         out[(int)r.get("entry").as_int()] = c;
     }

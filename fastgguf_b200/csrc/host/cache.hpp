@@ -14,7 +14,7 @@
 //     and one page table per sequence, so a full-attention group and a windowed group never share pages;
 //   * a windowed group gives pages back as soon as every position in them has left the window, except the pages
 //     of the sequence's first keep_first positions when its mixers go on reading those;
-//   * keys and values may have different head sizes (v_head_dim);
+//   * keys and values may have different head sizes (v_head_dim), and several key heads may share a value head (n_v_heads);
 //   * page 0 of every group is never handed out: padded rows of a fixed-shape step write there;
 //   * StatePool keeps [n_slots + 1, bytes] per schedule entry that asked for fixed-size state; a slot's
 //     rows are zeroed when a sequence takes the slot, and the last row is a spare for padded rows.
@@ -36,15 +36,17 @@ struct CacheRequest {
     int n_kv_heads = 0, head_dim = 0;
     int window = 0;                           // 0 keeps every position; w keeps the last w
     int v_head_dim = 0;                       // size of a value head; 0 = head_dim
+    int n_v_heads = 0;                        // value heads; 0 = n_kv_heads
     int keep_first = 0;                       // with a window: the first positions of a sequence that stay readable
+    int value_heads() const { return n_v_heads > 0 ? n_v_heads : n_kv_heads; }
     int value_dim() const { return v_head_dim > 0 ? v_head_dim : head_dim; }
     bool operator==(const CacheRequest &o) const {
-        return n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && window == o.window && value_dim() == o.value_dim() &&
+        return n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && window == o.window && value_dim() == o.value_dim() && value_heads() == o.value_heads() &&
                (window > 0 ? keep_first : 0) == (o.window > 0 ? o.keep_first : 0);
     }
     // the same storage: what a run that reads another run's cache must agree on with its owner
     bool same_storage(const CacheRequest &o) const {
-        return n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && value_dim() == o.value_dim();
+        return n_kv_heads == o.n_kv_heads && head_dim == o.head_dim && value_dim() == o.value_dim() && value_heads() == o.value_heads();
     }
     // keep whatever `o` reads as well (a reader with another window or other kept positions)
     void widen(const CacheRequest &o) {

@@ -159,11 +159,12 @@ std::unique_ptr<ModelConfig> salulorn_config_from_json(const Json &d);       // 
 std::unique_ptr<ModelConfig> pirozen_config_from_json(const Json &d);        // config_pirozen.cpp
 std::unique_ptr<ModelConfig> saluzen_config_from_json(const Json &d);        // config_saluzen.cpp
 std::unique_ptr<ModelConfig> zifelorn_config_from_json(const Json &d);       // config_zifelorn.cpp
+std::unique_ptr<ModelConfig> buguzen_config_from_json(const Json &d);        // config_buguzen.cpp
 static std::map<std::string, ConfigReader> &registry() {
     static std::map<std::string, ConfigReader> r = {{"LlamaForCausalLM", &LlamaConfig::from_json}, {"Zirivik", &zirivik_config_from_json},
                                                     {"Salulorn", &salulorn_config_from_json}, {"Pirozen", &pirozen_config_from_json},
                                                     {"Saluzen", &saluzen_config_from_json},
-                                                    {"Zifelorn", &zifelorn_config_from_json}};
+                                                    {"Zifelorn", &zifelorn_config_from_json}, {"Buguzen", &buguzen_config_from_json}};
     return r;
 }
 

@@ -62,6 +62,7 @@ ModelSpec ModelSpec::from_json(const Json &j) {
             rs.layer = (int)r.get("layer").as_int();
             if (r.get("cache_from").is_int()) rs.cache_from = (int)r.get("cache_from").as_int();
             rs.reenter = r.get("reenter").is_bool() && r.get("reenter").as_bool();
+            rs.pass = (int)param_int(r, "pass", 0, "model spec schedule");
         } else fail(FG_E_CONFIG, "model spec: a schedule entry is {\"layer\": i, \"cache_from\": j or null}");
         s.schedule.push_back(rs);
     }
@@ -135,6 +136,7 @@ DecoderModel::DecoderModel(const ModelSpec &spec_, int dtype, int device, cudaSt
     if (!spec.reentry.kind.empty()) {
         reentry_ = dynamic_cast<StreamMap *>(build(FG_ROLE_STREAM_MAP, spec.reentry));
         if (!reentry_) fail(FG_E_INTERNAL, "a part was registered under the wrong role");
+        for (auto &run : spec.schedule) if (run.reenter) reentry_->check_pass(run.pass);
     }
     final_norm_ = dynamic_cast<Norm *>(build(FG_ROLE_NORM, spec.final_norm));
     head_ = dynamic_cast<Head *>(build(FG_ROLE_HEAD, spec.head));
@@ -483,17 +485,26 @@ Tensor DecoderModel::forward(Runtime &rt, const Batch &batch) {
     Tensor x = rt.arena->matrix(batch.n_rows, spec.hidden_size, FG_F32);      // the float32 residual stream
     // an entry that the reentry map stands in front of reads a stream nobody has normalised yet
     auto reenters = [&](size_t i) { return i < n && spec.schedule[i].reenter && reentry_; };
-    Norm *first = (n && !block_at(0)->finished_norms() && !reenters(0)) ? entry_norm(block_at(0)) : nullptr;
-    DeferredNorm pending = embedding_->forward(rt, batch, x, first);
+    // a map that only adds a vector: whoever writes the stream in front of the pass adds it
+    auto row_of = [&](size_t i) -> const float * { return reenters(i) ? reentry_->added_row(spec.schedule[i].pass) : nullptr; };
+    const float *first_row = embedding_->takes_row() ? row_of(0) : nullptr;
+    bool row_added = first_row != nullptr;         // the entry that runs next has its vector already
+    Norm *first = (n && !block_at(0)->finished_norms() && (!reenters(0) || row_added)) ? entry_norm(block_at(0)) : nullptr;
+    DeferredNorm pending = embedding_->forward(rt, batch, x, first, first_row);
     Tensor x0;                                     // the embedding's output, kept for the reentry map
     bool any_reentry = false;
-    for (size_t i = 0; i < n; i++) any_reentry = any_reentry || reenters(i);
+    for (size_t i = 0; i < n; i++) any_reentry = any_reentry || (reenters(i) && !row_of(i));
     if (any_reentry && batch.n_rows > 0) {
         x0 = rt.arena->matrix(batch.n_rows, spec.hidden_size, FG_F32);
         FG_CUDA(cudaMemcpyAsync(x0.data, x.data, (size_t)batch.n_rows * spec.hidden_size * sizeof(float), cudaMemcpyDeviceToDevice, rt.stream));
     }
     for (size_t i = 0; i < n; i++) {
-        if (reenters(i) && batch.n_rows > 0) {
+        if (reenters(i) && row_of(i)) {
+            if (!row_added && batch.n_rows > 0) {
+                FG_LAUNCH("core", fg_add_row, x.ptr<float>(), row_of(i), batch.n_rows, (int)spec.hidden_size, rt.stream);
+                pending = DeferredNorm();
+            }
+        } else if (reenters(i) && batch.n_rows > 0) {
             Tensor fresh = rt.arena->matrix(batch.n_rows, spec.hidden_size, FG_F32);     // in the step's own lane: it outlives layers
             reentry_->forward(rt, x, x0, fresh);
             x = fresh;
@@ -505,12 +516,19 @@ Tensor DecoderModel::forward(Runtime &rt, const Batch &batch) {
         if (block_at(i)->finished_norms()) next = i + 1 == n ? head_norm : block_at(i + 1)->finished_norms() ? block_at(i + 1)->mixer_norm : nullptr;
         else if (i + 1 < n && block_at(i + 1)->finished_norms()) next = nullptr;
         // a layer that adds a token input behind its sublayers changes the stream after its last projection
-        if (reenters(i + 1) || block_at(i)->token_input) next = nullptr;
+        TokenInput *side = block_at(i)->token_input;
+        if (reenters(i + 1)) next = nullptr;
+        // (what its contraction wants is the rounded stream, which the block's last projection can write: a started norm of unit weight)
+        if (side) next = bf16 && !block_at(i)->finished_norms() ? side->stream_norm() : nullptr;
         rt.arena->begin_layer((int)i);                 // this entry's temporaries reuse the memory of entry i - 2
         pending = block_at(i)->forward(rt, x, batch, io[i], pending, next);
-        if (block_at(i)->token_input) {
-            block_at(i)->token_input->forward(rt, batch, x);
-            pending = DeferredNorm();
+        row_added = false;
+        if (side) {
+            // its last kernel may add the vector of the next pass, and finish the norm that reads the stream next
+            const float *row = row_of(i + 1);
+            Norm *reader = i + 1 == n ? head_norm : block_at(i + 1)->takes_finished_norm() && (row || !reenters(i + 1)) ? block_at(i + 1)->mixer_norm : nullptr;
+            pending = side->forward(rt, batch, x, pending, row, reader);
+            row_added = row != nullptr;
         }
         // the rounded stream itself is for a block that reads it so
         if (pending.defined() && !pending.weight && !(i + 1 < n && block_at(i + 1)->reads_stream())) pending = DeferredNorm();
@@ -550,7 +568,7 @@ void DecoderModel::block_forward(int entry, const std::vector<std::pair<int, int
     FG_CUDA(cudaMemcpyAsync(x.data, x_host, bytes, cudaMemcpyHostToDevice, runtime.stream));
     Block *blk = blocks_[(size_t)spec.schedule[(size_t)entry].layer].get();
     blk->forward(runtime, x, batch, io[(size_t)entry], DeferredNorm(), nullptr);
-    if (blk->token_input) blk->token_input->forward(runtime, batch, x);
+    if (blk->token_input) blk->token_input->forward(runtime, batch, x, DeferredNorm(), nullptr, nullptr);
     FG_CUDA(cudaMemcpyAsync(x_host, x.data, bytes, cudaMemcpyDeviceToHost, runtime.stream));
     FG_CUDA(cudaStreamSynchronize(runtime.stream));
     cache->commit(steps);

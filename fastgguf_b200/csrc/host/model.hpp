@@ -38,6 +38,7 @@ struct RunSpec {
     int layer = 0;
     int cache_from = -1;                             // an EARLIER schedule entry whose cache this run reads
     bool reenter = false;                            // the model's `reentry` map runs on the stream in front of this entry
+    int pass = 0;                                    // with reenter: the number of the pass that begins here
 };
 struct ModelSpec {
     int64_t hidden_size = 0, vocab_size = 0, max_positions = 0;

@@ -9,7 +9,7 @@
 
 namespace fg {
 
-static const int EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_GELU_MUL = 5;
+static const int EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_GELU_MUL = 5, EPI_RELU_MUL = 6;
 static const int KERNEL_BAD_SIZE = 10002;
 
 const char *role_name(int role) {
@@ -206,7 +206,9 @@ Tensor Linear::forward_relu2(Runtime &rt, const Tensor &a) const {
     return t;
 }
 
-bool Linear::forward_gated(Runtime &rt, const Tensor &a_in, const DeferredNorm *deferred, bool gelu, Tensor *out) const {
+bool Linear::forward_gated(Runtime &rt, const Tensor &a_in, const DeferredNorm *deferred, int act, Tensor *out) const {
+    static const int epi_of[3] = {EPI_SILU_MUL, EPI_GELU_MUL, EPI_RELU_MUL};
+    static const char *name_of[3] = {"silu", "gelu", "relu"};
     const Tensor &W = w_.t;
     Tensor a = deferred ? deferred->xw : a_in;
     if (!fast_ || rt.plain_kernels || a.dtype != FG_BF16 || W.rows % 128) return false;
@@ -218,8 +220,8 @@ bool Linear::forward_gated(Runtime &rt, const Tensor &a_in, const DeferredNorm *
     float ss_eps = 0.f;
     if (deferred) { ss_in = deferred->ss; ss_tiles = deferred->tiles; ss_size = deferred->size; ss_eps = deferred->eps; }
     count_launch();
-    ProfileScope scope("fg_gemm_tc", profile_on() ? format("%lld x %lld, %lld rows, %s", (long long)W.rows, (long long)a.cols, (long long)M, gelu ? "gelu" : "silu").c_str() : nullptr);
-    int code = FG_KERNEL("tc", fg_gemm_tc)(a.data, (int)a.ld, W.data, (int)W.ld, t.data, (int)t.ld, gelu ? EPI_GELU_MUL : EPI_SILU_MUL, (int)M,
+    ProfileScope scope("fg_gemm_tc", profile_on() ? format("%lld x %lld, %lld rows, %s", (long long)W.rows, (long long)a.cols, (long long)M, name_of[act]).c_str() : nullptr);
+    int code = FG_KERNEL("tc", fg_gemm_tc)(a.data, (int)a.ld, W.data, (int)W.ld, t.data, (int)t.ld, epi_of[act], (int)M,
                                            (int)W.rows, (int)a.cols, 0, ss_in, ss_tiles, ss_size, ss_eps, nullptr, nullptr,
                                            nullptr, &tiles_out, rt.stream);
     if (code == KERNEL_BAD_SIZE) return false;
@@ -386,6 +388,13 @@ std::vector<double> rotary_divisors(int rotary_dim, double theta, const Json &sc
     if (!scaling.is_object()) return div;
     const Json &kind = scaling.get("rope_type");
     if (kind.is_null() || (kind.is_string() && kind.as_string() == "default")) return div;
+    if (kind.is_string() && kind.as_string() == "linear") {
+        // every frequency divided by one factor
+        double factor = param_float(scaling, "factor", "rope scaling");
+        if (!(factor > 0)) fail(FG_E_CONFIG, "rope scaling linear: factor must be positive");
+        div.assign((size_t)half, factor);
+        return div;
+    }
     if (kind.is_string() && kind.as_string() == "yarn") {
         // Frequencies between two wavelengths are blended from "as trained" to "slowed by factor".  With
         // dim(t) = n_rot ln(orig / (2 pi t)) / (2 ln theta) - the (fractional) rotary dimension whose wave turns t times over
@@ -404,7 +413,7 @@ std::vector<double> rotary_divisors(int rotary_dim, double theta, const Json &sc
         return div;
     }
     if (!kind.is_string() || kind.as_string() != "llama3")
-        fail(FG_E_CONFIG, "rotary scaling " + kind.dump() + " is not known (known: default, llama3, yarn)");
+        fail(FG_E_CONFIG, "rotary scaling " + kind.dump() + " is not known (known: default, linear, llama3, yarn)");
     double factor = param_float(scaling, "factor", "rope scaling"), low = param_float(scaling, "low_freq_factor", "rope scaling");
     double high = param_float(scaling, "high_freq_factor", "rope scaling");
     double orig = param_float(scaling, "original_max_position_embeddings", "rope scaling");
@@ -638,15 +647,15 @@ private:
 // ------------------------------------------------------------------------------------ SwiGLU
 // down( silu(gate x) * (up x) ): gate and up in one fused pass (fastgguf.c:4870-4872), silu(z) = z / (1 + exp(-z))
 // (:3118) times up (:4876), down projection added onto the layer's input (:4877-4880).
-// activation "gelu_tanh": down(gelu_tanh(gate x) * (up x)) instead.
+// activation "gelu_tanh": down(gelu_tanh(gate x) * (up x)) instead; "relu": down(max(gate x, 0) * (up x)).
 class SwiGLU : public FeedForward {
 public:
     SwiGLU(const Json &p) : E_((int)param_int(p, "hidden_size", "swiglu")), F_((int)param_int(p, "d_ff", "swiglu")) {
         if (E_ <= 0 || F_ <= 0) fail(FG_E_CONFIG, "swiglu: sizes must be positive");
         const Json &a = p.get("activation");
         const std::string act = a.is_string() ? a.as_string() : "silu";
-        if (act != "silu" && act != "gelu_tanh") fail(FG_E_CONFIG, "swiglu: activation '" + act + "' is not known (known: silu, gelu_tanh)");
-        gelu_ = act == "gelu_tanh";
+        if (act != "silu" && act != "gelu_tanh" && act != "relu") fail(FG_E_CONFIG, "swiglu: activation '" + act + "' is not known (known: silu, gelu_tanh, relu)");
+        act_ = act == "gelu_tanh" ? GATED_GELU : act == "relu" ? GATED_RELU : GATED_SILU;
     }
     std::vector<TensorDecl> tensor_decls() const override {
         return {{"gate_proj.weight", {F_, E_}}, {"up_proj.weight", {F_, E_}}, {"down_proj.weight", {E_, F_}}};
@@ -673,12 +682,13 @@ public:
     DeferredNorm forward(Runtime &rt, const Tensor &xn, const DeferredNorm *deferred, const Batch &, Tensor &residual,
                          Norm *emit_norm) override {
         Tensor t;
-        bool done = fused_.defined() && fused_.forward_gated(rt, xn, deferred, gelu_, &t);
+        bool done = fused_.defined() && fused_.forward_gated(rt, xn, deferred, act_, &t);
         if (!done) {
             if (fused_.defined()) fail(FG_E_KERNEL, "the fused gate/up kernel refused a shape it was planned for");
             Tensor gu = gate_up_.forward(rt, xn, deferred, Tensor(), rt.dtype, false, nullptr, nullptr);
             t = rt.arena->matrix(gu.rows, F_, gu.dtype);
-            if (gu.rows > 0 && gelu_) FG_LAUNCH("core", fg_gelu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
+            if (gu.rows > 0 && act_ == GATED_RELU) FG_LAUNCH("core", fg_relu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
+            else if (gu.rows > 0 && act_ == GATED_GELU) FG_LAUNCH("core", fg_gelu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
             else if (gu.rows > 0) FG_LAUNCH("core", fg_silu_mul, gu.data, t.data, gu.dtype, (int)gu.rows, F_, rt.stream);
         }
         DeferredNorm started;
@@ -688,7 +698,7 @@ public:
 
 private:
     int E_, F_;
-    bool gelu_ = false;
+    int act_ = GATED_SILU;
     Linear fused_, gate_up_, down_;
 };
 
@@ -702,6 +712,7 @@ std::unique_ptr<FeedForward> make_swiglu(const Json &params) { return std::make_
 // that reads the normalised rows; parts that do not take part get plain normalised tensors.
 class PreNormBlock : public Block {
 public:
+    bool takes_finished_norm() const override { return true; }
     void check_layer() const override {
         Block::check_layer();
         if (mixer_post_norm || feed_forward_post_norm) fail(FG_E_CONFIG, "block 'prenorm' has no norms behind its sublayers (see 'sandwich')");
@@ -712,19 +723,21 @@ public:
         bool mixer_defers = bf16 && mixer->supports_deferred_norm();
         bool ffn_defers = bf16 && feed_forward && feed_forward->supports_deferred_norm();
         DeferredNorm started;
+        const bool finished = pending.defined() && pending.tiles == 0;          // (the norm itself, in the activation dtype)
+        auto mixer_in = [&]() -> Tensor { return finished ? pending.xw : mixer_norm->forward(rt, x, nullptr, 0); };
         if (!feed_forward) {
             // a layer of a mixer alone: its output projection may start the next layer's norm
-            if (mixer_defers && pending.defined()) return mixer->forward(rt, Tensor(), &pending, batch, io, x, next_norm);
-            if (mixer_defers) return mixer->forward(rt, mixer_norm->forward(rt, x, nullptr, 0), nullptr, batch, io, x, next_norm);
-            mixer->forward(rt, mixer_norm->forward(rt, x, nullptr, 0), nullptr, batch, io, x, nullptr);
+            if (mixer_defers && pending.defined() && !finished) return mixer->forward(rt, Tensor(), &pending, batch, io, x, next_norm);
+            if (mixer_defers) return mixer->forward(rt, mixer_in(), nullptr, batch, io, x, next_norm);
+            mixer->forward(rt, mixer_in(), nullptr, batch, io, x, nullptr);
             return DeferredNorm();
         }
         if (mixer_defers) {
             Norm *emit = (ffn_defers && feed_forward_norm->deferrable()) ? feed_forward_norm : nullptr;
-            if (pending.defined()) started = mixer->forward(rt, Tensor(), &pending, batch, io, x, emit);
-            else started = mixer->forward(rt, mixer_norm->forward(rt, x, nullptr, 0), nullptr, batch, io, x, emit);
+            if (pending.defined() && !finished) started = mixer->forward(rt, Tensor(), &pending, batch, io, x, emit);
+            else started = mixer->forward(rt, mixer_in(), nullptr, batch, io, x, emit);
         } else {
-            mixer->forward(rt, mixer_norm->forward(rt, x, nullptr, 0), nullptr, batch, io, x, nullptr);
+            mixer->forward(rt, mixer_in(), nullptr, batch, io, x, nullptr);
         }
         if (ffn_defers) {
             if (started.defined()) return feed_forward->forward(rt, Tensor(), &started, batch, x, next_norm);
@@ -757,6 +770,7 @@ public:
             if (n && !n->deferrable()) fail(FG_E_CONFIG, "block 'sandwich' takes norms of the form x / rms(x) * w");
     }
     bool finished_norms() const override { return true; }
+    bool takes_finished_norm() const override { return true; }
     // pending.xw (when defined, with tiles == 0) holds the FINISHED norm of x for this block's mixer, made by the block before
     DeferredNorm forward(Runtime &rt, Tensor &x, const Batch &batch, const LayerIO &io, const DeferredNorm &pending,
                          Norm *next_norm) override {
@@ -862,6 +876,7 @@ public:
 // are formed (one kernel, one statistic a row) before either sublayer adds to the stream.
 class ParallelBlock : public Block {
 public:
+    bool takes_finished_norm() const override { return !feed_forward_norm; }
     void check_layer() const override {
         if (!mixer || !mixer_norm) fail(FG_E_CONFIG, "a layer needs a mixer and its norm");
         if (mixer_post_norm || feed_forward_post_norm) fail(FG_E_CONFIG, "block 'parallel' has its norms in front of the sublayers");
@@ -946,12 +961,17 @@ public:
         proj_ = Linear(tensor_of(tensors, "proj"));
         const Weight &w = tensor_of(tensors, "norm");
         norm_w_ = w.t.dtype == FG_F32 ? w : concat_rows({w}, FG_F32, rt.stream);
+        stream_.load(E_, rt);
     }
-    void forward(Runtime &rt, const Batch &b, Tensor &x) override {
+    Norm *stream_norm() override { return &stream_; }
+    DeferredNorm forward(Runtime &rt, const Batch &b, Tensor &x, const DeferredNorm &stream, const float *add_row, Norm *reader) override {
         const int M = (int)x.rows;
-        if (M == 0) return;
+        DeferredNorm next;
+        if (M == 0) return next;
         Tensor xin = x;
-        if (rt.dtype != FG_F32) {
+        if (rt.dtype == FG_BF16 && stream.defined() && stream.weight == stream_.weight()) {
+            xin = stream.xw;                     // the contraction that wrote the stream rounded it as well
+        } else if (rt.dtype != FG_F32) {
             xin = rt.arena->matrix(M, E_, rt.dtype);
             FG_LAUNCH("core", fg_cast_rows, x.ptr<float>(), (int)x.ld, xin.data, xin.dtype, (int)xin.ld, M, (int)E_, rt.stream);
         }
@@ -960,11 +980,35 @@ public:
         FG_LAUNCH("core", fg_gelu_mul_gather, z.ptr<float>(), (int)z.ld, table_.t.data, table_.t.dtype, (int)table_.t.ld, (int)col_, b.tokens, g.data,
                   g.dtype, (int)g.ld, M, (int)D_, rt.stream);
         Tensor y = proj_.forward(rt, g, nullptr, Tensor(), FG_F32, false, nullptr, nullptr);
-        FG_LAUNCH("core", fg_norm_add_norm, y.ptr<float>(), norm_w_.t.ptr<float>(), x.ptr<float>(), nullptr, nullptr, rt.dtype, M, (int)E_, eps_, 0.f,
-                  rt.stream);
+        if (reader && !(reader->deferrable() && reader->weight() && reader->size() == E_ && E_ * (int64_t)sizeof(float) <= 48 * 1024)) reader = nullptr;
+        if (reader) {
+            next.xw = rt.arena->matrix(M, E_, rt.dtype);
+            next.tiles = 0; next.size = (int)E_; next.eps = reader->eps(); next.x = x; next.weight = reader->weight();
+        }
+        FG_LAUNCH("core", fg_norm_add_norm_row, y.ptr<float>(), norm_w_.t.ptr<float>(), add_row, x.ptr<float>(), next.weight, next.xw.data, rt.dtype, M, (int)E_,
+                  eps_, next.eps, rt.stream);
+        return next;
     }
 
 private:
+    // x * 1: what a contraction writes as this norm's started form is the stream rounded to bfloat16
+    class UnitNorm : public Norm {
+    public:
+        void load(int64_t E, Runtime &rt) {
+            ones_ = make_weight(1, E, FG_F32, "a unit norm weight");
+            FG_CUDA(cudaMemsetAsync(ones_.t.data, 0, (size_t)E * sizeof(float), rt.stream));
+            dev_shift_f32(ones_.t.ptr<float>(), E, 1.0f, rt.stream);
+        }
+        Tensor forward(Runtime &, const Tensor &, const int *, int) override { fail(FG_E_INTERNAL, "the stream's rounding is not a norm of its own"); }
+        bool deferrable() const override { return true; }
+        const float *weight() const override { return ones_.t.ptr<float>(); }
+        float eps() const override { return 0.f; }
+        int size() const override { return (int)ones_.t.cols; }
+
+    private:
+        Weight ones_;
+    };
+    UnitNorm stream_;
     int64_t E_ = 0, V_ = 0, D_ = 0, col_ = 0, TD_ = 0;
     float eps_ = 0.f;
     Weight table_, norm_w_;
@@ -993,6 +1037,29 @@ private:
     Linear w_;
 };
 
+// x <- x + step[t] in front of pass t of a looped span: one vector a pass, from a table [rows, E].  Nothing runs by itself: the
+// kernel that writes the stream in front of the pass adds the vector, or a kernel of the model's step does.
+class AddRow : public StreamMap {
+public:
+    AddRow(const Json &p) : E_(param_int(p, "hidden_size", "add_row")), rows_(param_int(p, "rows", "add_row")) {
+        if (E_ <= 0 || rows_ <= 0) fail(FG_E_CONFIG, "add_row: hidden_size and rows must be positive");
+    }
+    std::vector<TensorDecl> tensor_decls() const override { return {{"table", {rows_, E_}}}; }
+    void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
+        const Weight &w = tensor_of(tensors, "table");
+        table_ = w.t.dtype == FG_F32 ? w : concat_rows({w}, FG_F32, rt.stream);
+    }
+    void check_pass(int pass) const override {
+        if (pass < 0 || pass >= rows_) fail(FG_E_CONFIG, format("add_row: there is no vector for pass %d of %lld", pass, (long long)rows_));
+    }
+    const float *added_row(int pass) const override { return table_.t.ptr<float>() + (int64_t)pass * E_; }
+    void forward(Runtime &, const Tensor &, const Tensor &, Tensor &) override { fail(FG_E_INTERNAL, "add_row is added where the stream is written"); }
+
+private:
+    int64_t E_, rows_;
+    Weight table_;
+};
+
 // ------------------------------------------------------------------------------------ embedding and head
 // read_embedding copies row `token` of token_embd into the residual stream, times embd_scale, which is 1 for
 // Llama (fastgguf.c:4576-4581, :4652, :4219); the head is output.weight or, when that tensor is absent, the
@@ -1007,20 +1074,21 @@ public:
     }
     std::vector<TensorDecl> tensor_decls() const override { return {{"weight", {V_, E_}}}; }
     void load(const std::map<std::string, Weight> &tensors, Runtime &) override { w_ = tensor_of(tensors, "weight"); }
-    DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *emit_norm) override {
+    bool takes_row() const override { return true; }
+    DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *emit_norm, const float *add_row) override {
         DeferredNorm started;
         int M = batch.n_rows;
         if (M == 0) return started;
         if (emit_norm && emit_norm->deferrable() && emit_norm->size() == E_ && rt.dtype == FG_BF16 && scale_ == 1.0f) {
             Tensor xw = rt.arena->matrix(M, E_, FG_BF16);
             float *ss = (float *)rt.arena->alloc((size_t)M * sizeof(float));
-            FG_LAUNCH("core", fg_embed_gather_norm, w_.t.data, w_.t.dtype, batch.tokens, x.ptr<float>(), emit_norm->weight(), xw.data,
+            FG_LAUNCH("core", fg_embed_gather_norm_row, w_.t.data, w_.t.dtype, batch.tokens, add_row, x.ptr<float>(), emit_norm->weight(), xw.data,
                       ss, M, (int)E_, rt.stream);
             started.xw = xw; started.ss = ss; started.tiles = 1; started.size = (int)E_; started.eps = emit_norm->eps();
             started.x = x; started.weight = emit_norm->weight();
             return started;
         }
-        FG_LAUNCH("core", fg_embed_gather_scaled, w_.t.data, w_.t.dtype, batch.tokens, x.ptr<float>(), M, (int)E_, scale_, rt.stream);
+        FG_LAUNCH("core", fg_embed_gather_row, w_.t.data, w_.t.dtype, batch.tokens, add_row, x.ptr<float>(), M, (int)E_, scale_, rt.stream);
         return started;
     }
 
@@ -1230,7 +1298,7 @@ public:
     ExternalEmbedding(const fg_part_vtable &v, const std::string &k, const Json &p, int dtype) : core(v, k, FG_ROLE_EMBEDDING, p, dtype) {}
     std::vector<TensorDecl> tensor_decls() const override { return core.decls(); }
     void load(const std::map<std::string, Weight> &t, Runtime &) override { core.load(t); }
-    DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *) override {
+    DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *, const float *) override {
         fg_batch_view bv = batch.view(rt.stream);
         fg_part_call c = {};
         c.batch = &bv; c.x = x.view();
@@ -1342,6 +1410,7 @@ static std::map<std::string, PartFactory> &factories(int role) {
         r[FG_ROLE_HEAD]["lm_head"] = [](Runtime &, const Json &p, BuildContext &) { return std::make_unique<LMHead>(p); };
         r[FG_ROLE_TOKEN_INPUT]["gated_token_embedding"] = [](Runtime &, const Json &p, BuildContext &) { return std::make_unique<GatedTokenEmbedding>(p); };
         r[FG_ROLE_STREAM_MAP]["concat_linear"] = [](Runtime &, const Json &p, BuildContext &) { return std::make_unique<ConcatLinear>(p); };
+        r[FG_ROLE_STREAM_MAP]["add_row"] = [](Runtime &, const Json &p, BuildContext &) { return std::make_unique<AddRow>(p); };
         add_recurrent_kinds(r[FG_ROLE_MIXER]);
         add_attention_kinds(r[FG_ROLE_MIXER]);
         add_expert_kinds(r[FG_ROLE_FEED_FORWARD]);

@@ -152,8 +152,12 @@ public:
 // What a layer adds to the stream from the tokens themselves, behind its sublayers (a second embedding table read per layer).
 class TokenInput : public Part {
 public:
-    // x [M, E] float32 is updated in place; batch.tokens names the rows' tokens
-    virtual void forward(Runtime &rt, const Batch &batch, Tensor &x) = 0;
+    // x [M, E] float32 is updated in place; batch.tokens names the rows' tokens.  stream: x rounded to the activation dtype, if
+    // whoever wrote x made it (a started norm of stream_norm()); add_row ([E] or null): added to every row of the updated x as well;
+    // reader (or null): the norm that reads x next, which may be returned finished (xw, tiles == 0)
+    virtual DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, const DeferredNorm &stream, const float *add_row, Norm *reader) = 0;
+    // a norm of unit weight: STARTED (never finished) by the contraction that writes x it is x rounded to bfloat16; null: not wanted
+    virtual Norm *stream_norm() { return nullptr; }
 };
 
 // An arrangement of a mixer, a feed-forward and their norms around the residual stream.  A layer may have no
@@ -166,6 +170,8 @@ public:
     Norm *mixer_norm = nullptr, *feed_forward_norm = nullptr;
     Norm *mixer_post_norm = nullptr, *feed_forward_post_norm = nullptr;   // on a sublayer's output, before the residual add
     TokenInput *token_input = nullptr;       // optional; the model runs it on the stream right behind the block
+    // true: `pending` may be a FINISHED norm of the stream for this block's mixer
+    virtual bool takes_finished_norm() const { return false; }
     // refuses a layer this arrangement cannot run (called once, when the model is built)
     virtual void check_layer() const;
     // true: the block hands the NEXT block's first norm over finished (xw = the normalised rows, tiles == 0) instead of
@@ -183,8 +189,10 @@ public:
 
 class Embedding : public Part {
 public:
-    // fills x [M, E] f32; with emit_norm (deferrable) may also start that norm
-    virtual DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *emit_norm) = 0;
+    // fills x [M, E] f32; with emit_norm (deferrable) may also start that norm; add_row ([E] or null; only where takes_row()) is
+    // added to every row
+    virtual DeferredNorm forward(Runtime &rt, const Batch &batch, Tensor &x, Norm *emit_norm, const float *add_row = nullptr) = 0;
+    virtual bool takes_row() const { return false; }
 };
 
 class Head : public Part {
@@ -198,6 +206,10 @@ public:
 // run a span of layers several times feed the embedding's output back in at the start of every pass.
 class StreamMap : public Part {
 public:
+    // a map that only adds one vector [E] to every row, another one in every pass: that vector (whoever writes the stream in front
+    // of the pass may add it, and forward is not called); null: any other map
+    virtual const float *added_row(int pass) const { (void)pass; return nullptr; }
+    virtual void check_pass(int pass) const { (void)pass; }        // refuses a pass the map has nothing for
     // out [M, E] float32 (fresh memory) = f(x, x0); x: the stream, x0: the embedding's output, both [M, E] float32
     virtual void forward(Runtime &rt, const Tensor &x, const Tensor &x0, Tensor &out) = 0;
 };
@@ -242,6 +254,7 @@ double param_float(const Json &params, const char *key, double dflt, const char 
 // matvec / matmul (:2575-2622, :3004-3093); here the choice is by dtype, row count and alignment:
 // float32 operands, or sizes the fast kernels refuse -> the plain FMA kernel; bfloat16 with few rows
 // (decode) -> the weight-streaming tensor-core kernel; bfloat16 with many rows -> the tiled tcgen05 kernel.
+enum GatedAct { GATED_SILU = 0, GATED_GELU = 1, GATED_RELU = 2 };      // gelu: its tanh form
 class Linear {
 public:
     Linear() = default;
@@ -259,9 +272,8 @@ public:
     // max(a W^T, 0)^2 in the activation dtype: in the tensor-core kernel's epilogue where that kernel runs, else the
     // contraction and an elementwise pass
     Tensor forward_relu2(Runtime &rt, const Tensor &a) const;
-    // act(a gate^T) * (a up^T) as bf16 [M, F] from rows interleaved in blocks of 64, act SiLU or the tanh form of gelu; false if
-    // refused
-    bool forward_gated(Runtime &rt, const Tensor &a, const DeferredNorm *deferred, bool gelu, Tensor *out) const;
+    // act(a gate^T) * (a up^T) as bf16 [M, F] from rows interleaved in blocks of 64, act by its number in GatedAct; false if refused
+    bool forward_gated(Runtime &rt, const Tensor &a, const DeferredNorm *deferred, int act, Tensor *out) const;
 
 private:
     Weight w_;

@@ -20,6 +20,14 @@
 //   o <- o * sigmoid(W_g h) with W_g [heads * v_head_dim, hidden] ("gate": "full"); a bias on the output
 //   projection ("o_bias": true), stored as one more column of the output matrix that meets a column of ones, so the
 //   projection's own pass adds it.
+//   "values": "keys": there is no W_v, the values are the keys as projected (bias included), before norm and rotation.
+//   "differential": d: every query head and every key head is two maps [map 1 | map 2] of head_dim numbers (q has n_heads * 2 *
+//   head_dim rows, k n_kv_heads * 2 * head_dim), each an attention of its own over the SAME values; with their outputs a1, a2 and
+//       lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + d    (one number, from four vectors [head_dim])
+//       o = a1 - lambda a2,  o <- o / sqrt(mean(o^2) + eps) * (1 - d) over a head's values (no weight).
+//   The kernels see 2 n_heads query heads and 2 n_kv_heads key heads, two neighbouring key heads to a value head: the rows of q are
+//   reordered once at load from [head][map] to [key head][map][head of the group].  The maps' outputs stay float32 until the
+//   difference is normalised.
 //
 // "latent_attention": keys and values are linear maps of ONE small latent per token, c = norm(W_dkv h)[0:kv_rank], plus a
 // rotated key part of rot_dim numbers that all heads share; queries pass through a latent of their own,
@@ -56,6 +64,12 @@ public:
         scale_ = (float)param_float(p, "scale", 1.0 / std::sqrt((double)hd_), me);
         window_ = (int)param_int(p, "window", 0, me);
         chunk_ = (int)param_int(p, "chunk", 0, me);
+        const Json &vals = p.get("values");
+        if (!vals.is_null() && !(vals.is_string() && vals.as_string() == "keys")) fail(FG_E_CONFIG, "sink_attention: values " + vals.dump() + " is not known (known: keys)");
+        v_from_k_ = !vals.is_null();
+        differential_ = !p.get("differential").is_null();
+        diff_ = (float)param_float(p, "differential", 0.0, me);
+        maps_ = differential_ ? 2 : 1;
         softcap_ = (float)param_float(p, "softcap", 0.0, me);
         taps_ = (int)param_int(p, "conv_taps", 0, me);
         eps_ = (float)param_float(p, "eps", 1e-6, me);
@@ -79,7 +93,10 @@ public:
         pad_ = o_bias_ ? 8 - (int)(((int64_t)H_ * hdv_) % 8) : 0;
         if (window_ < 0 || softcap_ < 0.f || taps_ < 0) fail(FG_E_CONFIG, "sink_attention: window, softcap and conv_taps cannot be negative");
         if (hdv_ > 512) fail(FG_E_CONFIG, format("sink_attention: v_head_dim %d exceeds 512, the largest the kernel takes", hdv_));
-        if (((size_t)H_ * hd_ + (size_t)KV_ * (hd_ + hdv_)) * 4 > 200 * 1024) fail(FG_E_CONFIG, "sink_attention: a token's q, k and v exceed what the kernel holds in shared memory");
+        if (v_from_k_ && hdv_ != hd_) fail(FG_E_CONFIG, format("sink_attention: values that are the keys have their size (%d), not %d", hd_, hdv_));
+        if (v_from_k_ && (differential_ || taps_ > 0)) fail(FG_E_CONFIG, "sink_attention: values that are the keys stand beside neither a convolution nor two maps");
+        if (differential_ && (sink_ || unit_sink_ || taps_ > 0 || gate_)) fail(FG_E_CONFIG, "sink_attention: two maps stand beside neither sinks, a convolution nor a gate");
+        if ((size_t)channels() * 4 > 200 * 1024) fail(FG_E_CONFIG, "sink_attention: a token's q, k and v exceed what the kernel holds in shared memory");
         const Json &pos = p.get("position");
         if (!pos.is_null()) {
             position_ = dynamic_cast<PositionEncoding *>(ctx.nested(FG_ROLE_POSITION, pos));
@@ -92,10 +109,11 @@ public:
         }
     }
     std::vector<TensorDecl> tensor_decls() const override {
-        const int64_t Q = (int64_t)H_ * hd_, K = (int64_t)KV_ * hd_, V = (int64_t)KV_ * hdv_;
-        std::vector<TensorDecl> d = {{"q_proj.weight", {Q, E_}}, {"k_proj.weight", {K, E_}}, {"v_proj.weight", {V, E_}},
-                                     {"o_proj.weight", {E_, (int64_t)H_ * hdv_}}};
-        if (bias_) for (auto &n : std::vector<std::pair<const char *, int64_t>>{{"q_proj.bias", Q}, {"k_proj.bias", K}, {"v_proj.bias", V}}) d.push_back({n.first, {n.second}});
+        const int64_t Q = (int64_t)maps_ * H_ * hd_, K = (int64_t)maps_ * KV_ * hd_, V = v_from_k_ ? 0 : (int64_t)KV_ * hdv_;
+        std::vector<TensorDecl> d = {{"q_proj.weight", {Q, E_}}, {"k_proj.weight", {K, E_}}, {"o_proj.weight", {E_, (int64_t)H_ * hdv_}}};
+        if (V > 0) d.push_back({"v_proj.weight", {V, E_}});
+        if (bias_) for (auto &n : std::vector<std::pair<const char *, int64_t>>{{"q_proj.bias", Q}, {"k_proj.bias", K}, {"v_proj.bias", V}}) if (n.second > 0) d.push_back({n.first, {n.second}});
+        if (differential_) for (const char *n : {"lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2"}) d.push_back({n, {(int64_t)hd_}, false, 0, 0.1f});
         if (taps_ > 0)
             for (auto &n : std::vector<std::pair<const char *, int64_t>>{{"q_conv.weight", Q}, {"k_conv.weight", K}, {"v_conv.weight", V}})
                 d.push_back({n.first, {n.second, (int64_t)taps_}, false, 0, 0.5f});
@@ -110,21 +128,21 @@ public:
     }
     bool cache_request(CacheRequest *out) const override {
         // (a chunked mask keeps every page: a sequence's pages are given back when it ends)
-        out->n_kv_heads = KV_; out->head_dim = hd_; out->window = window_; out->v_head_dim = hdv_; out->keep_first = 0;
+        out->n_kv_heads = maps_ * KV_; out->head_dim = hd_; out->window = window_; out->v_head_dim = hdv_; out->n_v_heads = KV_; out->keep_first = 0;
         return true;
     }
-    int64_t channels() const { return (int64_t)H_ * hd_ + (int64_t)KV_ * (hd_ + hdv_); }
+    int64_t channels() const { return (int64_t)maps_ * (H_ + KV_) * hd_ + (v_from_k_ ? 0 : (int64_t)KV_ * hdv_); }
     int64_t state_bytes() const override { return taps_ > 1 ? (int64_t)(taps_ - 1) * channels() * (int64_t)sizeof(float) : 0; }
     bool supports_deferred_norm() const override { return true; }
     bool can_overwrite() const override { return true; }
     void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
-        const Weight &q = tensor_of(tensors, "q_proj.weight"), &k = tensor_of(tensors, "k_proj.weight"), &v = tensor_of(tensors, "v_proj.weight");
-        int dt = (q.t.dtype == k.t.dtype && k.t.dtype == v.t.dtype) ? q.t.dtype : FG_F32;
-        std::vector<Weight> rows = {q, k, v};
-        if (gate_) {
-            rows.push_back(tensor_of(tensors, "g_proj.weight"));        // the gate's rows ride in the same contraction
-            if (rows.back().t.dtype != dt) dt = FG_F32;
-        }
+        Weight q = tensor_of(tensors, "q_proj.weight");
+        if (differential_) q = gather_rows(q, map_order(), rt.stream);
+        std::vector<Weight> rows = {q, tensor_of(tensors, "k_proj.weight")};
+        if (!v_from_k_) rows.push_back(tensor_of(tensors, "v_proj.weight"));
+        if (gate_) rows.push_back(tensor_of(tensors, "g_proj.weight"));        // the gate's rows ride in the same contraction
+        int dt = q.t.dtype;
+        for (auto &w : rows) if (w.t.dtype != dt) dt = FG_F32;
         qkv_ = Linear(concat_rows(rows, dt, rt.stream));
         if (o_bias_) {
             // [W_o | b | 0 ...]: the bias as a column that meets the ones fg_head_gate writes behind the heads' outputs
@@ -143,19 +161,30 @@ public:
             o_ = Linear(tensor_of(tensors, "o_proj.weight"));
         }
         auto three = [&](const char *a, const char *b, const char *c, int64_t cols) {
-            Weight x = tensor_of(tensors, a), y = tensor_of(tensors, b), z = tensor_of(tensors, c);
-            // row-major [channels, cols]: the three lie one after another
-            Weight out = make_weight(x.t.numel() / cols + y.t.numel() / cols + z.t.numel() / cols, cols, FG_F32, "per-channel parameters of attention");
-            size_t at = 0;
-            for (const Weight *w : {&x, &y, &z}) {
-                dev_convert(w->t.data, w->t.dtype, (char *)out.t.data + at * 4, FG_F32, w->t.numel(), rt.stream);
-                at += (size_t)w->t.numel();
-            }
-            return out;
+            std::vector<Weight> ws = {tensor_of(tensors, a), tensor_of(tensors, b)};
+            if (!v_from_k_) ws.push_back(tensor_of(tensors, c));
+            for (auto &w : ws) { w.t.rows = w.t.numel() / cols; w.t.cols = w.t.ld = cols; }
+            if (differential_) ws[0] = gather_rows(ws[0], map_order(), rt.stream);
+            return concat_rows(ws, FG_F32, rt.stream);          // row-major [channels, cols]: they lie one after another
         };
         if (bias_) bias_w_ = three("q_proj.bias", "k_proj.bias", "v_proj.bias", 1);
         if (taps_ > 0) conv_w_ = three("q_conv.weight", "k_conv.weight", "v_conv.weight", taps_);
         if (qk_norm_) { qn_w_ = as_f32(tensor_of(tensors, "q_norm.weight"), rt.stream); kn_w_ = as_f32(tensor_of(tensors, "k_norm.weight"), rt.stream); }
+        if (differential_) {
+            // lambda: one number for the layer, from vectors of the checkpoint: formed once, on the host, in double precision
+            double dot[2] = {0.0, 0.0};
+            const char *names[4] = {"lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2"};
+            std::vector<float> v[4];
+            for (int i = 0; i < 4; i++) {
+                Weight w = as_f32(tensor_of(tensors, names[i]), rt.stream);
+                v[i].resize((size_t)hd_);
+                FG_CUDA(cudaMemcpyAsync(v[i].data(), w.t.data, (size_t)hd_ * sizeof(float), cudaMemcpyDeviceToHost, rt.stream));
+                FG_CUDA(cudaStreamSynchronize(rt.stream));
+            }
+            for (int i = 0; i < 2; i++)
+                for (int d = 0; d < hd_; d++) dot[i] += (double)v[2 * i][(size_t)d] * (double)v[2 * i + 1][(size_t)d];
+            lambda_ = (float)(std::exp(dot[0]) - std::exp(dot[1]) + (double)diff_);
+        }
         if (sink_) sinks_w_ = as_f32(tensor_of(tensors, "sinks"), rt.stream);
         if (unit_sink_) {
             sinks_w_ = make_weight(1, H_, FG_F32, "unit sinks");
@@ -172,43 +201,52 @@ public:
         // the projections feed a convolution, a norm and a rotation: they stay float32 until those are done
         Tensor proj = qkv_.forward(rt, xn, deferred, Tensor(), FG_F32, false, nullptr, nullptr);
         const int M = (int)proj.rows;
-        Tensor q = rt.arena->matrix(M, (int64_t)H_ * hd_, rt.dtype);
+        const int HQ = maps_ * H_, HK = maps_ * KV_;         // heads the kernels see
+        Tensor q = rt.arena->matrix(M, (int64_t)HQ * hd_, rt.dtype);
         const float *bias = bias_ ? bias_w_.t.ptr<float>() : nullptr;
         FG_LAUNCH("mix", fg_qkv_prepare_ext, proj.ptr<float>(), (int)proj.ld, bias, taps_ > 0 ? conv_w_.t.ptr<float>() : nullptr, taps_,
                   (const float *)io.state, qk_norm_ ? qn_w_.t.ptr<float>() : nullptr, qk_norm_ ? kn_w_.t.ptr<float>() : nullptr, eps_,
                   position_ ? position_->cos_table() : nullptr, position_ ? position_->sin_table() : nullptr, hd_ / 2, position_ ? rot_dims_ : 0,
-                  b.positions, b.row_seq, b.cu_rows, b.slots, table, b.table_width, q.data, (int)q.ld, io.k_pool, io.v_pool, rt.dtype, M, H_, KV_,
-                  hd_, hdv_, io.page_size, norm_per_head_ ? 1 : 0, rot_halves_ ? 1 : 0, rt.stream);
+                  b.positions, b.row_seq, b.cu_rows, b.slots, table, b.table_width, q.data, (int)q.ld, io.k_pool, io.v_pool, rt.dtype, M, HQ, HK,
+                  hd_, hdv_, io.page_size, norm_per_head_ ? 1 : 0, rot_halves_ ? 1 : 0, KV_, v_from_k_ ? 1 : 0, rt.stream);
         if (taps_ > 1)
             FG_LAUNCH("mix", fg_conv_state_update, proj.ptr<float>(), (int)proj.ld, bias, taps_, (float *)io.state, b.cu_rows, b.slots, b.n_seq,
                       (int)channels(), rt.stream);
         // (with an output bias the rows are wider than the heads' outputs: the columns behind them carry the ones)
+        // (two maps: their outputs side by side in float32; the difference, normalised, is what the projection reads)
         Tensor attn = rt.arena->matrix(M, (int64_t)H_ * hdv_ + pad_, rt.dtype);
+        Tensor each = differential_ ? rt.arena->matrix(M, (int64_t)HQ * hdv_, FG_F32) : attn;
+        const int f32_out = differential_ ? 1 : 0;
         const float *sinks = (sink_ || unit_sink_) ? sinks_w_.t.ptr<float>() : nullptr;
         const int mask = chunk_ > 0 ? -chunk_ : window_;     // what the kernels call a window: negative for a chunked mask
-        // bfloat16 with head size 64 / 128 for keys and values alike: the tensor-core kernels (a decode step: mma.sync with the
+        // bfloat16 with head size 64 / 128 for keys and values alike, or keys of 64 beside values of 128: the tensor-core kernels (a decode step: mma.sync with the
         // pages split over a cluster; portions: tcgen05 tiles of 128 rows, or mma.sync tiles of 64 for a few rows)
-        const bool fast = !rt.plain_kernels && rt.dtype == FG_BF16 && io.cache_dtype == FG_BF16 && (hd_ == 64 || hd_ == 128) && hdv_ == hd_ &&
+        const bool fast = !rt.plain_kernels && rt.dtype == FG_BF16 && io.cache_dtype == FG_BF16 && (hd_ == 64 || hd_ == 128) && (hdv_ == hd_ || (hd_ == 64 && hdv_ == 128)) &&
                           io.page_size == 64 && q.ld % 8 == 0 && ((uintptr_t)q.data % 16) == 0;
         if (fast && b.single_token) {
-            int n_splits = decode_splits(rt.n_sm, b.n_seq, H_, KV_, b.table_width, hd_);
+            int n_splits = decode_splits(rt.n_sm, b.n_seq, HQ, HK, b.table_width, hdv_);
             float *part_o = nullptr, *part_ml = nullptr;
             if (n_splits != 1 && n_splits != 2 && n_splits != 4 && n_splits != 8) {
-                part_o = (float *)rt.arena->alloc((size_t)b.n_seq * H_ * n_splits * hd_ * sizeof(float));
-                part_ml = (float *)rt.arena->alloc((size_t)b.n_seq * H_ * n_splits * 2 * sizeof(float));
+                part_o = (float *)rt.arena->alloc((size_t)b.n_seq * HQ * n_splits * hdv_ * sizeof(float));
+                part_ml = (float *)rt.arena->alloc((size_t)b.n_seq * HQ * n_splits * 2 * sizeof(float));
             }
-            FG_LAUNCH("attn", fg_attention_decode_ext, q.data, (int)q.ld, attn.data, (int)attn.ld, b.positions, table, b.table_width, io.k_pool,
-                      io.v_pool, b.n_seq, H_, KV_, hd_, io.page_size, scale_, mask, 0, n_splits, part_o, part_ml, softcap_, sinks, rt.stream);
+            FG_LAUNCH("attn", fg_attention_decode_ext, q.data, (int)q.ld, each.data, (int)each.ld, b.positions, table, b.table_width, io.k_pool,
+                      io.v_pool, b.n_seq, HQ, HK, hd_, io.page_size, scale_, mask, 0, n_splits, part_o, part_ml, softcap_, sinks, hdv_, maps_, f32_out,
+                      rt.stream);
         } else if (fast && b.max_new * (H_ / KV_) >= 64) {
-            FG_LAUNCH("attn", fg_attention_prefill_tc_ext, q.data, (int)q.ld, attn.data, (int)attn.ld, b.cu_rows, b.seq_start, table, b.table_width,
-                      io.k_pool, io.v_pool, io.n_pages, b.n_seq, b.max_new, H_, KV_, hd_, io.page_size, scale_, mask, 0, softcap_, sinks, rt.stream);
+            FG_LAUNCH("attn", fg_attention_prefill_tc_ext, q.data, (int)q.ld, each.data, (int)each.ld, b.cu_rows, b.seq_start, table, b.table_width,
+                      io.k_pool, io.v_pool, io.n_pages, b.n_seq, b.max_new, HQ, HK, hd_, io.page_size, scale_, mask, 0, softcap_, sinks, hdv_, maps_, f32_out,
+                      rt.stream);
         } else if (fast) {
-            FG_LAUNCH("attn", fg_attention_prefill_ext, q.data, (int)q.ld, attn.data, (int)attn.ld, b.cu_rows, b.seq_start, table, b.table_width,
-                      io.k_pool, io.v_pool, b.n_seq, b.max_new, H_, KV_, hd_, io.page_size, scale_, mask, 0, softcap_, sinks, rt.stream);
+            FG_LAUNCH("attn", fg_attention_prefill_ext, q.data, (int)q.ld, each.data, (int)each.ld, b.cu_rows, b.seq_start, table, b.table_width,
+                      io.k_pool, io.v_pool, b.n_seq, b.max_new, HQ, HK, hd_, io.page_size, scale_, mask, 0, softcap_, sinks, hdv_, maps_, f32_out, rt.stream);
         } else {
-            FG_LAUNCH("core", fg_attention_generic_ext, q.data, (int)q.ld, attn.data, (int)attn.ld, rt.dtype, b.positions, b.row_seq, table,
-                      b.table_width, io.k_pool, io.v_pool, M, H_, KV_, hd_, hdv_, io.page_size, scale_, mask, 0, softcap_, sinks, 0, rt.stream);
+            FG_LAUNCH("core", fg_attention_generic_ext, q.data, (int)q.ld, each.data, (int)each.ld, rt.dtype, b.positions, b.row_seq, table,
+                      b.table_width, io.k_pool, io.v_pool, M, HQ, HK, hd_, hdv_, io.page_size, scale_, mask, 0, softcap_, sinks, 0, maps_, f32_out, rt.stream);
         }
+        if (differential_)
+            FG_LAUNCH("mix", fg_differential_combine, each.ptr<float>(), (int)each.ld, attn.data, attn.dtype, (int)attn.ld, M, H_, KV_, hdv_, lambda_, eps_,
+                      1.0f - diff_, rt.stream);
         if (gate_full_)           // in place: a thread reads and writes its own number
             FG_LAUNCH("mix", fg_gate_slice, attn.data, (int)attn.ld, hdv_, proj.ptr<float>() + channels(), (int)proj.ld, attn.data, (int)attn.ld, attn.dtype, M,
                       H_, hdv_, rt.stream);
@@ -222,6 +260,19 @@ public:
 
 private:
     int E_ = 0, H_ = 0, KV_ = 0, hd_ = 0, hdv_ = 0, window_ = 0, chunk_ = 0, taps_ = 0, rot_dims_ = 0, pad_ = 0;
+    // q's rows in the kernels' order [key head][map][head of the group] from the checkpoint's [head][map]
+    std::vector<int64_t> map_order() const {
+        std::vector<int64_t> rows;
+        const int R = H_ / KV_;
+        for (int g = 0; g < KV_; g++)
+            for (int m = 0; m < 2; m++)
+                for (int i = 0; i < R; i++)
+                    for (int d = 0; d < hd_; d++) rows.push_back(((int64_t)(g * R + i) * 2 + m) * hd_ + d);
+        return rows;
+    }
+    int maps_ = 1;
+    bool v_from_k_ = false, differential_ = false;
+    float diff_ = 0.f, lambda_ = 0.f;
     float scale_ = 1.f, softcap_ = 0.f, eps_ = 1e-6f;
     bool bias_ = false, sink_ = false, unit_sink_ = false, qk_norm_ = false, norm_per_head_ = false, rot_halves_ = false, gate_ = false, gate_full_ = false,
          o_bias_ = false;
@@ -349,10 +400,10 @@ public:
                       b.positions, b.row_seq, tmp_table, width, qx.data, Kx, Vx, M, H_, d_, dr_, dv_, P, shared_kv_ ? 1 : 0, rt.stream);
             if (b.max_new >= 64)
                 FG_LAUNCH("attn", fg_attention_prefill_tc_ext, qx.data, (int)qx.ld, ox.data, (int)ox.ld, b.cu_rows, b.seq_start, tmp_table, width, Kx, Vx,
-                          n_pages, b.n_seq, b.max_new, H_, H_, HQ, P, scale_, 0, 0, 0.f, sinks, rt.stream);
+                          n_pages, b.n_seq, b.max_new, H_, H_, HQ, P, scale_, 0, 0, 0.f, sinks, HQ, 1, 0, rt.stream);
             else
                 FG_LAUNCH("attn", fg_attention_prefill_ext, qx.data, (int)qx.ld, ox.data, (int)ox.ld, b.cu_rows, b.seq_start, tmp_table, width, Kx, Vx,
-                          b.n_seq, b.max_new, H_, H_, HQ, P, scale_, 0, 0, 0.f, sinks, rt.stream);
+                          b.n_seq, b.max_new, H_, H_, HQ, P, scale_, 0, 0, 0.f, sinks, HQ, 1, 0, rt.stream);
             FG_LAUNCH("mix", fg_gate_slice, ox.data, (int)ox.ld, HQ, gate, (int)down.ld, o.data, (int)o.ld, o.dtype, M, H_, dv_, rt.stream);
         } else {
             // per head [q_abs (kv_rank) | q_rot (rot_dim)]
@@ -381,7 +432,7 @@ public:
                           io.k_pool, io.v_pool, M, H_, r_, dr_, io.page_size, scale_, sinks, n_splits, part, rt.stream);
             } else {
                 FG_LAUNCH("core", fg_attention_generic_ext, qf.data, (int)qf.ld, lat.data, (int)lat.ld, rt.dtype, b.positions, b.row_seq, table, b.table_width,
-                          io.k_pool, io.v_pool, M, H_, 1, dr_, r_, io.page_size, scale_, 0, 0, 0.f, sinks, 1, rt.stream);
+                          io.k_pool, io.v_pool, M, H_, 1, dr_, r_, io.page_size, scale_, 0, 0, 0.f, sinks, 1, 1, 0, rt.stream);
             }
             FG_LAUNCH("mix", fg_head_gemm, lat.data, lat.dtype, (int)lat.ld, r_, v_up_.t.data, v_up_.t.dtype, (int)v_up_.t.ld, 0, o.data, o.dtype, (int)o.ld,
                       dv_, gate, (int)down.ld, M, dv_, r_, H_, rt.stream);

@@ -12,6 +12,9 @@
 // per sequence slot (zeroed when a sequence takes the slot), and so are the projections' results that enter the
 // recurrence: the contraction writes float32 and the kernels of retention.cu keep rotation, decay powers, scores, the
 // unit norm and the gate in float32; y takes the engine's dtype for the output projection.
+// Options: "qkv_activation": "silu" - q, k and v each pass silu (before a rotation); "norm": "whole" - instead of the unit norm per
+// head, y = o / sqrt(mean(o^2) + eps) * w over all heads' outputs at once, with a weight [heads * v_head_dim]; "gate_activation":
+// "sigmoid" - sigmoid(g) in place of silu(g) (with "norm": "whole").  k_scale 1 and no position: nothing else happens to k.
 // A decode step and short portions walk their tokens one after another with S in shared memory; portions of
 // `chunk_threshold` tokens and more run in chunks over all sequences at once (retention.cu says how).
 #include <cmath>
@@ -31,7 +34,6 @@ public:
         eps_ = (float)param_float(p, "eps", me);
         k_scale_ = (float)param_float(p, "k_scale", 1.0 / std::sqrt((double)dk_), me);
         if (E_ <= 0 || H_ <= 0 || dk_ <= 0 || dv_ <= 0) fail(FG_E_CONFIG, "retention: sizes must be positive");
-        if (dk_ % 2) fail(FG_E_CONFIG, format("retention: head_dim must be even, got %d", dk_));
         if (dv_ > 256) fail(FG_E_CONFIG, format("retention: v_head_dim %d exceeds 256, the largest the kernels take", dv_));
         if ((size_t)dk_ * dv_ > 40 * 1024) fail(FG_E_CONFIG, "retention: a head's state exceeds what the kernels hold in shared memory");
         if (!(eps_ > 0.f)) fail(FG_E_CONFIG, "retention: eps must be positive");
@@ -43,6 +45,17 @@ public:
             decay_.push_back((float)v.as_double());
             all_positive_ = all_positive_ && v.as_double() > 0.0;
         }
+        auto option = [&](const char *key, const char *plain, const char *other) {
+            const Json &v = p.get(key);
+            if (v.is_null() || (v.is_string() && v.as_string() == plain)) return false;
+            if (!v.is_string() || v.as_string() != other)
+                fail(FG_E_CONFIG, format("retention: %s %s is not known (known: %s, %s)", key, v.dump().c_str(), plain, other));
+            return true;
+        };
+        silu_ = option("qkv_activation", "none", "silu");
+        whole_norm_ = option("norm", "head", "whole");
+        sigmoid_gate_ = option("gate_activation", "silu", "sigmoid");
+        if (sigmoid_gate_ && !whole_norm_) fail(FG_E_CONFIG, "retention: a sigmoid gate needs norm 'whole'");
         const Json &pos = p.get("position");
         if (!pos.is_null()) {
             position_ = dynamic_cast<PositionEncoding *>(ctx.nested(FG_ROLE_POSITION, pos));
@@ -53,10 +66,13 @@ public:
     }
     std::vector<TensorDecl> tensor_decls() const override {
         int64_t Q = (int64_t)H_ * dk_, V = (int64_t)H_ * dv_;
-        return {{"q_proj.weight", {Q, E_}}, {"k_proj.weight", {Q, E_}}, {"v_proj.weight", {V, E_}}, {"g_proj.weight", {V, E_}},
-                {"o_proj.weight", {E_, V}}};
+        std::vector<TensorDecl> d = {{"q_proj.weight", {Q, E_}}, {"k_proj.weight", {Q, E_}}, {"v_proj.weight", {V, E_}}, {"g_proj.weight", {V, E_}},
+                                     {"o_proj.weight", {E_, V}}};
+        if (whole_norm_) d.push_back({"norm.weight", {V}, false, 1, 0.01f});
+        return d;
     }
     bool can_overwrite() const override { return true; }
+    bool supports_deferred_norm() const override { return true; }
     int64_t state_bytes() const override { return (int64_t)H_ * dk_ * dv_ * (int64_t)sizeof(float); }
     void load(const std::map<std::string, Weight> &tensors, Runtime &rt) override {
         Weight q = tensor_of(tensors, "q_proj.weight"), k = tensor_of(tensors, "k_proj.weight");
@@ -73,32 +89,27 @@ public:
         bool same = q.t.dtype == k.t.dtype && k.t.dtype == v.t.dtype && v.t.dtype == g.t.dtype;
         proj_ = Linear(concat_rows({q, k, v, g}, same ? q.t.dtype : FG_F32, rt.stream));
         o_ = Linear(tensor_of(tensors, "o_proj.weight"));
+        if (whole_norm_) {
+            const Weight &w = tensor_of(tensors, "norm.weight");
+            norm_w_ = w.t.dtype == FG_F32 ? w : concat_rows({w}, FG_F32, rt.stream);
+        }
         decay_dev_ = make_weight(1, H_, FG_F32, "retention decays");
         FG_CUDA(cudaMemcpyAsync(decay_dev_.t.data, decay_.data(), decay_.size() * sizeof(float), cudaMemcpyHostToDevice, rt.stream));
         FG_CUDA(cudaStreamSynchronize(rt.stream));
     }
-    void prepare(Runtime &rt, int max_positions) override {
-        if (position_) { position_->prepare(rt, max_positions); return; }
-        // no rotation: identity tables, so that one kernel serves both
-        if (ident_cos_.buffer && ident_positions_ >= max_positions) return;
-        int half = dk_ / 2;
-        std::vector<float> c((size_t)max_positions * half, 1.0f);
-        ident_cos_ = make_weight(max_positions, half, FG_F32, "identity rotation tables");
-        ident_sin_ = make_weight(max_positions, half, FG_F32, "identity rotation tables");
-        FG_CUDA(cudaMemcpyAsync(ident_cos_.t.data, c.data(), c.size() * 4, cudaMemcpyHostToDevice, rt.stream));
-        FG_CUDA(cudaMemsetAsync(ident_sin_.t.data, 0, c.size() * 4, rt.stream));
-        FG_CUDA(cudaStreamSynchronize(rt.stream));
-        ident_positions_ = max_positions;
-    }
-    DeferredNorm forward(Runtime &rt, const Tensor &xn, const DeferredNorm *, const Batch &b, const LayerIO &io, Tensor &residual,
+    void prepare(Runtime &rt, int max_positions) override { if (position_) position_->prepare(rt, max_positions); }
+    DeferredNorm forward(Runtime &rt, const Tensor &xn, const DeferredNorm *deferred, const Batch &b, const LayerIO &io, Tensor &residual,
                          Norm *emit_norm) override {
         if (!io.state || io.state_bytes < state_bytes()) fail(FG_E_INTERNAL, "retention: the schedule entry has no state rows");
-        const float *cos_t = position_ ? position_->cos_table() : ident_cos_.t.ptr<float>();
-        const float *sin_t = position_ ? position_->sin_table() : ident_sin_.t.ptr<float>();
+        const float *cos_t = position_ ? position_->cos_table() : nullptr;
+        const float *sin_t = position_ ? position_->sin_table() : nullptr;
         // what enters the recurrence stays float32: the contraction accumulates in float32 and writes it as it is
-        Tensor proj = proj_.forward(rt, xn, nullptr, Tensor(), FG_F32, false, nullptr, nullptr);
+        Tensor proj = proj_.forward(rt, xn, deferred, Tensor(), FG_F32, false, nullptr, nullptr);
         const int M = (int)proj.rows;
         Tensor y = rt.arena->matrix(M, (int64_t)H_ * dv_, rt.dtype);
+        // (a norm over all heads: the recurrence's sums stay float32 until that norm is done)
+        Tensor o = whole_norm_ ? rt.arena->matrix(M, (int64_t)H_ * dv_, FG_F32) : y;
+        const int opts = (silu_ ? 1 : 0) | (whole_norm_ ? 2 : 0);
         const int *host_cu = b.host_cu_rows.empty() ? nullptr : b.host_cu_rows.data();
         const int RC = FG_KERNEL("mix", fg_retention_chunk_tokens)();
         bool chunked = host_cu && !b.single_token && all_positive_ && b.max_new >= chunk_threshold_ &&
@@ -109,26 +120,29 @@ public:
             for (int s = 0; s < b.n_seq; s++) n_chunks += (host_cu[s + 1] - host_cu[s] + RC - 1) / RC;
             int *plan = (int *)rt.arena->alloc(((size_t)2 * n_chunks + b.n_seq + 1) * sizeof(int));
             float *U = (float *)rt.arena->alloc((size_t)n_chunks * H_ * dk_ * dv_ * sizeof(float));
-            FG_LAUNCH("mix", fg_retention_chunked, proj.ptr<float>(), (int)proj.ld, y.data, y.dtype, (int)y.ld, b.positions, b.cu_rows,
+            FG_LAUNCH("mix", fg_retention_chunked, proj.ptr<float>(), (int)proj.ld, o.data, o.dtype, (int)o.ld, b.positions, b.cu_rows,
                       b.slots, cos_t, sin_t, decay_dev_.t.ptr<float>(), (float *)io.state, plan, U, b.n_seq, n_chunks, H_, dk_, dv_,
-                      k_scale_, eps_, rt.stream);
+                      k_scale_, eps_, opts, rt.stream);
         } else {
-            FG_LAUNCH("mix", fg_retention, proj.ptr<float>(), (int)proj.ld, y.data, y.dtype, (int)y.ld, b.positions, b.cu_rows, b.slots, cos_t,
-                      sin_t, decay_dev_.t.ptr<float>(), (float *)io.state, b.n_seq, H_, dk_, dv_, k_scale_, eps_, rt.stream);
+            FG_LAUNCH("mix", fg_retention, proj.ptr<float>(), (int)proj.ld, o.data, o.dtype, (int)o.ld, b.positions, b.cu_rows, b.slots, cos_t,
+                      sin_t, decay_dev_.t.ptr<float>(), (float *)io.state, b.n_seq, H_, dk_, dv_, k_scale_, eps_, opts, rt.stream);
         }
+        if (whole_norm_)
+            FG_LAUNCH("mix", fg_gated_group_norm, o.ptr<float>(), (int)o.ld, proj.ptr<float>() + (int64_t)2 * H_ * dk_ + (int64_t)H_ * dv_, (int)proj.ld,
+                      norm_w_.t.ptr<float>(), H_ * dv_, y.data, y.dtype, (int)y.ld, M, H_ * dv_, H_ * dv_, eps_, 0, sigmoid_gate_ ? 1 : 0, rt.stream);
         DeferredNorm started;
         o_.forward(rt, y, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
         return started;
     }
 
 private:
-    int E_ = 0, H_ = 0, dk_ = 0, dv_ = 0, chunk_threshold_ = 16, ident_positions_ = 0;
+    int E_ = 0, H_ = 0, dk_ = 0, dv_ = 0, chunk_threshold_ = 16;
     float eps_ = 0.f, k_scale_ = 1.f;
-    bool all_positive_ = true;
+    bool all_positive_ = true, silu_ = false, whole_norm_ = false, sigmoid_gate_ = false;
     std::vector<float> decay_;
     PositionEncoding *position_ = nullptr;
     Linear proj_, o_;
-    Weight decay_dev_, ident_cos_, ident_sin_;
+    Weight decay_dev_, norm_w_;
 };
 
 // "gated_linear_attention": linear attention whose state decays per key channel by a factor the token itself decides.
@@ -311,7 +325,7 @@ public:
                   y.ptr<float>(), (int)y.ld, b.cu_rows, b.slots, state + conv_floats(), stride, b.n_seq, H_, G_, N_, dv_, 0, rt.stream);
         Tensor yn = rt.arena->matrix(M, I, rt.dtype);
         FG_LAUNCH("mix", fg_gated_group_norm, y.ptr<float>(), (int)y.ld, proj.ptr<float>(), ld, norm_.t.ptr<float>(), I, yn.data, yn.dtype, (int)yn.ld, M, I,
-                  I / norm_groups_, eps_, 1, rt.stream);
+                  I / norm_groups_, eps_, 1, 0, rt.stream);
         DeferredNorm started;
         o_.forward(rt, yn, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
         return started;
@@ -410,7 +424,7 @@ public:
                   (int)o.ld, b.cu_rows, b.slots, state + conv_floats(), stride, b.n_seq, H_, G_, d_, dv_, 1, rt.stream);
         Tensor y = rt.arena->matrix(M, V, rt.dtype);
         FG_LAUNCH("mix", fg_gated_group_norm, o.ptr<float>(), (int)o.ld, proj.ptr<float>() + C + 2 * H_, ld, norm_.t.ptr<float>(), dv_, y.data, y.dtype,
-                  (int)y.ld, M, V, dv_, eps_, 0, rt.stream);
+                  (int)y.ld, M, V, dv_, eps_, 0, 0, rt.stream);
         DeferredNorm started;
         o_.forward(rt, y, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
         return started;

@@ -232,10 +232,13 @@ decay_recurrence_kernel(const float *__restrict__ q, int ldq, const float *__res
 // ------------------------------------------------------------------ gate and norm behind the recurrence
 // gate_first: t = y * silu(g), out = t / rms_group(t) * w[c]                         (groups of `group` neighbouring channels)
 // else:       out = y / rms_group(y) * w[c % w_period] * silu(g)
+// sigmoid_gate: sigmoid(g) where silu(g) stands
+__device__ __forceinline__ float rec_gate(float z, int sigmoid_gate) { return (sigmoid_gate ? 1.0f : z) / (1.0f + expf(-z)); }
 template <typename TO>
 __global__ void __launch_bounds__(256)
 gated_group_norm_kernel(const float *__restrict__ y, int ldy, const float *__restrict__ g, int ldg, const float *__restrict__ w,
-                        int w_period, TO *__restrict__ out, int ldo, int C, int group, float eps, int gate_first) {
+                        int w_period, TO *__restrict__ out, int ldo, int C, int group, float eps, int gate_first,
+                        int sigmoid_gate) {
     __shared__ float scratch[32];
     pdl_wait();
     const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -247,13 +250,13 @@ gated_group_norm_kernel(const float *__restrict__ y, int ldy, const float *__res
         for (int b0 = blockIdx.y * group; b0 < C; b0 += gridDim.y * group) {
             float ss = 0.f;
             for (int i = threadIdx.x; i < group; i += 256) {
-                const float t = gate_first ? yr[b0 + i] * rec_silu(gr[b0 + i]) : yr[b0 + i];
+                const float t = gate_first ? yr[b0 + i] * rec_gate(gr[b0 + i], sigmoid_gate) : yr[b0 + i];
                 ss = fmaf(t, t, ss);
             }
             const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)group + eps);
             for (int i = threadIdx.x; i < group; i += 256) {
                 const int c = b0 + i;
-                const float sg = rec_silu(gr[c]);
+                const float sg = rec_gate(gr[c], sigmoid_gate);
                 const float wc = w[whole ? c : (by_group ? i : c % w_period)];        // (no division where the weight spans the row or a group)
                 orow[c] = from_f32<TO>(gate_first ? yr[c] * sg * inv * wc : yr[c] * inv * wc * sg);
             }
@@ -264,14 +267,14 @@ gated_group_norm_kernel(const float *__restrict__ y, int ldy, const float *__res
         const int b0 = grp * group;
         float ss = 0.f;
         for (int i = lane; i < group; i += 32) {
-            const float t = gate_first ? yr[b0 + i] * rec_silu(gr[b0 + i]) : yr[b0 + i];
+            const float t = gate_first ? yr[b0 + i] * rec_gate(gr[b0 + i], sigmoid_gate) : yr[b0 + i];
             ss = fmaf(t, t, ss);
         }
         ss = warp_sum(ss);
         const float inv = 1.0f / sqrtf(ss / (float)group + eps);
         for (int i = lane; i < group; i += 32) {
             const int c = b0 + i;
-            const float sg = rec_silu(gr[c]);
+            const float sg = rec_gate(gr[c], sigmoid_gate);
             const float wc = w[whole ? c : (by_group ? i : c % w_period)];        // (no division where the weight spans the row or a group)
                 orow[c] = from_f32<TO>(gate_first ? yr[c] * sg * inv * wc : yr[c] * inv * wc * sg);
         }
@@ -369,16 +372,17 @@ extern "C" int fg_decay_recurrence(const float *q, int ldq, const float *k, int 
 }
 
 extern "C" int fg_gated_group_norm(const float *y, int ldy, const float *g, int ldg, const float *w, int w_period, void *out,
-                                   int out_dtype, int ldo, int M, int C, int group, float eps, int gate_first, cudaStream_t stream) {
+                                   int out_dtype, int ldo, int M, int C, int group, float eps, int gate_first, int sigmoid_gate,
+                                   cudaStream_t stream) {
     if (M <= 0) return 0;
     if (C <= 0 || group <= 0 || C % group || w_period <= 0) return FG_ERR_BAD_SIZE;
     const int groups = C / group;
     dim3 grid(M, group >= 1024 ? (groups < 4 ? groups : 4) : groups >= 64 ? 4 : 1);
     if (out_dtype == FG_F32)
         return fg_launch(gated_group_norm_kernel<float>, grid, dim3(256), 0, stream, y, ldy, g, ldg, w, w_period, (float *)out, ldo, C, group,
-                                  eps, gate_first);
+                                  eps, gate_first, sigmoid_gate);
     if (out_dtype == FG_BF16)
         return fg_launch(gated_group_norm_kernel<bf16>, grid, dim3(256), 0, stream, y, ldy, g, ldg, w, w_period, (bf16 *)out, ldo, C, group,
-                                  eps, gate_first);
+                                  eps, gate_first, sigmoid_gate);
     return FG_ERR_BAD_DTYPE;
 }

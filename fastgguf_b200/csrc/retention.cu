@@ -11,6 +11,9 @@
 // Rotation tables cos/sin are [positions, dk / 2] for pairs (j, j + dk / 2); dimensions that are not rotated have
 // cos 1, sin 0 (the rows of the q and k projections are permuted into that form when the weights are loaded).
 //
+// Options (`opts`, a sum): RET_SILU - q, k and v each pass silu as they are read; RET_RAW - the outputs are the sums o_t themselves,
+// without unit norm and gate (for a norm that spans the heads, in a kernel of its own).  Without tables (null) nothing is rotated.
+//
 // Two forms:
 //   * retention_seq_kernel: one block per (sequence, head) walks its tokens one after another with S in shared memory.
 //     A decode step (one token a sequence) and short portions run this way.
@@ -23,6 +26,8 @@
 
 #define RET_THREADS 256
 #define RC 32                       // tokens a chunk
+#define RET_SILU 1
+#define RET_RAW 2
 
 template <typename TO> __device__ __forceinline__ void store4(TO *dst, float a, float b, float c, float d);
 template <> __device__ __forceinline__ void store4<float>(float *dst, float a, float b, float c, float d) {
@@ -35,12 +40,18 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16 *dst, float a, flo
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
+__device__ __forceinline__ float opt_silu(float z, int opts) { return (opts & RET_SILU) ? silu_f(z) : z; }
+
 // rotate pair (j, j + half) of head vector `src` at position pos into dst (shared memory), times `mul`
 __device__ __forceinline__ void rotate_into(const float *__restrict__ src, float *dst, int dk, const float *cs, const float *sn,
-                                            float mul, int tid, int nthreads) {
+                                            float mul, int opts, int tid, int nthreads) {
+    if (!cs) {
+        for (int j = tid; j < dk; j += nthreads) dst[j] = opt_silu(src[j], opts) * mul;
+        return;
+    }
     const int half = dk >> 1;
     for (int j = tid; j < half; j += nthreads) {
-        float a = src[j], b = src[j + half], c = cs[j], s = sn[j];
+        float a = opt_silu(src[j], opts), b = opt_silu(src[j + half], opts), c = cs[j], s = sn[j];
         dst[j] = (a * c - b * s) * mul;
         dst[j + half] = (b * c + a * s) * mul;
     }
@@ -51,25 +62,34 @@ __device__ __forceinline__ void rotate_into(const float *__restrict__ src, float
 template <bool DECAY>
 __device__ __forceinline__ void rotate_chunk_into(const float *__restrict__ proj, int ld, int r0, int n, size_t head_off, float *dst,
                                                   int stride, int dk, const int *__restrict__ positions,
-                                                  const float *__restrict__ cos_t, const float *__restrict__ sin_t, float mul, float l2,
+                                                  const float *__restrict__ cos_t, const float *__restrict__ sin_t, float mul, float l2, int opts,
                                                   int tid) {
+    if (!cos_t) {
+#pragma unroll 4
+        for (int e = tid; e < n * dk; e += RET_THREADS) {
+            const int t = e / dk, j = e - t * dk;
+            const float m = DECAY ? mul * exp2f(l2 * (float)(n - 1 - t)) : mul;
+            dst[t * stride + j] = opt_silu(proj[(size_t)(r0 + t) * ld + head_off + j], opts) * m;
+        }
+        return;
+    }
     const int half = dk >> 1;
 #pragma unroll 4
     for (int e = tid; e < n * half; e += RET_THREADS) {
         const int t = e / half, j = e - t * half;
         const float *src = proj + (size_t)(r0 + t) * ld + head_off;
         const int pos = positions[r0 + t];
-        const float a = src[j], b = src[j + half], c = cos_t[(size_t)pos * half + j], sn = sin_t[(size_t)pos * half + j];
+        const float a = opt_silu(src[j], opts), b = opt_silu(src[j + half], opts), c = cos_t[(size_t)pos * half + j], sn = sin_t[(size_t)pos * half + j];
         const float m = DECAY ? mul * exp2f(l2 * (float)(n - 1 - t)) : mul;
         dst[t * stride + j] = (a * c - b * sn) * m;
         dst[t * stride + j + half] = (b * c + a * sn) * m;
     }
 }
-__device__ __forceinline__ void copy_chunk_into(const float *__restrict__ proj, int ld, int r0, int n, size_t off, float *dst, int dv, int tid) {
+__device__ __forceinline__ void copy_chunk_into(const float *__restrict__ proj, int ld, int r0, int n, size_t off, float *dst, int dv, int opts, int tid) {
 #pragma unroll 4
     for (int e = tid; e < n * dv; e += RET_THREADS) {
         const int t = e / dv, j = e - t * dv;
-        dst[e] = proj[(size_t)(r0 + t) * ld + off + j];
+        dst[e] = opt_silu(proj[(size_t)(r0 + t) * ld + off + j], opts);
     }
 }
 
@@ -78,7 +98,7 @@ __global__ void __launch_bounds__(RET_THREADS)
 retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ out, int ldo, const int *__restrict__ positions,
                      const int *__restrict__ cu_rows, const int *__restrict__ slots, const float *__restrict__ cos_t,
                      const float *__restrict__ sin_t, const float *__restrict__ decay, float *__restrict__ state, int H, int dk,
-                     int dv, float k_scale, float eps) {
+                     int dv, float k_scale, float eps, int opts) {
     extern __shared__ float sm[];
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -95,10 +115,10 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
     for (int r = row0; r < row1; r++) {
         const float *row = proj + (size_t)r * ld;
         const int pos = positions[r];
-        const float *cs = cos_t + (size_t)pos * half, *sn = sin_t + (size_t)pos * half;
-        rotate_into(row + (size_t)h * dk, qs, dk, cs, sn, 1.0f, tid, RET_THREADS);
-        rotate_into(row + (size_t)(H + h) * dk, ks, dk, cs, sn, k_scale, tid, RET_THREADS);
-        for (int j = tid; j < dv; j += RET_THREADS) vs[j] = row[(size_t)2 * H * dk + (size_t)h * dv + j];
+        const float *cs = cos_t ? cos_t + (size_t)pos * half : nullptr, *sn = cos_t ? sin_t + (size_t)pos * half : nullptr;
+        rotate_into(row + (size_t)h * dk, qs, dk, cs, sn, 1.0f, opts, tid, RET_THREADS);
+        rotate_into(row + (size_t)(H + h) * dk, ks, dk, cs, sn, k_scale, opts, tid, RET_THREADS);
+        for (int j = tid; j < dv; j += RET_THREADS) vs[j] = opt_silu(row[(size_t)2 * H * dk + (size_t)h * dv + j], opts);
         __syncthreads();
         if (tid < n_active) {
             const int j = tid % dv, g = tid / dv;
@@ -115,6 +135,11 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
         float o = 0.f;
         if (tid < dv)
             for (int g = 0; g < G; g++) o += part[g * dv + tid];
+        if (opts & RET_RAW) {
+            if (tid < dv) out[(size_t)r * ldo + (size_t)h * dv + tid] = from_f32<TO>(o);
+            __syncthreads();                   // part is rewritten by the next token
+            continue;
+        }
         float ss = block_sum(tid < dv ? o * o : 0.f, scratch);
         if (tid < dv) {
             float gate = row[(size_t)2 * H * dk + (size_t)(H + h) * dv + tid];
@@ -151,7 +176,7 @@ __global__ void __launch_bounds__(RET_THREADS)
 retention_chunk_state_kernel(const float *__restrict__ proj, int ld, const int *__restrict__ positions,
                              const int *__restrict__ chunk_row, const int *__restrict__ chunk_len,
                              const float *__restrict__ cos_t, const float *__restrict__ sin_t, const float *__restrict__ decay,
-                             float *__restrict__ U, int H, int dk, int dv, float k_scale) {
+                             float *__restrict__ U, int H, int dk, int dv, float k_scale, int opts) {
     extern __shared__ float sm[];
     pdl_launch_dependents();
     pdl_wait();
@@ -163,9 +188,9 @@ retention_chunk_state_kernel(const float *__restrict__ proj, int ld, const int *
     for (int t = 0; t < n; t++) {
         const float *row = proj + (size_t)(r0 + t) * ld;
         const int pos = positions[r0 + t];
-        rotate_into(row + (size_t)(H + h) * dk, K + t * dk, dk, cos_t + (size_t)pos * half, sin_t + (size_t)pos * half,
-                    k_scale * exp2f(l2 * (float)(n - 1 - t)), tid, RET_THREADS);
-        for (int j = tid; j < dv; j += RET_THREADS) V[t * dv + j] = row[(size_t)2 * H * dk + (size_t)h * dv + j];
+        rotate_into(row + (size_t)(H + h) * dk, K + t * dk, dk, cos_t ? cos_t + (size_t)pos * half : nullptr,
+                    cos_t ? sin_t + (size_t)pos * half : nullptr, k_scale * exp2f(l2 * (float)(n - 1 - t)), opts, tid, RET_THREADS);
+        for (int j = tid; j < dv; j += RET_THREADS) V[t * dv + j] = opt_silu(row[(size_t)2 * H * dk + (size_t)h * dv + j], opts);
     }
     __syncthreads();
     const int G = RET_THREADS / dv;
@@ -228,7 +253,7 @@ __global__ void __launch_bounds__(RET_THREADS)
 retention_chunk_out_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ out, int ldo, const int *__restrict__ positions,
                            const int *__restrict__ chunk_row, const int *__restrict__ chunk_len, const float *__restrict__ cos_t,
                            const float *__restrict__ sin_t, const float *__restrict__ decay, const float *__restrict__ U, int H,
-                           int dk, int dv, float k_scale, float eps) {
+                           int dk, int dv, float k_scale, float eps, int opts) {
     extern __shared__ float sm[];
     pdl_launch_dependents();
     pdl_wait();
@@ -241,10 +266,10 @@ retention_chunk_out_kernel(const float *__restrict__ proj, int ld, TO *__restric
     for (int t = 0; t < n; t++) {
         const float *row = proj + (size_t)(r0 + t) * ld;
         const int pos = positions[r0 + t];
-        const float *cs = cos_t + (size_t)pos * half, *sn = sin_t + (size_t)pos * half;
-        rotate_into(row + (size_t)h * dk, Q + t * dkp, dk, cs, sn, 1.0f, tid, RET_THREADS);
-        rotate_into(row + (size_t)(H + h) * dk, K + t * dkp, dk, cs, sn, k_scale, tid, RET_THREADS);
-        for (int j = tid; j < dv; j += RET_THREADS) V[t * dv + j] = row[(size_t)2 * H * dk + (size_t)h * dv + j];
+        const float *cs = cos_t ? cos_t + (size_t)pos * half : nullptr, *sn = cos_t ? sin_t + (size_t)pos * half : nullptr;
+        rotate_into(row + (size_t)h * dk, Q + t * dkp, dk, cs, sn, 1.0f, opts, tid, RET_THREADS);
+        rotate_into(row + (size_t)(H + h) * dk, K + t * dkp, dk, cs, sn, k_scale, opts, tid, RET_THREADS);
+        for (int j = tid; j < dv; j += RET_THREADS) V[t * dv + j] = opt_silu(row[(size_t)2 * H * dk + (size_t)h * dv + j], opts);
     }
     __syncthreads();
     for (int e = tid; e < n * RC; e += RET_THREADS) {
@@ -282,6 +307,13 @@ retention_chunk_out_kernel(const float *__restrict__ proj, int ld, TO *__restric
         }
     }
     __syncthreads();
+    if (opts & RET_RAW) {
+        for (int e = tid; e < n * dv; e += RET_THREADS) {
+            const int i = e / dv, j = e % dv;
+            out[(size_t)(r0 + i) * ldo + (size_t)h * dv + j] = from_f32<TO>(O[e]);
+        }
+        return;
+    }
     // unit norm of each token's head vector: a warp per token
     const int warp = tid >> 5, lane = tid & 31;
     for (int i = warp; i < n; i += RET_THREADS / 32) {
@@ -309,7 +341,7 @@ __global__ void __launch_bounds__(RET_THREADS)
 retention_chunk_state_fast(const float *__restrict__ proj, int ld, const int *__restrict__ positions,
                            const int *__restrict__ chunk_row, const int *__restrict__ chunk_len,
                            const float *__restrict__ cos_t, const float *__restrict__ sin_t, const float *__restrict__ decay,
-                           float *__restrict__ U, int H, float k_scale) {
+                           float *__restrict__ U, int H, float k_scale, int opts) {
     constexpr int NJ = DV / 4, NI = RET_THREADS / NJ, TI = DK / NI;
     __shared__ __align__(16) float K[RC * DK];
     __shared__ __align__(16) float V[RC * DV];
@@ -318,8 +350,8 @@ retention_chunk_state_fast(const float *__restrict__ proj, int ld, const int *__
     const int c = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int r0 = chunk_row[c], n = chunk_len[c];
     const float l2 = log2f(decay[h]);
-    rotate_chunk_into<true>(proj, ld, r0, n, (size_t)(H + h) * DK, K, DK, DK, positions, cos_t, sin_t, k_scale, l2, tid);
-    copy_chunk_into(proj, ld, r0, n, (size_t)2 * H * DK + (size_t)h * DV, V, DV, tid);
+    rotate_chunk_into<true>(proj, ld, r0, n, (size_t)(H + h) * DK, K, DK, DK, positions, cos_t, sin_t, k_scale, l2, opts, tid);
+    copy_chunk_into(proj, ld, r0, n, (size_t)2 * H * DK + (size_t)h * DV, V, DV, opts, tid);
     __syncthreads();
     const int tj = tid % NJ, ti = tid / NJ;
     float acc[TI][4];
@@ -347,7 +379,7 @@ __global__ void __launch_bounds__(RET_THREADS)
 retention_chunk_out_fast(const float *__restrict__ proj, int ld, TO *__restrict__ out, int ldo, const int *__restrict__ positions,
                          const int *__restrict__ chunk_row, const int *__restrict__ chunk_len, const float *__restrict__ cos_t,
                          const float *__restrict__ sin_t, const float *__restrict__ decay, const float *__restrict__ U, int H,
-                         float k_scale, float eps) {
+                         float k_scale, float eps, int opts) {
     constexpr int NJ = DV / 4, NI = RET_THREADS / NJ, TT = RC / NI, DKP = DK + 4;
     extern __shared__ __align__(16) float sm[];
     float *Q = sm, *K = Q + RC * DKP, *V = K + RC * DKP, *A = V + RC * DV;       // Q, K: [RC][DKP]; V: [RC][DV]; A: [RC][RC]
@@ -356,9 +388,9 @@ retention_chunk_out_fast(const float *__restrict__ proj, int ld, TO *__restrict_
     const int c = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int r0 = chunk_row[c], n = chunk_len[c];
     const float l2 = log2f(decay[h]);
-    rotate_chunk_into<false>(proj, ld, r0, n, (size_t)h * DK, Q, DKP, DK, positions, cos_t, sin_t, 1.0f, 0.f, tid);
-    rotate_chunk_into<false>(proj, ld, r0, n, (size_t)(H + h) * DK, K, DKP, DK, positions, cos_t, sin_t, k_scale, 0.f, tid);
-    copy_chunk_into(proj, ld, r0, n, (size_t)2 * H * DK + (size_t)h * DV, V, DV, tid);
+    rotate_chunk_into<false>(proj, ld, r0, n, (size_t)h * DK, Q, DKP, DK, positions, cos_t, sin_t, 1.0f, 0.f, opts, tid);
+    rotate_chunk_into<false>(proj, ld, r0, n, (size_t)(H + h) * DK, K, DKP, DK, positions, cos_t, sin_t, k_scale, 0.f, opts, tid);
+    copy_chunk_into(proj, ld, r0, n, (size_t)2 * H * DK + (size_t)h * DV, V, DV, opts, tid);
     for (int e = n * DKP + tid; e < RC * DKP; e += RET_THREADS) Q[e] = K[e] = 0.f;       // rows of a short last chunk
     for (int e = n * DV + tid; e < RC * DV; e += RET_THREADS) V[e] = 0.f;
     __syncthreads();
@@ -414,6 +446,10 @@ retention_chunk_out_fast(const float *__restrict__ proj, int ld, TO *__restrict_
 #pragma unroll
     for (int u = 0; u < TT; u++) {
         const int i = ti + u * NI;
+        if (opts & RET_RAW) {
+            if (i < n) store4<TO>(out + (size_t)(r0 + i) * ldo + (size_t)h * DV + tj * 4, acc[u][0], acc[u][1], acc[u][2], acc[u][3]);
+            continue;
+        }
         float ss = acc[u][0] * acc[u][0] + acc[u][1] * acc[u][1] + acc[u][2] * acc[u][2] + acc[u][3] * acc[u][3];
 #pragma unroll
         for (int o = NJ / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -432,9 +468,9 @@ extern "C" int fg_retention_chunk_tokens(void) { return RC; }
 
 extern "C" int fg_retention(const float *proj, int ld, void *out, int out_dtype, int ldo, const int *positions, const int *cu_rows,
                             const int *slots, const float *cos_t, const float *sin_t, const float *decay, float *state, int n_seq,
-                            int H, int dk, int dv, float k_scale, float eps, cudaStream_t stream) {
+                            int H, int dk, int dv, float k_scale, float eps, int opts, cudaStream_t stream) {
     if (n_seq <= 0) return 0;
-    if (dk <= 0 || dk % 2 || dv <= 0 || dv > RET_THREADS || H <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
+    if (dk <= 0 || (cos_t && dk % 2) || dv <= 0 || dv > RET_THREADS || H <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
     const int G = RET_THREADS / dv;
     size_t smem = ((size_t)dk * dv + 2 * dk + dv + (size_t)G * dv) * sizeof(float);
     if (smem > 200 * 1024) return FG_ERR_BAD_SIZE;
@@ -447,14 +483,14 @@ extern "C" int fg_retention(const float *proj, int ld, void *out, int out_dtype,
     }
     if (wide)
         return fg_launch(retention_seq_kernel<float>, dim3(n_seq, H), dim3(RET_THREADS), smem, stream, proj, ld, (float *)out, ldo,
-                         positions, cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps);
+                         positions, cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps, opts);
     return fg_launch(retention_seq_kernel<bf16>, dim3(n_seq, H), dim3(RET_THREADS), smem, stream, proj, ld, (bf16 *)out, ldo, positions,
-                     cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps);
+                     cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps, opts);
 }
 
 // 0 if the chunked form takes these sizes
 extern "C" int fg_retention_chunked_ok(int dk, int dv) {
-    if (dk <= 0 || dk % 2 || dv <= 0 || dv > RET_THREADS) return 0;
+    if (dk <= 0 || dv <= 0 || dv > RET_THREADS) return 0;
     size_t s1 = (size_t)RC * (dk + dv) * 4;
     size_t s3 = ((size_t)2 * RC * (dk + 1) + 2 * (size_t)RC * dv + RC * RC + RC) * 4;
     return s1 <= 200 * 1024 && s3 <= 200 * 1024;
@@ -465,8 +501,9 @@ extern "C" int fg_retention_chunked_ok(int dk, int dv) {
 extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int out_dtype, int ldo, const int *positions,
                                     const int *cu_rows, const int *slots, const float *cos_t, const float *sin_t,
                                     const float *decay, float *state, int *plan, float *U, int n_seq, int n_chunks, int H, int dk,
-                                    int dv, float k_scale, float eps, cudaStream_t stream) {
+                                    int dv, float k_scale, float eps, int opts, cudaStream_t stream) {
     if (n_seq <= 0 || n_chunks <= 0) return 0;
+    if (cos_t && dk % 2) return FG_ERR_BAD_SIZE;
     if (!fg_retention_chunked_ok(dk, dv) || H <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
     if (out_dtype != FG_F32 && out_dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
     const bool wide = out_dtype == FG_F32;
@@ -489,10 +526,10 @@ extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int ou
                          seq_chunk0);
     if (code) return code;
 #define RET_STATE_FAST(DK, DV) fg_launch(retention_chunk_state_fast<DK, DV>, dim3(n_chunks, H), dim3(RET_THREADS), 0, stream, proj, ld, positions, \
-        (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, U, H, k_scale)
+        (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, U, H, k_scale, opts)
     if (fast) code = dk == 64 ? (dv == 64 ? RET_STATE_FAST(64, 64) : RET_STATE_FAST(64, 128)) : (dv == 64 ? RET_STATE_FAST(128, 64) : RET_STATE_FAST(128, 128));
     else code = fg_launch(retention_chunk_state_kernel, dim3(n_chunks, H), dim3(RET_THREADS), s1, stream, proj, ld, positions, (const int *)chunk_row,
-                          (const int *)chunk_len, cos_t, sin_t, decay, U, H, dk, dv, k_scale);
+                          (const int *)chunk_len, cos_t, sin_t, decay, U, H, dk, dv, k_scale, opts);
 #undef RET_STATE_FAST
     if (code) return code;
     if ((dk * dv) % 4 == 0 && (((uintptr_t)U | (uintptr_t)state) & 15) == 0)
@@ -511,7 +548,7 @@ extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int ou
             if (e != cudaSuccess) return (int)e; \
         } \
         return fg_launch(retention_chunk_out_fast<DK, DV, TO>, dim3(n_chunks, H), dim3(RET_THREADS), sf, stream, proj, ld, (TO *)out, ldo, positions, \
-                         (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, k_scale, eps); } while (0)
+                         (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, k_scale, eps, opts); } while (0)
 #define RET_OUT_FAST_T(TO) do { \
         if (dk == 64 && dv == 64) RET_OUT_FAST(64, 64, TO); \
         if (dk == 64 && dv == 128) RET_OUT_FAST(64, 128, TO); \
@@ -524,7 +561,7 @@ extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int ou
     }
     if (wide)
         return fg_launch(retention_chunk_out_kernel<float>, dim3(n_chunks, H), dim3(RET_THREADS), s3, stream, proj, ld, (float *)out, ldo,
-                         positions, (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, dk, dv, k_scale, eps);
+                         positions, (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, dk, dv, k_scale, eps, opts);
     return fg_launch(retention_chunk_out_kernel<bf16>, dim3(n_chunks, H), dim3(RET_THREADS), s3, stream, proj, ld, (bf16 *)out, ldo,
-                     positions, (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, dk, dv, k_scale, eps);
+                     positions, (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, (const float *)U, H, dk, dv, k_scale, eps, opts);
 }

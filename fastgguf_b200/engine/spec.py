@@ -75,6 +75,8 @@ class RunSpec:
     cache_from: Optional[int] = None
     #: the model's ``reentry`` map (stream and embedding output -> stream) runs in front of this entry
     reenter: bool = False
+    #: with ``reenter``: the number of the pass that begins here
+    pass_number: Optional[int] = None
 
 
 @dataclass
@@ -100,7 +102,8 @@ class ModelSpec:
             "hidden_size": self.hidden_size, "vocab_size": self.vocab_size, "max_positions": self.max_positions,
             "embedding": self.embedding.to_json(), "final_norm": self.final_norm.to_json(), "head": self.head.to_json(),
             "layers": [l.to_json() for l in self.layers],
-            "schedule": [dict({"layer": r.layer, "cache_from": r.cache_from}, **({"reenter": True} if r.reenter else {})) for r in self.schedule],
+            "schedule": [dict({"layer": r.layer, "cache_from": r.cache_from}, **({"reenter": True} if r.reenter else {}),
+                          **({"pass": r.pass_number} if r.pass_number is not None else {})) for r in self.schedule],
             "stop_token_ids": list(self.stop_token_ids), "ignored_tensors": list(self.ignored_tensors),
         }
 
@@ -115,7 +118,7 @@ class ModelSpec:
             embedding=P(j["embedding"]), final_norm=P(j["final_norm"]), head=P(j["head"]),
             layers=[LayerSpec(l["block"], P(l["mixer"]), O(l.get("feed_forward")), O(l.get("mixer_norm")), O(l.get("feed_forward_norm")),
                               O(l.get("mixer_post_norm")), O(l.get("feed_forward_post_norm")), O(l.get("token_input"))) for l in j["layers"]],
-            schedule=[RunSpec(r["layer"], r.get("cache_from"), bool(r.get("reenter", False))) for r in j["schedule"]],
+            schedule=[RunSpec(r["layer"], r.get("cache_from"), bool(r.get("reenter", False)), r.get("pass")) for r in j["schedule"]],
             reentry=O(j.get("reentry")),
             stop_token_ids=tuple(j.get("stop_token_ids") or ()), ignored_tensors=tuple(j.get("ignored_tensors") or ()),
         )

@@ -21,10 +21,11 @@ from .config.salulorn import SalulornConfig
 from .config.pirozen import PirozenConfig
 from .config.saluzen import SaluzenConfig
 from .config.zifelorn import ZifelornConfig
+from .config.buguzen import BuguzenConfig
 from .engine.spec import ModelSpec
 
 _CLASSES = {"LlamaForCausalLM": LlamaConfig, "Zirivik": ZirivikConfig, "Salulorn": SalulornConfig, "Pirozen": PirozenConfig, "Saluzen": SaluzenConfig,
-            "Zifelorn": ZifelornConfig}
+            "Zifelorn": ZifelornConfig, "Buguzen": BuguzenConfig}
 _keep_alive = []
 
 
