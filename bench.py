@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--model 1b|3b|8b] [--dtype bfloat16|float32]
                     [--layers L] [--no-points] [--no-prefill] [--impl reference]
-    python bench.py --compare zirivik|salulorn|pirozen|saluzen [--sizes s,m] [--steps K] [--warmup W] [--batch 8]
+    python bench.py --compare zirivik|salulorn|pirozen|saluzen|zifelorn|buguzen [--sizes s,m] [--steps K] [--warmup W] [--batch 8]
 
 Default run: the layer sizes of Llama 3.2 1B with random weights, bfloat16, a batch of 8 sequences with random
 prompts of unequal lengths 128..1024, context 4096.  ``--model 3b``: prompts 64..2048, context 4096; ``--model 8b``:
@@ -18,7 +18,8 @@ made of.  Every step reads gigabytes of weights, far more than the 126 MB L2, so
 ``--compare zirivik`` (or ``salulorn``, ``pirozen``) leaves all of that alone and prints another line: prefill (one step of
 2,048 tokens) and decode (graph-replayed steps of a batch) of models of that design whose layers have the sizes of real models,
 beside Llama models of the same width, depth, heads and feed-forward size (Saluzen: beside Salulorn models, the engine's other
-mix of recurrent, windowed and latent layers; Pirozen: beside Zirivik models of windowed attention
+mix of recurrent, windowed and latent layers; Zifelorn and Buguzen: beside Zirivik models with the like layers in the
+same places; Pirozen: beside Zirivik models of windowed attention
 layers with experts of the same sizes, the closest the engine has), with the device time of every launcher of one prefill step
 and of decode steps run eagerly (``profile``), so that like kernels can be set side by side.
 """
@@ -237,9 +238,39 @@ def zifelorn_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_
             "logit_scale": 0.25, "layers": layers}
 
 
-DESIGNS = {"zifelorn": zifelorn_config, "zirivik": zirivik_config, "salulorn": salulorn_config, "pirozen": pirozen_config, "saluzen": saluzen_config}
+def buguzen_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff, blocks=2):
+    """Layers of a real model's sizes in the design's own mix: differential attention (two maps of 64 beside values of 128) + dense,
+    attention whose values are its keys (heads of 128, half of them rotated) + dense, linear attention + dense, linear attention
+    alone; `blocks` times; a token input of 256 numbers a layer; the whole stack is a loop that runs once."""
+    del heads, kv_heads, head_dim, expert_ff
+    H = width // 128
+    one = {"heads": H, "kv_heads": H // 4, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "mask": {"size": window},
+           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0}}}
+    two = {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+           "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    lin = {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 6 * h / max(1, H - 1)) for h in range(H)]}
+    dense = {"kind": "dense", "ff": ff}
+    layers = []
+    for _ in range(blocks):
+        layers += [{"type": "attention", "mixer": one, "mlp": dense}, {"type": "attention_2", "mixer": two, "mlp": dense},
+                   {"type": "lightning", "mixer": lin, "mlp": dense}, {"type": "lightning", "mixer": lin, "mlp": None}]
+    return {"architecture": "Buguzen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "token_side": {"dim": 256}, "layers": layers,
+            "loop": {"start": 0, "stop": len(layers), "times": 1}}
+
+
+def zirivik_dense_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff, blocks=2):
+    """The engine's closest model to Buguzen: Zirivik's layers in the same places - windowed attention + dense twice, retention + dense,
+    retention alone."""
+    z = zirivik_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff, 1)
+    ret, att, dense = z["layers"][0]["mixer"], z["layers"][2]["mixer"], z["layers"][0]["mlp"]
+    return dict(z, layers=[{"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": dense},
+                           {"type": "retention", "mixer": ret, "mlp": dense}, {"type": "retention", "mixer": ret, "mlp": None}] * blocks)
+
+
+DESIGNS = {"buguzen": buguzen_config, "zifelorn": zifelorn_config, "zirivik": zirivik_config, "salulorn": salulorn_config, "pirozen": pirozen_config, "saluzen": saluzen_config}
 #: the model a design stands beside, where that is not Llama
-COUNTERPARTS = {"pirozen": ("zirivik", zirivik_attention_config), "saluzen": ("salulorn", salulorn_config), "zifelorn": ("zirivik", zirivik_config)}
+COUNTERPARTS = {"pirozen": ("zirivik", zirivik_attention_config), "saluzen": ("salulorn", salulorn_config), "zifelorn": ("zirivik", zirivik_config),
+                "buguzen": ("zirivik", zirivik_dense_config)}
 
 #: name -> (width, heads, kv_heads, head_dim, ff, vocab, window, expert_ff)
 COMPARE_SIZES = {"s": (2048, 32, 8, 64, 8192, 32768, 1024, 2048), "m": (4096, 32, 8, 128, 14336, 32768, 2048, 4096)}
@@ -338,6 +369,11 @@ def compare_designs(args):
             row["config"].update({"latent": "rank 512 + 64 rotated, queries through %d, every second layer on the layer before's latents" % (width * 3 // 4),
                                   "recurrent": "%d channels in parts of 256, 4 taps" % width, "experts": "8 of ff %d, 2 a row" % eff,
                                   "beside": "Zirivik: retention, retention, windowed attention, attention on the layer before's keys; dense and experts alike"})
+        elif design == "buguzen":
+            row["config"].update({"differential": "%d heads of two maps of 64, values of 128, %d key/value heads" % (width // 128, width // 512),
+                                  "keys_as_values": "%d heads of 128, %d key heads, 64 rotated" % (width // 128, width // 512),
+                                  "linear": "%d heads of 128 x 128" % (width // 128), "token_input": "256 numbers a layer", "loop": "all layers, once",
+                                  "beside": "Zirivik: windowed attention + dense twice, retention + dense, retention alone"})
         else:
             row["config"].update({"gla": "%d heads of 64 x 128" % (width // 128), "latent": "rank 512 + 64 rotated, queries through %d" % (width * 3 // 4),
                                   "convolution": "4 taps", "loop": "all layers, once"})
