@@ -102,6 +102,17 @@ int fg_retention_chunked(const float *proj, int ld, void *out, int out_dtype, in
                          const int *cu_rows, const int *slots, const float *cos_t, const float *sin_t,
                          const float *decay, float *state, int *plan, float *U, int n_seq, int n_chunks, int H, int dk,
                          int dv, float k_scale, float eps, int opts, cudaStream_t stream);
+/* the same recurrence on bfloat16 activations, silu(q), silu(k), silu(v) of bfloat16 projections (decay_attention.cu): head sizes 64 and
+   128, raw sums out [M, H * dv] float32; and the norm over a whole row with its gate that follows */
+int fg_retention_plan(const int *cu_rows, int n_seq, int n_chunks, int chunk, int *plan, cudaStream_t stream);
+int fg_decay_attention_ok(int dk, int dv);
+int fg_decay_attention_chunk_tokens(void);
+int fg_decay_attention_chunked(void *proj, int ld, float *out, int ldo, const int *cu_rows, const int *slots, const float *decay, float *state,
+                               int *plan, float *U, void *P, int n_seq, int n_chunks, int H, int dk, int dv, cudaStream_t stream);
+int fg_decay_attention_step(const void *proj, int ld, float *out, int ldo, const int *cu_rows, const int *slots, const float *decay, float *state,
+                            int n_seq, int H, int dk, int dv, cudaStream_t stream);
+int fg_row_norm_gate(const float *o, int ldo, const void *g, int ldg, const float *w, void *out, int ldout, int M, int C, float eps, int sigmoid_gate,
+                     cudaStream_t stream);
 /* gated linear attention (gla.cu): proj rows q [H, dk] | k [H, dk] | v [H, dv] | g [H, dv] float32, z rows [H, dk] decay logits
    without their bias; state [slots, H, dk, dv] float32; out [M, H * dv] */
 int fg_gla(const float *proj, int ld, const float *z, int ldz, const float *z_bias, const float *norm_w, void *out, int out_dtype,

@@ -34,8 +34,6 @@ public:
         eps_ = (float)param_float(p, "eps", me);
         k_scale_ = (float)param_float(p, "k_scale", 1.0 / std::sqrt((double)dk_), me);
         if (E_ <= 0 || H_ <= 0 || dk_ <= 0 || dv_ <= 0) fail(FG_E_CONFIG, "retention: sizes must be positive");
-        if (dv_ > 256) fail(FG_E_CONFIG, format("retention: v_head_dim %d exceeds 256, the largest the kernels take", dv_));
-        if ((size_t)dk_ * dv_ > 40 * 1024) fail(FG_E_CONFIG, "retention: a head's state exceeds what the kernels hold in shared memory");
         if (!(eps_ > 0.f)) fail(FG_E_CONFIG, "retention: eps must be positive");
         const Json &d = p.get("decay");
         if (!d.is_array() || (int)d.size() != H_) fail(FG_E_CONFIG, format("retention: 'decay' must list one number for each of the %d heads", H_));
@@ -55,6 +53,8 @@ public:
         silu_ = option("qkv_activation", "none", "silu");
         whole_norm_ = option("norm", "head", "whole");
         sigmoid_gate_ = option("gate_activation", "silu", "sigmoid");
+        if (!whole_norm_ && dv_ > 256) fail(FG_E_CONFIG, format("retention: v_head_dim %d exceeds 256, the largest the kernels take", dv_));
+        if (!whole_norm_ && (size_t)dk_ * dv_ > 40 * 1024) fail(FG_E_CONFIG, "retention: a head's state exceeds what the kernels hold in shared memory");
         if (sigmoid_gate_ && !whole_norm_) fail(FG_E_CONFIG, "retention: a sigmoid gate needs norm 'whole'");
         const Json &pos = p.get("position");
         if (!pos.is_null()) {
@@ -103,6 +103,11 @@ public:
         if (!io.state || io.state_bytes < state_bytes()) fail(FG_E_INTERNAL, "retention: the schedule entry has no state rows");
         const float *cos_t = position_ ? position_->cos_table() : nullptr;
         const float *sin_t = position_ ? position_->sin_table() : nullptr;
+        const int *host_cu = b.host_cu_rows.empty() ? nullptr : b.host_cu_rows.data();
+        // activations of the engine's dtype and sums taken as they are: the tensor-core forms
+        if (rt.dtype == FG_BF16 && !rt.plain_kernels && silu_ && whole_norm_ && !position_ && k_scale_ == 1.f && all_positive_ &&
+            H_ * dv_ % 8 == 0 && H_ * dv_ <= 8192 && FG_KERNEL("mix", fg_decay_attention_ok)(dk_, dv_))
+            return forward_on_activations(rt, xn, deferred, b, io, residual, emit_norm, host_cu);
         // what enters the recurrence stays float32: the contraction accumulates in float32 and writes it as it is
         Tensor proj = proj_.forward(rt, xn, deferred, Tensor(), FG_F32, false, nullptr, nullptr);
         const int M = (int)proj.rows;
@@ -110,7 +115,6 @@ public:
         // (a norm over all heads: the recurrence's sums stay float32 until that norm is done)
         Tensor o = whole_norm_ ? rt.arena->matrix(M, (int64_t)H_ * dv_, FG_F32) : y;
         const int opts = (silu_ ? 1 : 0) | (whole_norm_ ? 2 : 0);
-        const int *host_cu = b.host_cu_rows.empty() ? nullptr : b.host_cu_rows.data();
         const int RC = FG_KERNEL("mix", fg_retention_chunk_tokens)();
         bool chunked = host_cu && !b.single_token && all_positive_ && b.max_new >= chunk_threshold_ &&
                        FG_KERNEL("mix", fg_retention_chunked_ok)(dk_, dv_);
@@ -136,6 +140,30 @@ public:
     }
 
 private:
+    DeferredNorm forward_on_activations(Runtime &rt, const Tensor &xn, const DeferredNorm *deferred, const Batch &b, const LayerIO &io, Tensor &residual,
+                                        Norm *emit_norm, const int *host_cu) {
+        Tensor proj = proj_.forward(rt, xn, deferred, Tensor(), FG_BF16, false, nullptr, nullptr);
+        const int M = (int)proj.rows, V = H_ * dv_, DC = FG_KERNEL("mix", fg_decay_attention_chunk_tokens)();
+        Tensor o = rt.arena->matrix(M, V, FG_F32), y = rt.arena->matrix(M, V, FG_BF16);
+        if (host_cu && !b.single_token && b.max_new >= DC / 2) {
+            int n_chunks = 0;
+            for (int s = 0; s < b.n_seq; s++) n_chunks += (host_cu[s + 1] - host_cu[s] + DC - 1) / DC;
+            int *plan = (int *)rt.arena->alloc(((size_t)2 * n_chunks + b.n_seq + 1) * sizeof(int));
+            float *U = (float *)rt.arena->alloc((size_t)n_chunks * H_ * dk_ * dv_ * sizeof(float));
+            void *P = rt.arena->alloc((size_t)n_chunks * H_ * dk_ * dv_ * 3 * 2);      // the states in front of the chunks, three bfloat16 pieces each
+            FG_LAUNCH("mix", fg_decay_attention_chunked, proj.data, (int)proj.ld, o.ptr<float>(), (int)o.ld, b.cu_rows, b.slots, decay_dev_.t.ptr<float>(),
+                      (float *)io.state, plan, U, P, b.n_seq, n_chunks, H_, dk_, dv_, rt.stream);
+        } else {
+            FG_LAUNCH("mix", fg_decay_attention_step, proj.data, (int)proj.ld, o.ptr<float>(), (int)o.ld, b.cu_rows, b.slots, decay_dev_.t.ptr<float>(),
+                      (float *)io.state, b.n_seq, H_, dk_, dv_, rt.stream);
+        }
+        const uint16_t *g = (const uint16_t *)proj.data + (int64_t)2 * H_ * dk_ + V;
+        FG_LAUNCH("mix", fg_row_norm_gate, o.ptr<float>(), (int)o.ld, g, (int)proj.ld, norm_w_.t.ptr<float>(), y.data, (int)y.ld, M, V, eps_, sigmoid_gate_ ? 1 : 0,
+                  rt.stream);
+        DeferredNorm started;
+        o_.forward(rt, y, nullptr, residual, FG_F32, !rt.overwrite, emit_norm, &started);
+        return started;
+    }
     int E_ = 0, H_ = 0, dk_ = 0, dv_ = 0, chunk_threshold_ = 16;
     float eps_ = 0.f, k_scale_ = 1.f;
     bool all_positive_ = true, silu_ = false, whole_norm_ = false, sigmoid_gate_ = false;

@@ -93,12 +93,12 @@ __device__ __forceinline__ void copy_chunk_into(const float *__restrict__ proj, 
     }
 }
 
-template <typename TO>
+template <typename TO, bool SLAB>
 __global__ void __launch_bounds__(RET_THREADS)
 retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ out, int ldo, const int *__restrict__ positions,
                      const int *__restrict__ cu_rows, const int *__restrict__ slots, const float *__restrict__ cos_t,
                      const float *__restrict__ sin_t, const float *__restrict__ decay, float *__restrict__ state, int H, int dk,
-                     int dv, float k_scale, float eps, int opts) {
+                     int dv_all, float k_scale, float eps, int opts, int slab) {
     extern __shared__ float sm[];
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -106,10 +106,12 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
     const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int row0 = cu_rows[seq], row1 = cu_rows[seq + 1];
     if (row1 <= row0) return;
+    // (raw sums: columns do not meet, so a block may own a slab of them; else the slab is the head)
+    const int col0 = SLAB ? blockIdx.z * slab : 0, dv = SLAB ? min(slab, dv_all - col0) : dv_all;
     const int G = RET_THREADS / dv, n_active = G * dv;      // threads (g, j): column j of S, rows g, g + G, ...
     float *S = sm, *qs = S + dk * dv, *ks = qs + dk, *vs = ks + dk, *part = vs + dv;
-    float *Sg = state + ((size_t)slots[seq] * H + h) * dk * dv;
-    for (int e = tid; e < dk * dv; e += RET_THREADS) S[e] = Sg[e];
+    float *Sg = state + ((size_t)slots[seq] * H + h) * dk * dv_all + col0;
+    for (int e = tid; e < dk * dv; e += RET_THREADS) S[e] = Sg[SLAB ? (e / dv) * dv_all + e % dv : e];
     const float dec = decay[h];
     const int half = dk >> 1;
     for (int r = row0; r < row1; r++) {
@@ -118,7 +120,7 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
         const float *cs = cos_t ? cos_t + (size_t)pos * half : nullptr, *sn = cos_t ? sin_t + (size_t)pos * half : nullptr;
         rotate_into(row + (size_t)h * dk, qs, dk, cs, sn, 1.0f, opts, tid, RET_THREADS);
         rotate_into(row + (size_t)(H + h) * dk, ks, dk, cs, sn, k_scale, opts, tid, RET_THREADS);
-        for (int j = tid; j < dv; j += RET_THREADS) vs[j] = opt_silu(row[(size_t)2 * H * dk + (size_t)h * dv + j], opts);
+        for (int j = tid; j < dv; j += RET_THREADS) vs[j] = opt_silu(row[(size_t)2 * H * dk + (size_t)h * dv_all + col0 + j], opts);
         __syncthreads();
         if (tid < n_active) {
             const int j = tid % dv, g = tid / dv;
@@ -136,7 +138,7 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
         if (tid < dv)
             for (int g = 0; g < G; g++) o += part[g * dv + tid];
         if (opts & RET_RAW) {
-            if (tid < dv) out[(size_t)r * ldo + (size_t)h * dv + tid] = from_f32<TO>(o);
+            if (tid < dv) out[(size_t)r * ldo + (size_t)h * dv_all + col0 + tid] = from_f32<TO>(o);
             __syncthreads();                   // part is rewritten by the next token
             continue;
         }
@@ -147,27 +149,27 @@ retention_seq_kernel(const float *__restrict__ proj, int ld, TO *__restrict__ ou
         }
     }
     __syncthreads();
-    for (int e = tid; e < dk * dv; e += RET_THREADS) Sg[e] = S[e];
+    for (int e = tid; e < dk * dv; e += RET_THREADS) Sg[SLAB ? (e / dv) * dv_all + e % dv : e] = S[e];
 }
 
 // ------------------------------------------------------------------ chunked form
 // Chunk c of the step covers tokens [chunk_row[c], chunk_row[c] + chunk_len[c]); the chunks of a sequence are consecutive
 // and in order, sequence s owning chunks [seq_chunk0[s], seq_chunk0[s + 1]).  The plan is made on the device from the
 // step's row offsets; the host only knows how many chunks there are.
-__global__ void retention_chunk_plan_kernel(const int *__restrict__ cu_rows, int n_seq, int *__restrict__ chunk_row,
+__global__ void retention_chunk_plan_kernel(const int *__restrict__ cu_rows, int n_seq, int chunk, int *__restrict__ chunk_row,
                                             int *__restrict__ chunk_len, int *__restrict__ seq_chunk0) {
     pdl_launch_dependents();
     pdl_wait();
     if (threadIdx.x == 0) {
         int at = 0;
-        for (int s = 0; s < n_seq; s++) { seq_chunk0[s] = at; at += (cu_rows[s + 1] - cu_rows[s] + RC - 1) / RC; }
+        for (int s = 0; s < n_seq; s++) { seq_chunk0[s] = at; at += (cu_rows[s + 1] - cu_rows[s] + chunk - 1) / chunk; }
         seq_chunk0[n_seq] = at;
     }
     __syncthreads();
     for (int s = threadIdx.x; s < n_seq; s += blockDim.x) {
         const int r0 = cu_rows[s], r1 = cu_rows[s + 1];
         int c = seq_chunk0[s];
-        for (int r = r0; r < r1; r += RC, c++) { chunk_row[c] = r; chunk_len[c] = min(RC, r1 - r); }
+        for (int r = r0; r < r1; r += chunk, c++) { chunk_row[c] = r; chunk_len[c] = min(chunk, r1 - r); }
     }
 }
 
@@ -462,7 +464,7 @@ retention_chunk_out_fast(const float *__restrict__ proj, int ld, TO *__restrict_
 }
 
 // ------------------------------------------------------------------ launchers
-static FgPerDevice g_seq_setup[2], g_state_setup, g_out_setup[2];
+static FgPerDevice g_state_setup, g_out_setup[2];
 
 extern "C" int fg_retention_chunk_tokens(void) { return RC; }
 
@@ -470,22 +472,48 @@ extern "C" int fg_retention(const float *proj, int ld, void *out, int out_dtype,
                             const int *slots, const float *cos_t, const float *sin_t, const float *decay, float *state, int n_seq,
                             int H, int dk, int dv, float k_scale, float eps, int opts, cudaStream_t stream) {
     if (n_seq <= 0) return 0;
-    if (dk <= 0 || (cos_t && dk % 2) || dv <= 0 || dv > RET_THREADS || H <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
-    const int G = RET_THREADS / dv;
-    size_t smem = ((size_t)dk * dv + 2 * dk + dv + (size_t)G * dv) * sizeof(float);
+    if (dk <= 0 || (cos_t && dk % 2) || dv <= 0 || H <= 0 || H > 65535) return FG_ERR_BAD_SIZE;
+    // raw sums of a head whose state is large: a block per slab of columns
+    int slab = dv;
+    if (opts & RET_RAW)
+        while (slab > 1 && (slab > RET_THREADS || (size_t)dk * slab > 40 * 1024)) slab = (slab + 1) / 2;
+    if (slab > RET_THREADS) return FG_ERR_BAD_SIZE;
+    const dim3 grid(n_seq, H, (dv + slab - 1) / slab);
+    size_t smem = ((size_t)dk * slab + 2 * dk + slab + (size_t)RET_THREADS) * sizeof(float);
+
     if (smem > 200 * 1024) return FG_ERR_BAD_SIZE;
     if (out_dtype != FG_F32 && out_dtype != FG_BF16) return FG_ERR_BAD_DTYPE;
-    const bool wide = out_dtype == FG_F32;
-    if (fg_needs_setup(g_seq_setup[wide ? 0 : 1])) {
-        cudaError_t e = wide ? cudaFuncSetAttribute(retention_seq_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)
-                             : cudaFuncSetAttribute(retention_seq_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        if (e != cudaSuccess) return (int)e;
+#define RET_SEQ(TO, SLAB) do { \
+        static FgPerDevice setup; \
+        if (fg_needs_setup(setup)) { \
+            cudaError_t e = cudaFuncSetAttribute(retention_seq_kernel<TO, SLAB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            if (e != cudaSuccess) return (int)e; \
+        } \
+        return fg_launch(retention_seq_kernel<TO, SLAB>, grid, dim3(RET_THREADS), smem, stream, proj, ld, (TO *)out, ldo, positions, cu_rows, slots, cos_t, \
+                         sin_t, decay, state, H, dk, dv, k_scale, eps, opts, slab); } while (0)
+    if (slab < dv) {
+        if (out_dtype == FG_F32) RET_SEQ(float, true);
+        RET_SEQ(bf16, true);
     }
-    if (wide)
-        return fg_launch(retention_seq_kernel<float>, dim3(n_seq, H), dim3(RET_THREADS), smem, stream, proj, ld, (float *)out, ldo,
-                         positions, cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps, opts);
-    return fg_launch(retention_seq_kernel<bf16>, dim3(n_seq, H), dim3(RET_THREADS), smem, stream, proj, ld, (bf16 *)out, ldo, positions,
-                     cu_rows, slots, cos_t, sin_t, decay, state, H, dk, dv, k_scale, eps, opts);
+    if (out_dtype == FG_F32) RET_SEQ(float, false);
+    RET_SEQ(bf16, false);
+#undef RET_SEQ
+}
+
+// The chunk table (decay_attention.cu asks for it too).  plan: ints
+// [chunk_row | chunk_len | seq_chunk0], 2 * n_chunks + n_seq + 1 of them, for chunks of `chunk` tokens.
+extern "C" int fg_retention_plan(const int *cu_rows, int n_seq, int n_chunks, int chunk, int *plan, cudaStream_t stream) {
+    return fg_launch(retention_chunk_plan_kernel, dim3(1), dim3(n_seq >= 256 ? 256 : 32), 0, stream, cu_rows, n_seq, chunk, plan, plan + n_chunks,
+                     plan + 2 * n_chunks);
+}
+static int retention_scan(const int *plan, int n_chunks, const int *slots, const float *decay, float *U, float *state, int n_seq, int H, int dk, int dv,
+                          cudaStream_t stream) {
+    const int *chunk_len = plan + n_chunks, *seq_chunk0 = plan + 2 * n_chunks;
+    if ((dk * dv) % 4 == 0 && (((uintptr_t)U | (uintptr_t)state) & 15) == 0)
+        return fg_launch(retention_chunk_scan_kernel<float4>, dim3(n_seq, H, (dk * dv / 4 + RET_THREADS - 1) / RET_THREADS), dim3(RET_THREADS), 0, stream,
+                         seq_chunk0, chunk_len, slots, decay, U, state, H, dk, dv);
+    return fg_launch(retention_chunk_scan_kernel<float>, dim3(n_seq, H, (dk * dv + RET_THREADS - 1) / RET_THREADS), dim3(RET_THREADS), 0, stream,
+                     seq_chunk0, chunk_len, slots, decay, U, state, H, dk, dv);
 }
 
 // 0 if the chunked form takes these sizes
@@ -518,12 +546,11 @@ extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int ou
                              : cudaFuncSetAttribute(retention_chunk_out_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return (int)e;
     }
-    int *chunk_row = plan, *chunk_len = plan + n_chunks, *seq_chunk0 = plan + 2 * n_chunks;
+    int *chunk_row = plan, *chunk_len = plan + n_chunks;
     // head sizes 64 / 128 with 16-byte aligned rows: the kernels with register tiles
     const bool fast = (dk == 64 || dk == 128) && (dv == 64 || dv == 128) && ld % 4 == 0 && (((uintptr_t)proj | (uintptr_t)U) & 15) == 0 &&
                       ldo % 4 == 0 && ((uintptr_t)out & 15) == 0;
-    int code = fg_launch(retention_chunk_plan_kernel, dim3(1), dim3(n_seq >= 256 ? 256 : 32), 0, stream, cu_rows, n_seq, chunk_row, chunk_len,
-                         seq_chunk0);
+    int code = fg_retention_plan(cu_rows, n_seq, n_chunks, RC, plan, stream);
     if (code) return code;
 #define RET_STATE_FAST(DK, DV) fg_launch(retention_chunk_state_fast<DK, DV>, dim3(n_chunks, H), dim3(RET_THREADS), 0, stream, proj, ld, positions, \
         (const int *)chunk_row, (const int *)chunk_len, cos_t, sin_t, decay, U, H, k_scale, opts)
@@ -532,12 +559,7 @@ extern "C" int fg_retention_chunked(const float *proj, int ld, void *out, int ou
                           (const int *)chunk_len, cos_t, sin_t, decay, U, H, dk, dv, k_scale, opts);
 #undef RET_STATE_FAST
     if (code) return code;
-    if ((dk * dv) % 4 == 0 && (((uintptr_t)U | (uintptr_t)state) & 15) == 0)
-        code = fg_launch(retention_chunk_scan_kernel<float4>, dim3(n_seq, H, (dk * dv / 4 + RET_THREADS - 1) / RET_THREADS), dim3(RET_THREADS), 0,
-                         stream, (const int *)seq_chunk0, (const int *)chunk_len, slots, decay, U, state, H, dk, dv);
-    else
-        code = fg_launch(retention_chunk_scan_kernel<float>, dim3(n_seq, H, (dk * dv + RET_THREADS - 1) / RET_THREADS), dim3(RET_THREADS), 0, stream,
-                         (const int *)seq_chunk0, (const int *)chunk_len, slots, decay, U, state, H, dk, dv);
+    code = retention_scan(plan, n_chunks, slots, decay, U, state, n_seq, H, dk, dv, stream);
     if (code) return code;
     if (fast) {
         const size_t sf = ((size_t)2 * RC * (dk + 4) + (size_t)RC * dv + RC * RC) * sizeof(float);
