@@ -15,8 +15,18 @@
 
 #define PREP_THREADS 256
 
+// four neighbours of a row: 16 bytes of float32, or 8 of bfloat16
+template <typename T> __device__ __forceinline__ void put4(T *dst, const float *p);
+template <> __device__ __forceinline__ void put4<float>(float *dst, const float *p) { *(float4 *)dst = *(const float4 *)p; }
+template <> __device__ __forceinline__ void put4<bf16>(bf16 *dst, const float *p) {
+    const float4 v = *(const float4 *)p;
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *(uint2 *)dst = make_uint2(*(uint32_t *)&lo, *(uint32_t *)&hi);
+}
+
 // cos/sin: [positions, tbl_half] float32, column i = pair i.
-template <typename T>
+// VEC: no convolution, and rows, heads and pools allow accesses of four numbers.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(1024)
 qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restrict__ bias, const float *__restrict__ conv_w, int taps,
                    const float *__restrict__ conv_state, const float *__restrict__ qn_w, const float *__restrict__ kn_w, float eps,
@@ -25,7 +35,7 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
                    const int *__restrict__ slots, const int *__restrict__ block_table, int table_width, T *__restrict__ q_out, int ldq,
                    T *__restrict__ k_pool, T *__restrict__ v_pool, int H, int KV, int VH, int hd, int hdv, int page_size, int norm_per_head,
                    int rot_halves, int v_from_k) {
-    extern __shared__ float row[];
+    extern __shared__ __align__(16) float row[];
     __shared__ float scratch[32];
     pdl_launch_dependents_small_step(gridDim.x);
     pdl_wait();
@@ -34,7 +44,13 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
     const int seq = row_seq[m], pos = positions[m];
     const int i_step = m - cu_rows[seq];                 // the token's index among the step's tokens of its sequence
     const float *mine = proj + (size_t)m * ld;
-    if (conv_w) {
+    if (VEC) {
+        for (int c = tid * 4; c < C; c += nthr * 4) {
+            float4 v = *(const float4 *)(mine + c);
+            if (bias) { const float4 b = *(const float4 *)(bias + c); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+            *(float4 *)(row + c) = v;
+        }
+    } else if (conv_w) {
         const float *st = conv_state + (size_t)slots[seq] * (taps - 1) * C;
         for (int c = tid; c < C; c += nthr) {
             const float b = bias ? bias[c] : 0.f;
@@ -55,9 +71,16 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
     if (v_from_k && v_pool) {
         // the values are the keys as projected (bias included), before norm and rotation
         const int page = block_table[(size_t)seq * table_width + pos / page_size], off = pos % page_size;
-        for (int c = tid; c < Ck; c += nthr) {
-            const int vh = c / hdv, d = c - vh * hdv;
-            v_pool[(((size_t)page * VH + vh) * page_size + off) * hdv + d] = from_f32<T>(row[Cq + c]);
+        if (VEC) {
+            for (int c = tid * 4; c < Ck; c += nthr * 4) {
+                const int vh = c / hdv, d = c - vh * hdv;
+                put4<T>(v_pool + (((size_t)page * VH + vh) * page_size + off) * hdv + d, row + Cq + c);
+            }
+        } else {
+            for (int c = tid; c < Ck; c += nthr) {
+                const int vh = c / hdv, d = c - vh * hdv;
+                v_pool[(((size_t)page * VH + vh) * page_size + off) * hdv + d] = from_f32<T>(row[Cq + c]);
+            }
         }
         __syncthreads();
     }
@@ -99,6 +122,20 @@ qkv_prepare_kernel(const float *__restrict__ proj, int ld, const float *__restri
             p[other] = b * c + a * s;
         }
         __syncthreads();
+    }
+    if (VEC) {
+        for (int c = tid * 4; c < Cq; c += nthr * 4) put4<T>(q_out + (size_t)m * ldq + c, row + c);
+        if (!k_pool) return;
+        const int page = block_table[(size_t)seq * table_width + pos / page_size], off = pos % page_size;
+        for (int c = tid * 4; c < Ck; c += nthr * 4) {
+            const int kvh = c / hd, d = c - kvh * hd;
+            put4<T>(k_pool + (((size_t)page * KV + kvh) * page_size + off) * hd + d, row + Cq + c);
+        }
+        for (int c = tid * 4; c < (v_from_k ? 0 : VH * hdv); c += nthr * 4) {
+            const int vh = c / hdv, d = c - vh * hdv;
+            put4<T>(v_pool + (((size_t)page * VH + vh) * page_size + off) * hdv + d, row + Cq + Ck + c);
+        }
+        return;
     }
     for (int c = tid; c < Cq; c += nthr) q_out[(size_t)m * ldq + c] = from_f32<T>(row[c]);
     if (k_pool) {
@@ -396,22 +433,28 @@ extern "C" int fg_qkv_prepare_ext(const float *proj, int ld, const float *bias, 
     const int C_all = H * hd + KV * hd + (v_from_k ? 0 : VH * hdv);
     const size_t smem = (size_t)C_all * sizeof(float);
     if (smem > 200 * 1024) return FG_ERR_BAD_SIZE;
-    static FgPerDevice setup[2];
-    if (smem > 48 * 1024 && fg_needs_setup(setup[dtype == FG_F32 ? 0 : 1])) {
-        cudaError_t e = dtype == FG_F32 ? cudaFuncSetAttribute(qkv_prepare_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)
-                                        : cudaFuncSetAttribute(qkv_prepare_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        if (e != cudaSuccess) return (int)e;
-    }
     // few rows (a decode step) leave most of the GPU idle: a row's channels are then spread over more threads
     const int threads = (M < 64 && C_all >= 2048) ? 1024 : PREP_THREADS;
-    if (dtype == FG_F32)
-        return fg_launch(qkv_prepare_kernel<float>, dim3(M), dim3(threads), smem, stream, proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w,
-                         eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq, cu_rows, slots, block_table, table_width, (float *)q_out,
-                         ldq, (float *)k_pool, (float *)v_pool, H, KV, VH, hd, hdv, page_size, norm_per_head, rot_halves, v_from_k);
-    if (dtype == FG_BF16)
-        return fg_launch(qkv_prepare_kernel<bf16>, dim3(M), dim3(threads), smem, stream, proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w,
-                         eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq, cu_rows, slots, block_table, table_width, (bf16 *)q_out, ldq,
-                         (bf16 *)k_pool, (bf16 *)v_pool, H, KV, VH, hd, hdv, page_size, norm_per_head, rot_halves, v_from_k);
+    const bool vec = !conv_w && hd % 4 == 0 && hdv % 4 == 0 && ld % 4 == 0 && ldq % 4 == 0 &&
+                     ((((uintptr_t)proj) | ((uintptr_t)bias) | ((uintptr_t)q_out) | ((uintptr_t)k_pool) | ((uintptr_t)v_pool)) & 15) == 0;
+#define PREP_RUN(T, VEC) do { \
+        static FgPerDevice setup; \
+        if (smem > 48 * 1024 && fg_needs_setup(setup)) { \
+            cudaError_t e = cudaFuncSetAttribute(qkv_prepare_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            if (e != cudaSuccess) return (int)e; \
+        } \
+        return fg_launch(qkv_prepare_kernel<T, VEC>, dim3(M), dim3(threads), smem, stream, proj, ld, bias, conv_w, taps, conv_state, qn_w, kn_w, \
+                         eps, cos_t, sin_t, tbl_half, rot_dims, positions, row_seq, cu_rows, slots, block_table, table_width, (T *)q_out, \
+                         ldq, (T *)k_pool, (T *)v_pool, H, KV, VH, hd, hdv, page_size, norm_per_head, rot_halves, v_from_k); } while (0)
+    if (dtype == FG_F32) {
+        if (vec) PREP_RUN(float, true);
+        PREP_RUN(float, false);
+    }
+    if (dtype == FG_BF16) {
+        if (vec) PREP_RUN(bf16, true);
+        PREP_RUN(bf16, false);
+    }
+#undef PREP_RUN
     return FG_ERR_BAD_DTYPE;
 }
 

@@ -22,7 +22,8 @@
 #define DC 64                       // tokens a chunk
 #define DA_THREADS 256
 
-__device__ __forceinline__ float da_silu(float z) { return z / (1.0f + expf(-z)); }
+// (fast exponential and division, 2 ulp each: the result is rounded to bfloat16 right after)
+__device__ __forceinline__ float da_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 // silu of a projection's bfloat16, rounded to bfloat16
 __device__ __forceinline__ float da_act(bf16 z) { return __bfloat162float(__float2bfloat16_rn(da_silu(__bfloat162float(z)))); }
 

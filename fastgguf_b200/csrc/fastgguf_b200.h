@@ -259,6 +259,9 @@ int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, void *out, int
 long long fg_gemm_tc_workspace_bytes(int M, int N, int K, int epi);
 int fg_gemm_tc_max_ss_tiles(int N);
 /* grouped contraction over runs of rows, each with its own matrix of a stack (see gemm_tc.cu); tiles: device int4 table */
+/* out = bf16(gelu_tanh(X W^T) * table[tokens[m], col + n]) */
+int fg_gemm_tc_gelu_gather(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int M, int N, int K, const void *table, int ldt, int col,
+                           const int *tokens, void *workspace, long long workspace_bytes, cudaStream_t stream);
 int fg_gemm_tc_grouped_bn(int N);
 int fg_gemm_tc_grouped(const void *X, int ldx, int rows, const void *W, int ldw, int stack_rows, float *out, int ldc, int N, int K,
                        const void *tiles, int n_tiles, cudaStream_t stream);

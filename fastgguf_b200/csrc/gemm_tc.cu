@@ -48,7 +48,8 @@
 #define WAIT_SHORT_CYCLES 1000000ll
 
 enum { EPI_BF16 = 0, EPI_F32 = 1, EPI_ADD_F32 = 2, EPI_SILU_MUL = 3, EPI_RELU2_BF16 = 4 /* launcher only: EPI_BF16 + act */,
-       EPI_GELU_MUL = 5 /* launcher only: EPI_SILU_MUL + act 1 */, EPI_RELU_MUL = 6 /* launcher only: EPI_SILU_MUL + act 2 */ };
+       EPI_GELU_MUL = 5 /* launcher only: EPI_SILU_MUL + act 1 */, EPI_RELU_MUL = 6 /* launcher only: EPI_SILU_MUL + act 2 */,
+       EPI_GELU_GATHER = 7 /* launcher only: EPI_BF16 + act 2 */ };
 
 __device__ int g_gemm_error = 0;      // 0, or (code << 8 | role) of the first wait that ran out
 // How long a wait may last, in SM cycles (about a second).  A variable, so that a test can make a wait run out within a
@@ -210,13 +211,24 @@ struct GemmArgs {
     int epi, stages;      // decode kernel: epilogue and ring depth are run-time values
     int test_skip_copy;   // tests only: the decode kernel's producer omits the activation copy of its first stage
     int splits;           // prefill kernel: > 1 = partial products of `kb_per_split` K-blocks each into out[split][M][ldc]
-    int act;              // bf16 epilogue: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward); gated epilogue: 1 = gelu, 2 = relu, not SiLU
+    int act;              // bf16 epilogue: 1 = store max(x, 0)^2 (the squared ReLU of a plain feed-forward), 2 = gelu(x) times a table's entry; gated epilogue: 1 = gelu, 2 = relu, not SiLU
     // prefill kernel, grouped contraction (rows in runs, each run with a weight matrix of its own out of a stack): tile t
     // is tiles[t] = {first row, end of its run, first row of the run's matrix in W, tile index along N}; null: one matrix
     const int4 *tiles;
+    // bf16 epilogue with act 2: store gelu(x) * gate_table[gate_tokens[m], gate_col + n] (a token's own numbers, gated by the contraction)
+    const bf16 *gate_table;
+    const int *gate_tokens;
+    int gate_ld, gate_col;
 };
 
 __device__ __forceinline__ float relu2(float x) { return x > 0.f ? x * x : 0.f; }
+// (out of line: the epilogues of every other contraction keep their size)
+__device__ __noinline__ float gelu_gather(const bf16 *row, int n, float x) {
+    return gated_mul(x, __bfloat162float(row[n]), 1);
+}
+__device__ __forceinline__ float bf16_act(const GemmArgs &a, int m, int n, float x) {
+    return a.act == 0 ? x : a.act == 1 ? relu2(x) : gelu_gather(a.gate_table + (size_t)a.gate_tokens[m] * a.gate_ld + a.gate_col, n, x);
+}
 
 __device__ __forceinline__ float inv_rms(const GemmArgs &a, int m) {
     float s = 0.f;
@@ -269,9 +281,19 @@ __device__ __forceinline__ void epilogue_token_major(const GemmArgs &a, uint32_t
             if (!m_ok || n0 >= a.N) continue;
 #pragma unroll
             for (int j = 0; j < 16; j++) v[j] *= iv;
-            if (EPI == EPI_BF16 && a.act) {
+            if (EPI == EPI_BF16 && a.act == 1) {
 #pragma unroll
                 for (int j = 0; j < 16; j++) v[j] = relu2(v[j]);
+            } else if (EPI == EPI_BF16 && a.act == 2) {
+                const bf16 *entry = a.gate_table + (size_t)a.gate_tokens[m] * a.gate_ld + a.gate_col + n0;
+                if (n0 + 16 <= a.N && ((uintptr_t)entry & 15) == 0) {
+                    const uint4 e[2] = {((const uint4 *)entry)[0], ((const uint4 *)entry)[1]};
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] = gated_mul(v[j], __bfloat162float(((const bf16 *)e)[j]), 1);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] = n0 + j < a.N ? gelu_gather(entry, j, v[j]) : 0.f;
+                }
             }
             const size_t idx = (out_row0 + (size_t)m) * a.ldc + n0;       // (out_row0: the split's block of a partial product)
             const bool full = a.vec_ok && n0 + 16 <= a.N;
@@ -753,7 +775,7 @@ gemm_tc_decode_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
                     const int n = p0 + lane + 32 * i;
                     if (n >= a.N) continue;
                     const size_t idx = (size_t)m * a.ldc + n;
-                    if (epi == EPI_BF16) ((bf16 *)a.out)[idx] = __float2bfloat16_rn(a.act ? relu2(v[i]) : v[i]);
+                    if (epi == EPI_BF16) ((bf16 *)a.out)[idx] = __float2bfloat16_rn(bf16_act(a, m, n, v[i]));
                     else {
                         ((float *)a.out)[idx] = v[i];
                         if (emit) a.xw_out[(size_t)m * a.N + n] = __float2bfloat16_rn(v[i] * nw_pre[i]);
@@ -967,7 +989,7 @@ gemm_splitk_finish_kernel(GemmArgs a, const float *__restrict__ ws, int S) {
         if (n >= a.N) continue;
         const size_t idx = (size_t)m * a.ldc + n;
         float x = v[i] * iv;
-        if (EPI == EPI_BF16) { ((bf16 *)a.out)[idx] = __float2bfloat16_rn(a.act ? relu2(x) : x); continue; }
+        if (EPI == EPI_BF16) { ((bf16 *)a.out)[idx] = __float2bfloat16_rn(bf16_act(a, m, n, x)); continue; }
         if (EPI == EPI_ADD_F32) x += res[i];
         ((float *)a.out)[idx] = x;
         if (EPI == EPI_ADD_F32 && a.norm_w) {
@@ -1338,6 +1360,16 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
                              float ss_eps, const float *norm_w, void *xw_out, float *ss_out, int *ss_tiles_out,
                              void *workspace, long long workspace_bytes, cudaStream_t stream);
 
+// what the epilogue of code 7 reads besides
+struct GateGather {
+    const bf16 *table;
+    const int *tokens;
+    int ld, col;
+};
+static int gemm_tc_run(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int epi, int M, int N, int K, int force_splits,
+                       const float *ss_in, int ss_tiles, int ss_size, float ss_eps, const float *norm_w, void *xw_out, float *ss_out,
+                       int *ss_tiles_out, void *workspace, long long workspace_bytes, const GateGather &gate, cudaStream_t stream);
+
 extern "C" int fg_gemm_tc(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int epi,
                           int M, int N, int K, int force_splits, const float *ss_in, int ss_tiles, int ss_size,
                           float ss_eps, const float *norm_w, void *xw_out, float *ss_out, int *ss_tiles_out,
@@ -1354,12 +1386,31 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
                              int M, int N, int K, int force_splits, const float *ss_in, int ss_tiles, int ss_size,
                              float ss_eps, const float *norm_w, void *xw_out, float *ss_out, int *ss_tiles_out,
                              void *workspace, long long workspace_bytes, cudaStream_t stream) {
+    if (epi == EPI_GELU_GATHER) return FG_ERR_BAD_DTYPE;
+    return gemm_tc_run(X, ldx, W, ldw, out, ldc, epi, M, N, K, force_splits, ss_in, ss_tiles, ss_size, ss_eps, norm_w, xw_out, ss_out, ss_tiles_out,
+                       workspace, workspace_bytes, GateGather{}, stream);
+}
+
+// out[m, n] = bf16(gelu_tanh((X W^T)[m, n]) * table[tokens[m], col + n]): a token's own numbers, gated by the contraction.  table bfloat16
+// with ldt numbers a row; workspace as for fg_gemm_tc_ws (fg_gemm_tc_workspace_bytes with epilogue 0).
+extern "C" int fg_gemm_tc_gelu_gather(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int M, int N, int K, const void *table, int ldt,
+                                      int col, const int *tokens, void *workspace, long long workspace_bytes, cudaStream_t stream) {
+    if (!table || !tokens || col < 0 || col + N > ldt) return FG_ERR_BAD_SIZE;
+    int tiles = 0;
+    return gemm_tc_run(X, ldx, W, ldw, out, ldc, EPI_GELU_GATHER, M, N, K, 0, nullptr, 0, 1, 0.f, nullptr, nullptr, nullptr, &tiles, workspace, workspace_bytes,
+                       GateGather{(const bf16 *)table, tokens, ldt, col}, stream);
+}
+
+static int gemm_tc_run(const void *X, int ldx, const void *W, int ldw, void *out, int ldc, int epi, int M, int N, int K, int force_splits,
+                       const float *ss_in, int ss_tiles, int ss_size, float ss_eps, const float *norm_w, void *xw_out, float *ss_out,
+                       int *ss_tiles_out, void *workspace, long long workspace_bytes, const GateGather &gate, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return FG_ERR_BAD_SIZE;
     // epilogue code 4: bfloat16 output of max(x, 0)^2 - the bf16 epilogue with its activation flag set
+    // epilogue code 7: bfloat16 output of gelu(x) times an entry of a table
     // epilogue codes 5, 6: the gated epilogue with the tanh form of gelu, or max(., 0), on the gate
-    const int act = epi == EPI_RELU_MUL ? 2 : (epi == EPI_RELU2_BF16 || epi == EPI_GELU_MUL) ? 1 : 0;
-    if (act) epi = epi == EPI_RELU2_BF16 ? EPI_BF16 : EPI_SILU_MUL;
+    const int act = (epi == EPI_RELU_MUL || epi == EPI_GELU_GATHER) ? 2 : (epi == EPI_RELU2_BF16 || epi == EPI_GELU_MUL) ? 1 : 0;
+    if (act) epi = (epi == EPI_RELU2_BF16 || epi == EPI_GELU_GATHER) ? EPI_BF16 : EPI_SILU_MUL;
     if (epi == EPI_SILU_MUL && N % 128) return FG_ERR_BAD_SIZE;
     // Up to 128 rows the weights stream through the decode kernel, in blocks of 64 tokens whose CTAs run side by side
     // and share each weight tile through L2; beyond that the prefill kernel is faster (measured: 56.6 against 45.5 k tok/s
@@ -1380,7 +1431,8 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
             const int esz = (epi == EPI_F32 || epi == EPI_ADD_F32) ? 4 : 2;
             const int vec = ((uintptr_t)out % 16 == 0) && ((size_t)ldc * esz % 16 == 0);
             if (ss_tiles_out) *ss_tiles_out = (N + 127) / 128;
-            GemmArgs fin{out, M, N, K, ldc, kbs, vec, ss_in, ss_tiles, ss_size, ss_eps, norm_w, (bf16 *)xw_out, ss_out, epi, 0, 0, S, act};
+            GemmArgs fin{out, M, N, K, ldc, kbs, vec, ss_in, ss_tiles, ss_size, ss_eps, norm_w, (bf16 *)xw_out, ss_out, epi, 0, 0, S, act, nullptr, gate.table,
+                         gate.tokens, gate.ld, gate.col};
             dim3 grid((N + 127) / 128, (M + 7) / 8);
             const float *ws = (const float *)workspace;
             // The second kernel starts in plain stream order, when the partial products are complete.  Launched as a
@@ -1442,7 +1494,7 @@ extern "C" int fg_gemm_tc_ws(const void *X, int ldx, const void *W, int ldw, voi
     int vec_ok = ((uintptr_t)out % 16 == 0) && ((size_t)ldc * esz % 16 == 0);
     if (ss_tiles_out) *ss_tiles_out = (int)grid.y * (bn < 0 && epi == EPI_ADD_F32 ? 2 : 1);
     GemmArgs a{out, M, N, K, ldc, kb_per_split, vec_ok, ss_in, ss_tiles, ss_size, ss_eps, norm_w, (bf16 *)xw_out, ss_out, epi, 0,
-               g_test_skip_copy, 0, act};
+               g_test_skip_copy, 0, act, nullptr, gate.table, gate.tokens, gate.ld, gate.col};
     switch (epi) {
     case EPI_BF16: return dispatch<EPI_BF16>(swap, bn, tmP, tmQ, a, grid, stream);
     case EPI_F32: return dispatch<EPI_F32>(swap, bn, tmP, tmQ, a, grid, stream);

@@ -206,6 +206,24 @@ Tensor Linear::forward_relu2(Runtime &rt, const Tensor &a) const {
     return t;
 }
 
+bool Linear::forward_gelu_gather(Runtime &rt, const Tensor &a, const Tensor &table, const int *tokens, int64_t col, Tensor *out) const {
+    const Tensor &W = w_.t;
+    if (!fast_ || rt.plain_kernels || a.dtype != FG_BF16 || table.dtype != FG_BF16) return false;
+    const int64_t M = a.rows, K = a.cols, N = W.rows;
+    Tensor t = rt.arena->matrix(M, N, FG_BF16);
+    if (M == 0) { *out = t; return true; }
+    count_launch();
+    ProfileScope scope("fg_gemm_tc", profile_on() ? format("%lld x %lld, %lld rows, gelu x table", (long long)N, (long long)K, (long long)M).c_str() : nullptr);
+    const long long ws_bytes = FG_KERNEL("tc", fg_gemm_tc_workspace_bytes)((int)M, (int)N, (int)K, EPI_BF16);
+    void *ws = ws_bytes > 0 ? rt.arena->alloc((size_t)ws_bytes) : nullptr;
+    int code = FG_KERNEL("tc", fg_gemm_tc_gelu_gather)(a.data, (int)a.ld, W.data, (int)W.ld, t.data, (int)t.ld, (int)M, (int)N, (int)K, table.data,
+                                                       (int)table.ld, (int)col, tokens, ws, ws_bytes, rt.stream);
+    if (code == KERNEL_BAD_SIZE) return false;
+    check_kernel(code, "fg_gemm_tc (gelu x table)");
+    *out = t;
+    return true;
+}
+
 bool Linear::forward_gated(Runtime &rt, const Tensor &a_in, const DeferredNorm *deferred, int act, Tensor *out) const {
     static const int epi_of[3] = {EPI_SILU_MUL, EPI_GELU_MUL, EPI_RELU_MUL};
     static const char *name_of[3] = {"silu", "gelu", "relu"};
@@ -938,7 +956,8 @@ private:
 // them by the stream, projects them to the width and adds the normalised result:
 //     g = gelu_tanh(W_gate x) * e,   y = W_proj g,   x <- x + y / sqrt(mean(y^2) + eps) * w
 // x is the stream itself (no norm in front).  The residual sum and the norm's statistics are 32-bit; in bfloat16 the stream is
-// rounded for the gate contraction as every contraction's input is, and its float32 result meets gelu and e in float32.
+// rounded for the gate contraction as every contraction's input is (by the contraction that writes the stream, where it can), and its
+// float32 result meets gelu and e in float32 - in the contraction's epilogue, where that runs on the tensor cores.
 class GatedTokenEmbedding : public TokenInput {
 public:
     GatedTokenEmbedding(const Json &p) {
@@ -975,10 +994,13 @@ public:
             xin = rt.arena->matrix(M, E_, rt.dtype);
             FG_LAUNCH("core", fg_cast_rows, x.ptr<float>(), (int)x.ld, xin.data, xin.dtype, (int)xin.ld, M, (int)E_, rt.stream);
         }
-        Tensor z = gate_.forward(rt, xin, nullptr, Tensor(), FG_F32, false, nullptr, nullptr);
-        Tensor g = rt.arena->matrix(M, D_, rt.dtype);
-        FG_LAUNCH("core", fg_gelu_mul_gather, z.ptr<float>(), (int)z.ld, table_.t.data, table_.t.dtype, (int)table_.t.ld, (int)col_, b.tokens, g.data,
-                  g.dtype, (int)g.ld, M, (int)D_, rt.stream);
+        Tensor g;
+        if (!gate_.forward_gelu_gather(rt, xin, table_.t, b.tokens, col_, &g)) {
+            Tensor z = gate_.forward(rt, xin, nullptr, Tensor(), FG_F32, false, nullptr, nullptr);
+            g = rt.arena->matrix(M, D_, rt.dtype);
+            FG_LAUNCH("core", fg_gelu_mul_gather, z.ptr<float>(), (int)z.ld, table_.t.data, table_.t.dtype, (int)table_.t.ld, (int)col_, b.tokens, g.data,
+                      g.dtype, (int)g.ld, M, (int)D_, rt.stream);
+        }
         Tensor y = proj_.forward(rt, g, nullptr, Tensor(), FG_F32, false, nullptr, nullptr);
         if (reader && !(reader->deferrable() && reader->weight() && reader->size() == E_ && E_ * (int64_t)sizeof(float) <= 48 * 1024)) reader = nullptr;
         if (reader) {

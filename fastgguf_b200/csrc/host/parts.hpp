@@ -272,6 +272,8 @@ public:
     // max(a W^T, 0)^2 in the activation dtype: in the tensor-core kernel's epilogue where that kernel runs, else the
     // contraction and an elementwise pass
     Tensor forward_relu2(Runtime &rt, const Tensor &a) const;
+    // gelu_tanh(a W^T)[m, n] * table[tokens[m], col + n] as bf16, in the tensor-core kernel's epilogue; false if refused
+    bool forward_gelu_gather(Runtime &rt, const Tensor &a, const Tensor &table, const int *tokens, int64_t col, Tensor *out) const;
     // act(a gate^T) * (a up^T) as bf16 [M, F] from rows interleaved in blocks of 64, act by its number in GatedAct; false if refused
     bool forward_gated(Runtime &rt, const Tensor &a, const DeferredNorm *deferred, int act, Tensor *out) const;
 
