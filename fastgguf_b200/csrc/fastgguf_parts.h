@@ -22,7 +22,8 @@
  *                                                               name a layer twice (a cache of its own each
  *                                                               time) or read an EARLIER entry's cache;
  *                                                               "reenter": true runs the spec's "reentry" part on
- *                                                               the stream in front of the entry
+ *                                                               the stream in front of the entry ("pass": the number of the
+ *                                                               pass of a looped span that begins there, default 0)
  *    "reentry": PART (optional),                                x <- f(x, the embedding's output), role stream_map
  *    "stop_token_ids": [...], "ignored_tensors": ["regex", ...]}
  *   PART = {"kind": "rmsnorm", "params": {...}, "tensors": {"local name": "checkpoint name"}}
@@ -31,31 +32,36 @@
  *
  * Built-in kinds
  *   norm          "rmsnorm"        {size, eps, offset: 0.0, gain: 1.0}     y = x / rms(x) * gain * (offset + w)
- *   position      "rope"           {head_dim, theta, scaling: null | {rope_type: "llama3", ...} | {rope_type: "yarn", factor,
+ *   position      "rope"           {head_dim, theta, scaling: null | {rope_type: "linear", factor} | {rope_type: "llama3", ...} | {rope_type: "yarn", factor,
  *                                   original_max_position_embeddings, beta_fast, beta_slow},
  *                                   rotary_dim: head_dim, layout: "halves" | "adjacent"}
  *   mixer         "gqa_attention"  {hidden_size, n_heads, n_kv_heads, head_dim, position: PART | null,
  *                                   scale: null = 1/sqrt(head_dim), window: null, keep_first: 0,
  *                                   v_head_dim: head_dim}        tensors q/k/v/o_proj.weight
  *                 "retention"      {hidden_size, n_heads, head_dim, v_head_dim, decay: [per head], position: PART | null,
- *                                   k_scale: null = 1/sqrt(head_dim), eps}   linear attention with a fixed decay per
- *                                   head, state [heads, head_dim, v_head_dim] float32 per sequence; tensors
- *                                   q/k/v/g/o_proj.weight
+ *                                   k_scale: null = 1/sqrt(head_dim), eps, qkv_activation: null | "silu", norm: "head" |
+ *                                   "whole", gate_activation: "silu" | "sigmoid"}   linear attention with a fixed decay per
+ *                                   head, state [heads, head_dim, v_head_dim] float32 per sequence; a unit norm per head, or one
+ *                                   over all heads with a weight (then the gate may be a sigmoid); tensors
+ *                                   q/k/v/g/o_proj.weight, norm.weight (norm "whole")
  *                 "gated_linear_attention"  {hidden_size, n_heads, head_dim, v_head_dim, tau, q_scale, eps, decay_rank: from the
  *                                   checkpoint}   a decay per key channel and token, sigmoid(low-rank(h) + b)^(1/tau); state as
  *                                   retention's; tensors q/k/v/g/o_proj.weight, decay_down/up.weight, decay_up.bias, norm.weight
  *                 "sink_attention" {hidden_size, n_heads, n_kv_heads, head_dim, v_head_dim, scale, window: 0, softcap: 0,
  *                                   chunk: 0, conv_taps: 0, bias: false, o_bias: false, sink: false, unit_sink: false,
- *                                   qk_norm: null | "whole" | "head", gate: null | "head" | "full", eps, position: PART | null}
+ *                                   qk_norm: null | "whole" | "head", gate: null | "head" | "full", values: null | "keys",
+ *                                   differential: null | d, eps, position: PART | null}
  *                                   grouped-query attention with biases, a short convolution over time (its last inputs are
  *                                   per-sequence state), norms over the whole of q and of k ("whole": weights [heads * head_dim])
  *                                   or per head ("head": one weight [head_dim] for all heads), rotation in the position part's
  *                                   layout (adjacent pairs, or halves of the rotated part), capped scores, a sink, a sigmoid
  *                                   gate per head from the mixer's input ("head": g_proj.weight [heads, hidden]) or per number
  *                                   ("full": [heads * v_head_dim, hidden]); chunk c instead of a window: a row sees the keys of
- *                                   its run of c positions counted from the sequence's first; unit_sink: a sink of score 0; tensors
+ *                                   its run of c positions counted from the sequence's first; unit_sink: a sink of score 0; values "keys": the values are the
+ *                                   keys as projected; differential: two maps a head over the same values, subtracted with weight
+ *                                   exp(lq1 . lk1) - exp(lq2 . lk2) + d, normalised per head, times 1 - d; tensors
  *                                   q/k/v/o_proj.weight, q/k/v_proj.bias, o_proj.bias, q/k/v_conv.weight, q/k_norm.weight,
- *                                   sinks, g_proj.weight
+ *                                   sinks, g_proj.weight, lambda_q1/k1/q2/k2
  *                 "latent_attention" {hidden_size, n_heads, head_dim, rot_dim, v_head_dim, kv_rank, q_rank, scale, eps,
  *                                   sink: false, gate: false, shared_kv: false, position: PART}   keys and values from one latent
  *                                   a token plus a shared rotated key part (only those are cached); shared_kv: no latent of its
@@ -80,7 +86,7 @@
  *                                   normalize: false, eps}   two mixers on the same rows, y = left_scale f(left) + right_scale
  *                                   f(right), f an RMS norm over the width with a weight where normalize is true; tensors
  *                                   left.<the left mixer's>, right.<the right mixer's>, left_norm.weight, right_norm.weight
- *   feed_forward  "swiglu"         {hidden_size, d_ff, activation: "silu" | "gelu_tanh"}   down(act(gate x) * (up x))
+ *   feed_forward  "swiglu"         {hidden_size, d_ff, activation: "silu" | "gelu_tanh" | "relu"}   down(act(gate x) * (up x))
  *                 "mlp"            {hidden_size, d_ff, activation: "relu2"}   down(act(up x))
  *                 "moe"            {hidden_size, d_ff, n_experts, top_k, limit, alpha: 1.702, router: "sigmoid_input"}
  *                                   tensors router.weight, experts.<e>.gate/up/down_proj.weight
@@ -103,6 +109,7 @@
  *                                   column + dim), y = W_proj (gelu_tanh(W_gate x) * e), x <- x + y / rms(y) * w; tensors table
  *                                   [vocab, table_dim] (layers may share it), gate [dim, E], proj [E, dim], norm [E]
  *   stream_map    "concat_linear"  {hidden_size}   x <- W [x; embedding output], W [E, 2 E]; tensor weight
+ *                 "add_row"        {hidden_size, rows}   x <- x + table[pass], table [rows, E]; tensor table
  *   embedding     "embedding"      {vocab_size, hidden_size, scale: 1.0}
  *   head          "lm_head"        {vocab_size, hidden_size, softcap: null}   logits <- cap tanh(logits / cap)
  *

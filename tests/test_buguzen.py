@@ -100,6 +100,8 @@ MIXERS = {
     "lightning, small": lightning(3, 16, 24, [0.5, 0.93, 0.999]),
     "lightning, odd sizes, one head that forgets at once": lightning(4, 9, 13, [0.0, 0.7, 1.0, 0.995]),
     "lightning, one head": lightning(1, 40, 8, [0.97]),
+    "lightning, a state larger than a block holds": lightning(1, 180, 300, [0.9]),
+    "lightning, values of more numbers than a block has threads": lightning(2, 9, 330, [0.97, 0.0]),
     "long two maps, keys of 64 beside values of 128": differential(4, 2, 64, 128, 0.125, 0.55, size=70, rot=(300000.0, 16)),
     "long two maps, 64 and 64, groups of three": differential(6, 2, 64, 64, 0.2, 0.3, rot=(1000.0, 64), scaling=(2.0,)),
     "long two maps, 128 and 128": differential(2, 1, 128, 128, 0.09, 0.45, size=129, rot=(1000.0, 32)),
@@ -196,6 +198,73 @@ def test_layer_with_everything(tmp_path, ff, side, rows, dtype):
     err = np.array([rel_err(got[r], want[r]) for r in range(rows)])
     assert (err > (2e-5 if dtype == "float32" else 5e-2)).sum() <= rows // 25, np.sort(err)[-5:]
     assert apart(got, mid.numpy()) > 1e-2            # what stands behind the mixer is there
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("rows", [3, 40, 200, 1100])
+def test_token_input_at_a_real_width(rows, dtype):
+    """x + norm(P (gelu(G x) * e)) at sizes where the gate contraction runs on few rows, split along a cluster, and split along K
+    through scratch memory, with the table's entry in its epilogue."""
+    from fastgguf_b200.parts import run_part
+    E, V, D, layer, n_layers = 2048, 90, 136, 1, 3
+    g = torch.Generator().manual_seed(41)
+    Wb = {"side.embed": torch.randn(V, D * n_layers, generator=g), "gate": torch.randn(D, E, generator=g) / E ** 0.5 * 2.0,
+          "proj": torch.randn(E, D, generator=g) / D ** 0.5, "norm": 1.0 + 0.3 * torch.randn(E, generator=g)}
+    Wb = {k: v.to(torch.bfloat16) for k, v in Wb.items()}
+    W = {("s." + k if k != "side.embed" else k): v.double() for k, v in Wb.items()}
+    x = torch.randn(rows, E, generator=g, dtype=torch.float64)
+    toks = [int(v) for v in torch.randint(0, V, (rows,), generator=g)]
+    want = pb.token_input(x, torch.tensor(toks), W, "s.", layer, D, 1e-4).numpy()
+    params = dict(hidden_size=E, vocab_size=V, dim=D, column=layer * D, table_dim=n_layers * D, eps=1e-4)
+    got = run_part("token_input", "gated_token_embedding", params, {"table": Wb["side.embed"], "gate": Wb["gate"], "proj": Wb["proj"], "norm": Wb["norm"]},
+                   dtype, tokens=toks, x=f32(x))
+    for r in range(rows):
+        assert rel_err(got[r], want[r]) < (1e-5 if dtype == "float32" else 2e-2), r
+
+
+@pytest.mark.parametrize("dim,vdim", [(64, 64), (64, 128), (128, 64), (128, 128)])
+def test_the_tensor_core_recurrence_keeps_float32(tmp_path, dim, vdim):
+    """In bfloat16, with projections that bfloat16 holds exactly, what the chunked and the single-token forms return differs from the
+    float64 recurrence over the SAME rounded activations by float32 rounding only: state, decays and weighted scores are not rounded
+    to bfloat16 on the way.  (o times a norm and a gate of one is read off the stream, whose sum is float32.)"""
+    H = 2
+    layer = lightning(H, dim, vdim, [0.9, 0.999])
+    E, V = 256, H * vdim
+    cfg = one_layer(layer, width=E)
+
+    def change(W):
+        g = torch.Generator().manual_seed(2)
+        W["l0.norm1"] = torch.ones_like(W["l0.norm1"])
+        for n in ("q", "k", "v"):
+            # one input a row, so that a projection is one product: exact in bfloat16 for inputs and weights that are powers of two
+            w = torch.zeros_like(W["l0.mix." + n])
+            w[torch.arange(w.shape[0]), torch.randint(0, E, (w.shape[0],), generator=g)] = 1.0
+            W["l0.mix." + n] = w
+        W["l0.mix.g"] = torch.zeros_like(W["l0.mix.g"])
+        W["l0.mix.norm"] = torch.ones_like(W["l0.mix.norm"])
+        W["l0.mix.o"] = torch.zeros_like(W["l0.mix.o"])
+        W["l0.mix.o"][torch.arange(V) % E, torch.arange(V)] = 1.0
+    d, W = make_model(tmp_path, cfg, 4, change=change)
+    T = 200
+    g = torch.Generator().manual_seed(3)
+    x = torch.randint(0, 2, (T, E), generator=g).double() * 2.0 - 1.0            # rows of +-1: the norm leaves them (1 / sqrt(1 + eps))
+    act = lambda z: pb.silu(z).to(torch.bfloat16).double()
+    h = x.to(torch.bfloat16).double()
+    q, k, v = (act(h @ W["l0.mix." + n].T).view(T, H, -1) for n in ("q", "k", "v"))
+    o = pb.decayed_sums(q, k, v, torch.tensor([0.9, 0.999], dtype=torch.float64)).reshape(T, V)
+    y = (pb.rms_norm(o, 1.0, EPS) * 0.5).to(torch.bfloat16).double()             # what the output projection reads
+    want = (x + y @ W["l0.mix.o"].T).numpy()
+    for cuts in ([T], [70, 2, 100] + [1] * 28):
+        eng = engine_for(d, "bfloat16")
+        s, at, got = eng.acquire(), 0, []
+        for n in cuts:
+            got.append(eng.block_forward(0, [(s, n)], f32(x[at:at + n])))
+            at += n
+        got = np.concatenate(got)
+        # a bfloat16 rounding of y may fall to the other side of a tie; nearly every number agrees to float32
+        same = np.abs(got - want) < 1e-5 * np.abs(want).max()
+        assert same.mean() > 0.995, (cuts[:3], same.mean())
+        assert np.abs(got - want).max() < 2.0 ** -7 * np.abs(want).max()
 
 
 def test_the_relu_gate_shuts(tmp_path):
