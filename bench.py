@@ -245,9 +245,9 @@ def buguzen_config(width, heads, kv_heads, head_dim, ff, vocab, window, expert_f
     del heads, kv_heads, head_dim, expert_ff
     H = width // 128
     one = {"heads": H, "kv_heads": H // 4, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "mask": {"size": window},
-           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0}}}
+           "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 2.0}}}
     two = {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
-           "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+           "rot": {"base": 200000.0, "dims": 64, "scaling": {"factor": 16.0, "low": 1.0, "high": 3.0, "original": 8192}}}
     lin = {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 6 * h / max(1, H - 1)) for h in range(H)]}
     dense = {"kind": "dense", "ff": ff}
     layers = []

@@ -633,7 +633,7 @@ def test_many_steps_back_to_back():
     from fastgguf_b200.registry import config_from_dict
     cfg = config(1024, 4096, [
         (differential(8, 4, 64, 128, 0.125, 0.5, size=512, rot=(10000.0, 32), scaling=(2.0,)), 4096),
-        (keys_as_values(8, 2, 128, 0.09, size=700, rot=(500000.0, 64), scaling=(8.0, 1.0, 4.0, 1024)), 4096),
+        (keys_as_values(8, 2, 128, 0.09, size=700, rot=(200000.0, 64), scaling=(16.0, 1.0, 3.0, 2048)), 4096),
         (lightning(8, 128, 128, [0.5, 0.8, 0.9, 0.95, 0.98, 0.99, 0.995, 0.999]), 4096),
         (lightning(8, 64, 128, [0.5, 0.8, 0.9, 0.95, 0.98, 0.99, 0.995, 0.999]), None),
     ], loop=(0, 4, 2), side=256)
